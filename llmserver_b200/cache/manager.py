@@ -6,8 +6,8 @@ mixer that keeps several things: two state tensors, or pages beside state); the 
 nothing about models.  Schedule entries with the same page shape and the same window form one
 *group* with a page pool, a storage tensor and per-request block tables of its own, so a group
 that keeps every key and a group that keeps only a window can grow and shrink independently.
-Pages are given back when a request ends and, in windowed groups, as soon as the window has
-passed them; they are reused by later allocations.
+Pages are given back when a request ends and, in windowed or chunked groups, as soon as the window (or the
+chunk) has passed them; they are reused by later allocations.
 
 The reference has one cache shape for all layers (utils/engine.py:77-85, utils/kv_cache.py:84-89)
 and no per-request state in its paged path; groups and state slots are this engine's own.  Storage
@@ -31,14 +31,18 @@ class KVPagesNeed:
     """Keys and values of ``kv_heads`` heads of ``head_dim``; ``window`` None keeps all tokens,
     else only the last ``window`` tokens are ever read.  ``value_dim``: the size of a value head where it differs
     from a key head's (None: the same).  ``keys_only``: what is cached serves as key and as value (a latent from which
-    both are made): one tensor is kept and handed out as both."""
+    both are made): one tensor is kept and handed out as both.  ``chunk``: positions are cut into chunks of that many from
+    0 on and a query only ever reads keys of its own chunk, so everything in front of the chunk is done with."""
     kv_heads: int
     head_dim: int
     window: Optional[int] = None
     value_dim: Optional[int] = None
     keys_only: bool = False
+    chunk: Optional[int] = None
 
     def __post_init__(self):
+        if self.chunk is not None and (self.window is not None or int(self.chunk) <= 0):
+            raise ValueError("a cache is bounded by a window or by chunks of a positive size, not by both")
         if self.keys_only and self.value_dim is not None:
             raise ValueError("a cache of keys alone has no value size of its own")
         if self.value_dim is not None and int(self.value_dim) == int(self.head_dim):
@@ -71,6 +75,11 @@ class CacheGroup:
     def window(self) -> Optional[int]:
         return self.need.window
 
+    @property
+    def gives_back(self) -> bool:
+        """Whether pages are given back before their request ends."""
+        return self.need.window is not None or self.need.chunk is not None
+
     def pages_for(self, request_id, total_tokens: int) -> int:
         """Pages to allocate so that positions < total_tokens have a slot."""
         table = self.tables[request_id]
@@ -78,6 +87,8 @@ class CacheGroup:
 
     def passed_pages(self, num_computed: int) -> int:
         """Number of leading pages no later query can read when ``num_computed`` tokens are done."""
+        if self.need.chunk is not None:      # the query at position num_computed sees its own chunk
+            return num_computed // self.need.chunk * self.need.chunk // self.page_size
         if self.window is None:
             return 0
         first_needed = num_computed - self.window + 1  # earliest key of the query at position num_computed
@@ -155,7 +166,7 @@ class CacheManager:
                 raise TypeError(f"schedule entry {entry}: unknown cache need {need!r}")
         self.slots = StateSlots(num_slots)
         self.requests: Dict[object, int] = {}   # request -> tokens that have a slot in every group
-        self.has_windows = any(group.window is not None for group in self.groups)
+        self.has_windows = any(group.gives_back for group in self.groups)      # windows or chunks
         # A prefix can be skipped only if every layer's cache of it is at hand.  Groups that keep every key qualify:
         # what their pages hold is a function of the prefix alone, and each keeps a digest chain of its own.  A
         # windowed group gives pages back and per-request state is not kept in pages at all, so a model with
@@ -271,7 +282,7 @@ class CacheManager:
         self.requests[request_id] = max(self.requests[request_id], total_tokens)
 
     def advance(self, request_id, num_computed: int) -> int:
-        """Called after a step: gives back the pages of windowed groups that no later query of this
+        """Called after a step: gives back the pages of windowed and chunked groups that no later query of this
         request can read.  Returns how many pages were released."""
         if not self.has_windows:
             return 0

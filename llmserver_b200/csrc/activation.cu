@@ -16,12 +16,26 @@ __device__ __forceinline__ float silu_times(float gate, float up) {
     return gate / (1.0f + expf(-gate)) * up;
 }
 
+// gelu(x) * y in 32-bit, gelu in its tanh form 0.5 x (1 + tanh(u)) = x sigmoid(2 u), u = sqrt(2 / pi) (x + 0.044715 x^3).
+template <typename T>
+__device__ __forceinline__ float gelu_times(float gate, float up) {
+    const float u2 = 1.5957691216057308f * fmaf(0.044715f * gate * gate, gate, gate);
+    if (sizeof(T) == 2) return __fdividef(gate, 1.0f + __expf(-u2)) * up;
+    return gate / (1.0f + expf(-u2)) * up;
+}
+
+enum : int { GLU_SILU = 0, GLU_GELU = 1 };
+template <typename T, int ACT>
+__device__ __forceinline__ float gate_times(float gate, float up) {
+    return ACT == GLU_GELU ? gelu_times<T>(gate, up) : silu_times<T>(gate, up);
+}
+
 // Where output column `column` finds its gate value in a row of gate_up, and how far behind the up value lies.
 __device__ __forceinline__ int gate_column(int column, int group) {
     return group > 0 ? (column / group) * 2 * group + column % group : column;
 }
 
-template <typename T>
+template <typename T, int ACT>
 __global__ void silu_mul_vec_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int intermediate,
                                     size_t total_vectors, int group) {
     pdl_trigger();   // let the next kernel start launching
@@ -45,17 +59,17 @@ __global__ void silu_mul_vec_kernel(const T* __restrict__ gate_up, T* __restrict
         Vec16<T>::load(src_w, gate_w);
         Vec16<T>::load(src_w + to_up, up_w);
 #pragma unroll
-        for (int i = 0; i < kCount; ++i) result[i] = silu_times<T>(gate_v[i], up_v[i]);
+        for (int i = 0; i < kCount; ++i) result[i] = gate_times<T, ACT>(gate_v[i], up_v[i]);
         Vec16<T>::store(out + row_v * (size_t)intermediate + column_v, result);
         if (second) {
 #pragma unroll
-            for (int i = 0; i < kCount; ++i) result[i] = silu_times<T>(gate_w[i], up_w[i]);
+            for (int i = 0; i < kCount; ++i) result[i] = gate_times<T, ACT>(gate_w[i], up_w[i]);
             Vec16<T>::store(out + row_w * (size_t)intermediate + column_w, result);
         }
     }
 }
 
-template <typename T>
+template <typename T, int ACT>
 __global__ void silu_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int intermediate, size_t total, int group) {
     pdl_trigger();   // let the next kernel start launching
     pdl_wait();      // everything before this kernel in the stream is complete and visible
@@ -65,15 +79,15 @@ __global__ void silu_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ o
         const T* src = gate_up + row * 2 * (size_t)intermediate + gate_column(column, group);
         const float gate = Num<T>::load(src);
         const float up = Num<T>::load(src + (group > 0 ? group : intermediate));
-        Num<T>::store(out + e, gate / (1.0f + expf(-gate)) * up);
+        Num<T>::store(out + e, ACT == GLU_GELU ? gelu_times<float>(gate, up) : gate / (1.0f + expf(-gate)) * up);
     }
 }
 
-LLM_EXPORT int llm_silu_mul(const void* gate_up, void* out, int n_rows, int intermediate, int group, int dtype,
-                            cudaStream_t stream) {
+template <int ACT>
+static int glu_launch(const void* gate_up, void* out, int n_rows, int intermediate, int group, int dtype, cudaStream_t stream) {
     if (n_rows == 0 || intermediate == 0) return LLM_OK;
     if (group < 0 || (group > 0 && intermediate % group)) {
-        llm_set_error("silu_mul: the intermediate size %d is no multiple of the group %d", intermediate, group);
+        llm_set_error("silu_mul / gelu_mul: the intermediate size %d is no multiple of the group %d", intermediate, group);
         return LLM_REFUSED;
     }
     const int per_vector = dtype == LLM_F32 ? 4 : 8;
@@ -84,13 +98,22 @@ LLM_EXPORT int llm_silu_mul(const void* gate_up, void* out, int n_rows, int inte
     if (vector_form) blocks = (blocks + 1) / 2;      // two vectors per thread and turn
     if (blocks > 148 * 16) blocks = 148 * 16;
     if (vector_form) {
-        LLM_DISPATCH_DTYPE(dtype, (llm_launch(silu_mul_vec_kernel<T>, (unsigned)blocks, threads, 0, stream, 
+        LLM_DISPATCH_DTYPE(dtype, (llm_launch(silu_mul_vec_kernel<T, ACT>, (unsigned)blocks, threads, 0, stream,
                                       (const T*)gate_up, (T*)out, intermediate, work, group)));
     } else {
-        LLM_DISPATCH_DTYPE(dtype, (llm_launch(silu_mul_kernel<T>, (unsigned)blocks, threads, 0, stream, 
+        LLM_DISPATCH_DTYPE(dtype, (llm_launch(silu_mul_kernel<T, ACT>, (unsigned)blocks, threads, 0, stream,
                                       (const T*)gate_up, (T*)out, intermediate, work, group)));
     }
-    return llm_check_launch("silu_mul");
+    return llm_check_launch(ACT == GLU_GELU ? "gelu_mul" : "silu_mul");
+}
+
+LLM_EXPORT int llm_silu_mul(const void* gate_up, void* out, int n_rows, int intermediate, int group, int dtype, cudaStream_t stream) {
+    return glu_launch<GLU_SILU>(gate_up, out, n_rows, intermediate, group, dtype, stream);
+}
+
+// The same layouts with gelu (tanh form) in silu's place.
+LLM_EXPORT int llm_gelu_mul(const void* gate_up, void* out, int n_rows, int intermediate, int group, int dtype, cudaStream_t stream) {
+    return glu_launch<GLU_GELU>(gate_up, out, n_rows, intermediate, group, dtype, stream);
 }
 
 // Point-wise steps that stand alone (32-bit arithmetic, one rounding on the store):

@@ -16,6 +16,10 @@
 // Values may have another size than keys (`value_dim`; the output then has Hq * value_dim columns).  With `sinks`
 // (one 32-bit number per query head) the softmax's denominator also holds exp(sinks[h]): a score without a key
 // and without a value, not scaled, counted once.
+//
+// With `chunk` > 0 the sequence is cut into chunks of that many positions and a query sees the keys of its own chunk
+// only (from (p / chunk) * chunk on).  With `bias` (32-bit [Hq, bias_len]) the score of the key n positions back gets
+// bias[h][min(n, bias_len - 1)] added, which the scale does not multiply.
 #include "common.cuh"
 
 #define ATTN_MAX_D 512
@@ -27,6 +31,7 @@ __global__ void attention_generic_kernel(const T* __restrict__ q, int q_stride, 
                                          const int* __restrict__ positions, T* __restrict__ out, int n_q_heads,
                                          int n_kv_heads, int head_dim, int value_dim, int page_size, int num_pages,
                                          float scale, int window, const float* __restrict__ sinks,
+                                         int chunk, const float* __restrict__ bias, int bias_len,
                                          int* __restrict__ error_flag) {
     pdl_trigger();   // let the next kernel start launching
     pdl_wait();      // everything before this kernel in the stream is complete and visible
@@ -50,7 +55,8 @@ __global__ void attention_generic_kernel(const T* __restrict__ q, int q_stride, 
     for (int i = 0; i < ATTN_MAX_D / 32; ++i) accumulator[i] = 0.0f;
     float running_max = -INFINITY, normaliser = 0.0f;
 
-    const int first = (window > 0 && position - window + 1 > 0) ? position - window + 1 : 0;
+    int first = (window > 0 && position - window + 1 > 0) ? position - window + 1 : 0;
+    if (chunk > 0) first = max(first, position / chunk * chunk);
     for (int base = first; base <= position; base += 32) {
         const int key = base + lane;
         const bool valid = key <= position;
@@ -67,6 +73,7 @@ __global__ void attention_generic_kernel(const T* __restrict__ q, int q_stride, 
             float dot = 0.0f;
             for (int d = 0; d < head_dim; ++d) dot += q_row[d] * Num<T>::load(k_row + d);
             score = dot * scale;
+            if (bias) score += bias[(size_t)head * bias_len + min(position - key, bias_len - 1)];
         }
         const float chunk_max = warp_max(score);
         const float new_max = fmaxf(running_max, chunk_max);
@@ -109,7 +116,7 @@ LLM_EXPORT int llm_attention_generic(const void* q, int q_stride, const void* k_
                                      const int* block_tables, int max_blocks, const int* seq_of_token,
                                      const int* positions, void* out, int n_tokens, int n_q_heads, int n_kv_heads,
                                      int head_dim, int value_dim, int page_size, int num_pages, float scale, int window,
-                                     const float* sinks, int* error_flag, int dtype, cudaStream_t stream) {
+                                     const float* sinks, int chunk, const float* bias, int bias_len, int* error_flag, int dtype, cudaStream_t stream) {
     if (n_tokens == 0) return LLM_OK;
     if (head_dim > ATTN_MAX_D || head_dim <= 0) {
         llm_set_error("attention_generic: head_dim %d is outside 1..%d", head_dim, ATTN_MAX_D);
@@ -127,12 +134,16 @@ LLM_EXPORT int llm_attention_generic(const void* q, int q_stride, const void* k_
         llm_set_error("attention_generic: %d query heads are no multiple of %d kv heads", n_q_heads, n_kv_heads);
         return LLM_REFUSED;
     }
+    if (chunk < 0 || (bias && bias_len <= 0)) {
+        llm_set_error("attention_generic: a chunk of %d positions or a bias of %d distances", chunk, bias_len);
+        return LLM_REFUSED;
+    }
     const int warps = 4;
     dim3 grid(n_tokens, (n_q_heads + warps - 1) / warps);
     const size_t shared = (size_t)warps * head_dim * sizeof(float);
     LLM_DISPATCH_DTYPE(dtype, (llm_launch(attention_generic_kernel<T>, grid, warps * 32, shared, stream, 
                                   (const T*)q, q_stride, (const T*)k_pages, (const T*)v_pages, block_tables,
                                   max_blocks, seq_of_token, positions, (T*)out, n_q_heads, n_kv_heads, head_dim,
-                                  value_dim, page_size, num_pages, scale, window, sinks, error_flag)));
+                                  value_dim, page_size, num_pages, scale, window, sinks, chunk, bias, bias_len, error_flag)));
     return llm_check_launch("attention_generic");
 }

@@ -25,7 +25,10 @@
 // The cp.async kernels also come in a form for models whose attention weights have to stay 32-bit and whose softmax
 // has a sink (llm_attention_mma_sinks): values may have another size than keys (each 64 or 128), every probability
 // enters the P V product as the sum of two bfloat16 numbers (its rounding and the rounding of what that left over:
-// 16 significant bits, two MMAs instead of one), and exp(sink) joins the denominator once per row.
+// 16 significant bits, two MMAs instead of one), and exp(sink) joins the denominator once per row.  That form also
+// takes attention in chunks (a query sees the keys of its own chunk of positions only) and a learned bias per head and
+// distance between query and key, added to the scaled score (BIAS): the group's rows of the bias are staged in shared
+// memory, or read where they lie when they are too long for it.
 #include "common.cuh"
 #include "tma.cuh"
 #include "tcgen05.cuh"
@@ -67,7 +70,32 @@ struct AttnParams {
                              // of the pool; 6: a context needs more splits than max_splits (may be null)
     const float* sinks = nullptr;   // [Hq] or null: one more term exp(sinks[h]) in head h's softmax denominator (a score
                                     // without key or value, neither scaled nor masked); cp.async kernels only
+    int chunk = 0;                  // > 0: a query at position p sees keys (p / chunk) * chunk .. p only
+    const float* bias = nullptr;    // [Hq, bias_len], times log2(e): added to the score of the key n positions back, n
+    int bias_len = 0;               // at most bias_len - 1 (farther keys: the last entry); BIAS kernels only
+    int bias_stride = 0;            // floats between two heads' staged rows; 0: the bias is not staged
+    int bias_offset = 0;            // where the staged rows lie in the kernel's shared memory (bytes)
 };
+
+// The first key that the query at `position` may see.
+__device__ __forceinline__ int first_visible(const AttnParams& p, int position) {
+    int low = p.window > 0 ? max(0, position - p.window + 1) : 0;
+    if (p.chunk > 0 && position >= 0) low = max(low, position / p.chunk * p.chunk);
+    return low;
+}
+
+// Stages the group's rows of the bias behind the tiles (the caller's next block barrier makes them visible) and returns
+// where a row's distances start, one pointer per row of the thread.
+__device__ __forceinline__ const float* stage_bias(const AttnParams& p, float* shared, int kv_head, int group, int* stride) {
+    if (p.bias_stride == 0) {
+        *stride = p.bias_len;
+        return p.bias + (size_t)kv_head * group * p.bias_len;
+    }
+    for (int e = threadIdx.x; e < group * p.bias_len; e += kThreads)
+        shared[e / p.bias_len * p.bias_stride + e % p.bias_len] = p.bias[(size_t)kv_head * group * p.bias_len + e];
+    *stride = p.bias_stride;
+    return shared;
+}
 
 // A block-table entry as the kernels may follow it: an entry that names no page of the pool is reported and replaced
 // by page 0, so nothing outside the pool is ever addressed (the keys it stands for are wrong, and the flag says so).
@@ -234,11 +262,12 @@ __device__ __forceinline__ void load_kv_tile(__nv_bfloat16* k_tile, __nv_bfloat1
 //
 // DV: the size of a value row (V tiles are laid out by VLayout).  PRECISE: each probability enters the P V product as
 // two bfloat16 numbers, its rounding and the rounding of the rest, so the weights keep 16 significant bits.
-template <int D, int NT, class Layout = XorLayout<D>, int DV = D, bool PRECISE = false, class VLayout = Layout>
+template <int D, int NT, class Layout = XorLayout<D>, int DV = D, bool PRECISE = false, class VLayout = Layout, bool BIAS = false>
 __device__ __forceinline__ void warp_tile(const uint32_t (&q_frag)[D / 16][4], const __nv_bfloat16* k_tile,
                                           const __nv_bfloat16* v_tile, int key_row, int key_index,
                                           const int (&row_low)[2], const int (&row_high)[2], float scale_log2,
-                                          float (&o_acc)[DV / 8][4], float (&row_max)[2], float (&row_sum)[2]) {
+                                          float (&o_acc)[DV / 8][4], float (&row_max)[2], float (&row_sum)[2],
+                                          const float* const* bias_row = nullptr, int bias_last = 0) {
     const int lane = threadIdx.x & 31;
     const int matrix = lane >> 3, matrix_row = lane & 7;
     float s_acc[NT][4];
@@ -270,7 +299,8 @@ __device__ __forceinline__ void warp_tile(const uint32_t (&q_frag)[D / 16][4], c
             const int h = i >> 1;
             const int key = key_index + n * 8 + 2 * t + (i & 1);
             const bool seen = key >= row_low[h] && key <= row_high[h];
-            s_acc[n][i] = seen ? s_acc[n][i] * scale_log2 : -INFINITY;
+            if (BIAS) s_acc[n][i] = seen ? fmaf(s_acc[n][i], scale_log2, bias_row[h][min(row_high[h] - key, bias_last)]) : -INFINITY;
+            else s_acc[n][i] = seen ? s_acc[n][i] * scale_log2 : -INFINITY;
             tile_max[h] = fmaxf(tile_max[h], s_acc[n][i]);
         }
     }
@@ -335,7 +365,7 @@ __device__ __forceinline__ void warp_tile(const uint32_t (&q_frag)[D / 16][4], c
 // ------------------------------------------------------------------------------------------------
 // portions of prompts
 // ------------------------------------------------------------------------------------------------
-template <int D, int DV = D, bool PRECISE = false>
+template <int D, int DV = D, bool PRECISE = false, bool BIAS = false>
 __global__ void __launch_bounds__(kThreads) attention_portions_kernel(const AttnParams p) {
     pdl_trigger();   // let the next kernel start launching
     pdl_wait();      // everything before this kernel in the stream is complete and visible
@@ -384,8 +414,7 @@ __global__ void __launch_bounds__(kThreads) attention_portions_kernel(const Attn
     const int last_token = last_row / group;
     const int base_position = context - q_len;
     const int high_key = base_position + last_token;
-    int low_key = 0;
-    if (p.window > 0) low_key = max(0, base_position + first_token - p.window + 1);
+    const int low_key = first_visible(p, base_position + first_token);
     const int first_tile_key = (low_key / kTileKeys) * kTileKeys;
     const int n_tiles = (high_key - first_tile_key) / kTileKeys + 1;
 
@@ -401,11 +430,18 @@ __global__ void __launch_bounds__(kThreads) attention_portions_kernel(const Attn
         if (r < n_rows) {
             const int position = base_position + r / group;
             row_high[h] = position;
-            row_low[h] = p.window > 0 ? max(0, position - p.window + 1) : 0;
+            row_low[h] = first_visible(p, position);
         } else {
             row_high[h] = -1;
             row_low[h] = 0;
         }
+    }
+    const float* bias_row[2] = {nullptr, nullptr};
+    if (BIAS) {
+        int stride;
+        const float* bias = stage_bias(p, reinterpret_cast<float*>(shared_raw + p.bias_offset), kv_head, group, &stride);
+#pragma unroll
+        for (int h = 0; h < 2; ++h) bias_row[h] = bias + (size_t)((first_row + warp * 16 + g + 8 * h) % group) * stride;
     }
     float o_acc[DV / 8][4];
 #pragma unroll
@@ -440,7 +476,7 @@ __global__ void __launch_bounds__(kThreads) attention_portions_kernel(const Attn
         const int tile_key = first_tile_key + it * kTileKeys;
         // a warp whose rows all end before this tile has nothing to add (the causal upper triangle)
         if (tile_key <= warp_high)
-            warp_tile<D, 8, XorLayout<D>, DV, PRECISE, XorLayout<DV>>(q_frag, k_tile, v_tile, 0, tile_key, row_low, row_high, p.scale_log2, o_acc, row_max, row_sum);
+            warp_tile<D, 8, XorLayout<D>, DV, PRECISE, XorLayout<DV>, BIAS>(q_frag, k_tile, v_tile, 0, tile_key, row_low, row_high, p.scale_log2, o_acc, row_max, row_sum, bias_row, p.bias_len - 1);
         __syncthreads();   // the stage is overwritten by the load issued in the next iteration
     }
 
@@ -480,7 +516,7 @@ __device__ __forceinline__ void zero_output(const AttnParams& p, int token, int 
         p.out[(size_t)token * p.n_q_heads * D + (size_t)(kv_head * group) * D + index] = __float2bfloat16_rn(0.0f);
 }
 
-template <int D, int DV = D, bool PRECISE = false>
+template <int D, int DV = D, bool PRECISE = false, bool BIAS = false>
 __global__ void __launch_bounds__(kThreads) attention_decode_kernel(const AttnParams p) {
     pdl_trigger();   // let the next kernel start launching
     pdl_wait();      // everything before this kernel in the stream is complete and visible
@@ -495,7 +531,7 @@ __global__ void __launch_bounds__(kThreads) attention_decode_kernel(const AttnPa
     const int group = p.n_q_heads / p.n_kv_heads;
     const int context = p.context_len[seq];
     const int position = context - 1;
-    const int low_key = p.window > 0 ? max(0, position - p.window + 1) : 0;
+    const int low_key = first_visible(p, position);
     const int first_key = (low_key / kTileKeys) * kTileKeys;
     const int split_len = split_length(p, context - first_key);
     const int n_splits = (context - first_key + split_len - 1) / split_len;
@@ -529,6 +565,13 @@ __global__ void __launch_bounds__(kThreads) attention_decode_kernel(const AttnPa
         row_high[h] = exists ? position : -1;
         row_low[h] = low_key;
     }
+    const float* bias_row[2] = {nullptr, nullptr};
+    if (BIAS) {
+        int stride;
+        const float* bias = stage_bias(p, reinterpret_cast<float*>(shared_raw + p.bias_offset), kv_head, group, &stride);
+#pragma unroll
+        for (int h = 0; h < 2; ++h) bias_row[h] = bias + (size_t)min(g + 8 * h, group - 1) * stride;
+    }
     float o_acc[DV / 8][4];
 #pragma unroll
     for (int n = 0; n < DV / 8; ++n)
@@ -561,7 +604,7 @@ __global__ void __launch_bounds__(kThreads) attention_decode_kernel(const AttnPa
         // each warp takes 16 of the tile's 64 keys
         const int key_index = split_begin + it * kTileKeys + warp * 16;
         if (key_index < split_end)
-            warp_tile<D, 2, XorLayout<D>, DV, PRECISE, XorLayout<DV>>(q_frag, k_tile, v_tile, warp * 16, key_index, row_low, row_high, p.scale_log2, o_acc, row_max, row_sum);
+            warp_tile<D, 2, XorLayout<D>, DV, PRECISE, XorLayout<DV>, BIAS>(q_frag, k_tile, v_tile, warp * 16, key_index, row_low, row_high, p.scale_log2, o_acc, row_max, row_sum, bias_row, p.bias_len - 1);
         __syncthreads();
     }
 
@@ -922,7 +965,7 @@ __global__ void attention_decode_merge_kernel(const AttnParams p) {
     const int token = p.q_start[seq];
     if (p.q_start[seq + 1] - token != 1) return;
     const int context = p.context_len[seq];
-    const int low_key = p.window > 0 ? max(0, context - p.window) : 0;
+    const int low_key = first_visible(p, context - 1);
     const int first_key = (low_key / kTileKeys) * kTileKeys;
     const int split_len = split_length(p, context - first_key);
     const int n_splits = min((context - first_key + split_len - 1) / split_len, p.max_splits);
@@ -941,38 +984,55 @@ __global__ void attention_decode_merge_kernel(const AttnParams p) {
     }
 }
 
-template <int D, int DV = D, bool PRECISE = false>
-int launch_portions(const AttnParams& p, int total_tiles, cudaStream_t stream) {
-    const size_t shared = (size_t)(kTileRows * D + 2 * kTileKeys * (D + DV)) * sizeof(__nv_bfloat16);
-    if (int limit_status = llm_raise_shared_limit(reinterpret_cast<const void*>(attention_portions_kernel<D, DV, PRECISE>), shared, "attention_portions")) return limit_status;
+// Where the group's rows of the bias go: behind `tiles` bytes of shared memory when they are short enough, else they
+// stay in global memory.  Returns the shared memory the kernel then needs.
+constexpr size_t kBiasSharedMax = 24 * 1024;
+size_t place_bias(AttnParams& p, size_t tiles) {
+    const int group = p.n_q_heads / p.n_kv_heads;
+    p.bias_offset = (int)((tiles + 15) / 16 * 16);
+    // rows eight banks apart: the rows a warp reads side by side (token, head of the group) then fall into different banks
+    const int stride = (p.bias_len + 31) / 32 * 32 + 8;
+    const size_t bytes = (size_t)group * stride * sizeof(float);
+    p.bias_stride = bytes <= kBiasSharedMax ? stride : 0;
+    return p.bias_stride ? p.bias_offset + bytes : tiles;
+}
+
+template <int D, int DV = D, bool PRECISE = false, bool BIAS = false>
+int launch_portions(const AttnParams& given, int total_tiles, cudaStream_t stream) {
+    AttnParams p = given;
+    size_t shared = (size_t)(kTileRows * D + 2 * kTileKeys * (D + DV)) * sizeof(__nv_bfloat16);
+    if (BIAS) shared = place_bias(p, shared);
+    if (int limit_status = llm_raise_shared_limit(reinterpret_cast<const void*>(attention_portions_kernel<D, DV, PRECISE, BIAS>), shared, "attention_portions")) return limit_status;
     dim3 grid(total_tiles, p.n_kv_heads);
-    llm_launch(attention_portions_kernel<D, DV, PRECISE>, grid, kThreads, shared, stream, p);
+    llm_launch(attention_portions_kernel<D, DV, PRECISE, BIAS>, grid, kThreads, shared, stream, p);
     return llm_check_launch("attention_portions");
 }
 
-template <int D, int DV = D, bool PRECISE = false>
-int launch_decode_cp_async(const AttnParams& p, cudaStream_t stream) {
+template <int D, int DV = D, bool PRECISE = false, bool BIAS = false>
+int launch_decode_cp_async(const AttnParams& given, cudaStream_t stream) {
+    AttnParams p = given;
     size_t shared = (size_t)(16 * D + 2 * kTileKeys * (D + DV)) * sizeof(__nv_bfloat16);
     const size_t merge = (size_t)4 * 16 * (DV + 2) * sizeof(float) + 16 * D * sizeof(__nv_bfloat16);
     if (merge > shared) shared = merge;
-    if (int limit_status = llm_raise_shared_limit(reinterpret_cast<const void*>(attention_decode_kernel<D, DV, PRECISE>), shared, "attention_decode")) return limit_status;
+    if (BIAS) shared = place_bias(p, shared);
+    if (int limit_status = llm_raise_shared_limit(reinterpret_cast<const void*>(attention_decode_kernel<D, DV, PRECISE, BIAS>), shared, "attention_decode")) return limit_status;
     dim3 grid(p.max_splits, p.n_kv_heads, p.n_seqs);
-    llm_launch(attention_decode_kernel<D, DV, PRECISE>, grid, kThreads, shared, stream, p);
+    llm_launch(attention_decode_kernel<D, DV, PRECISE, BIAS>, grid, kThreads, shared, stream, p);
     return llm_check_launch("attention_decode");
 }
 
 // The form with 32-bit-grade attention weights, sinks and a value size of its own: the cp.async kernels, splits merged
 // by the merge kernel.
-template <int D, int DV>
+template <int D, int DV, bool BIAS>
 int launch_precise(const AttnParams& p, int run_portions, int total_tiles, int run_decode, cudaStream_t stream) {
     int status = LLM_OK;
-    if (run_portions && total_tiles > 0) status = launch_portions<D, DV, true>(p, total_tiles, stream);
+    if (run_portions && total_tiles > 0) status = launch_portions<D, DV, true, BIAS>(p, total_tiles, stream);
     if (status != LLM_OK || !run_decode) return status;
     if (p.max_splits > 1 && (p.partial_out == nullptr || p.partial_ml == nullptr)) {
         llm_set_error("attention_decode: %d splits need the scratch buffers for partial results", p.max_splits);
         return LLM_REFUSED;
     }
-    status = launch_decode_cp_async<D, DV, true>(p, stream);
+    status = launch_decode_cp_async<D, DV, true, BIAS>(p, stream);
     if (status != LLM_OK || p.max_splits <= 1) return status;
     dim3 merge_grid(p.n_q_heads, p.n_seqs);
     llm_launch(attention_decode_merge_kernel<DV>, merge_grid, DV < 128 ? DV : 128, 0, stream, p);
@@ -1277,6 +1337,9 @@ LLM_EXPORT int llm_attention_mma_sinks_supports(int head_dim, int value_dim, int
     return n_q_heads / n_kv_heads <= 16;
 }
 
+// `chunk` > 0: a query sees the keys of its own chunk of positions only.  `bias` (float32 [Hq, bias_len], given times
+// log2(e); may be null): what is added to the score of the key n positions back, at min(n, bias_len - 1).
+//
 // Attention whose weights keep 16 significant bits in the P V product (see PRECISE above), with value heads of
 // `value_dim` elements and, with `sinks` (float32 [Hq], may be null), one more term exp(sinks[h]) in every row's
 // denominator.  The other arguments as for llm_attention_mma; out is [N, Hq * value_dim].
@@ -1284,7 +1347,7 @@ LLM_EXPORT int llm_attention_mma_sinks(const void* q, int q_stride, const void* 
                                        const int* block_tables, int max_blocks, const int* q_start, const int* context_len,
                                        void* out, int n_seqs, int n_q_heads, int n_kv_heads, int head_dim, int value_dim,
                                        int page_size, int num_pages, float scale, int window, const float* sinks,
-                                       int run_portions, int total_tiles, int run_decode, int split_len, int max_splits,
+                                       int chunk, const float* bias, int bias_len, int run_portions, int total_tiles, int run_decode, int split_len, int max_splits,
                                        float* partial_out, float* partial_ml, int* error_flag, cudaStream_t stream) {
     if (!llm_attention_mma_sinks_supports(head_dim, value_dim, n_q_heads, n_kv_heads)) {
         llm_set_error("attention_mma_sinks: keys of %d and values of %d with %d/%d heads are not supported (64 or 128 each, "
@@ -1326,10 +1389,22 @@ LLM_EXPORT int llm_attention_mma_sinks(const void* q, int q_stride, const void* 
     p.partial_ml = partial_ml;
     p.error_flag = error_flag;
     p.sinks = sinks;
-    if (head_dim == 64) {
-        return value_dim == 64 ? launch_precise<64, 64>(p, run_portions, total_tiles, run_decode, stream)
-                               : launch_precise<64, 128>(p, run_portions, total_tiles, run_decode, stream);
+    if (chunk < 0 || (bias && bias_len <= 0)) {
+        llm_set_error("attention_mma_sinks: a chunk of %d positions or a bias of %d distances", chunk, bias_len);
+        return LLM_REFUSED;
     }
-    return value_dim == 64 ? launch_precise<128, 64>(p, run_portions, total_tiles, run_decode, stream)
-                           : launch_precise<128, 128>(p, run_portions, total_tiles, run_decode, stream);
+    p.chunk = chunk;
+    p.bias = bias;
+    p.bias_len = bias_len;
+#define LLM_PRECISE(BIAS)                                                                                                  \
+    do {                                                                                                                   \
+        if (head_dim == 64)                                                                                                \
+            return value_dim == 64 ? launch_precise<64, 64, BIAS>(p, run_portions, total_tiles, run_decode, stream)        \
+                                   : launch_precise<64, 128, BIAS>(p, run_portions, total_tiles, run_decode, stream);      \
+        return value_dim == 64 ? launch_precise<128, 64, BIAS>(p, run_portions, total_tiles, run_decode, stream)           \
+                               : launch_precise<128, 128, BIAS>(p, run_portions, total_tiles, run_decode, stream);         \
+    } while (0)
+    if (bias) LLM_PRECISE(true);
+    LLM_PRECISE(false);
+#undef LLM_PRECISE
 }

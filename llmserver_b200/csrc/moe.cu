@@ -3,7 +3,11 @@
 //   route      z = W_r x (32-bit), s = sigmoid(z); the `top` experts with the largest s + correction are chosen
 //              (ties: the lower index), each with the weight s * scale (the correction only chooses; nothing is
 //              renormalised).  One block per token.  `select` is the same choice from logits that a matrix product
-//              has already made (one warp per token).
+//              has already made (one warp per token).  Options of the choice (RouteRule): s = softmax(z) over all
+//              experts; the weights divided by their sum (+ 1e-20); only the `keep` best of `groups` equal groups of
+//              neighbouring experts can be chosen, a group's score being the largest in it.  A router may have one
+//              more row behind its experts': the pre-activation of a gate on the shared expert, whose sigmoid is
+//              left in `gate_out`.
 //   indexed    out[p] = W[index[p]] in[p / in_div]: every (token, chosen expert) pair p multiplies its own expert's
 //   linear     matrix.  One warp per output element, its sum taken over k in an order that depends on the inner size
 //              alone, so a pair's result does not depend on what else the step holds.  As a gated form the matrix
@@ -13,39 +17,66 @@
 //              With `in_scale` pair p's input row is multiplied by in_scale[p] as it is read (32-bit): a routing
 //              weight that acts on what goes into an expert.  Read-once for steps of few tokens; prompts take the tiled
 //              kernels of moe_grouped.cu.
-//   combine    out[t] = sum_j weight[t, j] * down[t * top + j] (+ shared[t]) in 32-bit, slots in order.
+//   combine    out[t] = sum_j weight[t, j] * down[t * top + j] (+ gate[t] * shared[t]) in 32-bit, slots in order.
 #include "common.cuh"
 
 #define MOE_MAX_TOP 32
 
-template <typename T>
-__global__ void moe_route_kernel(const T* __restrict__ x, const float* __restrict__ router, const float* __restrict__ correction,
-                                 int* __restrict__ chosen, float* __restrict__ weights, int* __restrict__ counts,
-                                 int width, int experts, int top, float scale) {
-    pdl_trigger();
-    pdl_wait();
-    extern __shared__ float route_shared[];      // [width] the token's row, [experts] scores, [experts] choice scores
-    float* row = route_shared;
-    float* score = route_shared + width;
-    float* choice = score + experts;
-    const int token = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
-    const T* src = x + (size_t)token * width;
-    for (int i = threadIdx.x; i < width; i += blockDim.x) row[i] = Num<T>::load(src + i);
-    __syncthreads();
-    for (int e = warp; e < experts; e += warps) {
-        const float* w = router + (size_t)e * width;
+struct RouteRule {
+    int experts, top;
+    int softmax;          // scores: 0 sigmoid, 1 softmax over all experts
+    int groups, keep;     // groups > 0: only experts of the `keep` best groups can be chosen
+    int renormalise;      // the chosen weights are divided by their sum
+    float scale;
+};
+
+// The choice by one warp.  On entry `score` holds the router's logits z (32-bit); `choice` is scratch of the same size.
+__device__ __forceinline__ void choose_experts(float* score, float* choice, const RouteRule& rule, const float* __restrict__ correction,
+                                               int* __restrict__ chosen, float* __restrict__ weights, int* __restrict__ counts) {
+    const int lane = threadIdx.x & 31, experts = rule.experts;
+    if (rule.softmax) {
+        float best = -INFINITY;
+        for (int e = lane; e < experts; e += 32) best = fmaxf(best, score[e]);
+        best = warp_max(best);
         float sum = 0.0f;
-        for (int i = lane; i < width; i += 32) sum = fmaf(row[i], w[i], sum);
-        sum = warp_sum(sum);
-        if (lane == 0) {
-            const float s = 1.0f / (1.0f + expf(-sum));
+        for (int e = lane; e < experts; e += 32) {
+            const float s = expf(score[e] - best);
             score[e] = s;
-            choice[e] = s + (correction ? correction[e] : 0.0f);
+            sum += s;
         }
+        sum = warp_sum(sum);
+        for (int e = lane; e < experts; e += 32) score[e] /= sum;
+    } else {
+        for (int e = lane; e < experts; e += 32) score[e] = 1.0f / (1.0f + expf(-score[e]));
     }
-    __syncthreads();
-    if (warp != 0) return;
-    for (int j = 0; j < top; ++j) {
+    __syncwarp();
+    for (int e = lane; e < experts; e += 32) choice[e] = score[e] + (correction ? correction[e] : 0.0f);
+    __syncwarp();
+    if (rule.groups > 0) {
+        // a lane looks after whole groups: it ranks each of them among all (ties: the lower index) and, when `keep` groups
+        // are better, takes its experts out of the choice; every rank is formed before anything is taken out
+        const int size = experts / rule.groups;
+        for (int first = 0; first < rule.groups; first += 32) {
+            const int g = first + lane;
+            bool out = false;
+            if (g < rule.groups) {
+                float own = -INFINITY;
+                for (int e = 0; e < size; ++e) own = fmaxf(own, choice[g * size + e]);
+                int better = 0;
+                for (int other = 0; other < rule.groups; ++other) {
+                    float theirs = -INFINITY;
+                    for (int e = 0; e < size; ++e) theirs = fmaxf(theirs, score[other * size + e] + (correction ? correction[other * size + e] : 0.0f));
+                    better += theirs > own || (theirs == own && other < g);
+                }
+                out = better >= rule.keep;
+            }
+            if (out)
+                for (int e = 0; e < size; ++e) choice[g * size + e] = -INFINITY;
+        }
+        __syncwarp();
+    }
+    float total = 0.0f;
+    for (int j = 0; j < rule.top; ++j) {
         float best = -INFINITY;
         int best_index = 0x7fffffff;
         for (int e = lane; e < experts; e += 32) {
@@ -65,60 +96,68 @@ __global__ void moe_route_kernel(const T* __restrict__ x, const float* __restric
             }
         }
         if (best_index == 0x7fffffff) best_index = 0;      // every score was NaN or -inf: never expected
+        const float s = score[best_index];
+        total += s;
         if (lane == 0) {
-            chosen[(size_t)token * top + j] = best_index;
-            weights[(size_t)token * top + j] = score[best_index] * scale;
+            chosen[j] = best_index;
+            if (!rule.renormalise) weights[j] = s * rule.scale;
             if (counts) atomicAdd(counts + best_index, 1);
             choice[best_index] = -INFINITY;
         }
         __syncwarp();
     }
+    if (rule.renormalise) {      // lane j looks after choice j
+        const float factor = rule.scale / (total + 1e-20f);
+        for (int j = lane; j < rule.top; j += 32) weights[j] = score[chosen[j]] * factor;
+    }
 }
 
-// The choice alone, from router logits that a matrix product has made: z float32 [N, experts].  One warp per token.
+template <typename T>
+__global__ void moe_route_kernel(const T* __restrict__ x, const float* __restrict__ router, const float* __restrict__ correction,
+                                 int* __restrict__ chosen, float* __restrict__ weights, int* __restrict__ counts,
+                                 int width, RouteRule rule, float* __restrict__ gate_out) {
+    pdl_trigger();
+    pdl_wait();
+    extern __shared__ float route_shared[];      // [width] the token's row, [experts] scores, [experts] choice scores
+    float* row = route_shared;
+    float* score = route_shared + width;
+    float* choice = score + rule.experts;
+    const int token = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+    const T* src = x + (size_t)token * width;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) row[i] = Num<T>::load(src + i);
+    __syncthreads();
+    const int rows = rule.experts + (gate_out ? 1 : 0);
+    for (int e = warp; e < rows; e += warps) {
+        const float* w = router + (size_t)e * width;
+        float sum = 0.0f;
+        for (int i = lane; i < width; i += 32) sum = fmaf(row[i], w[i], sum);
+        sum = warp_sum(sum);
+        if (lane == 0) {
+            if (e < rule.experts) score[e] = sum;
+            else gate_out[token] = 1.0f / (1.0f + expf(-sum));
+        }
+    }
+    __syncthreads();
+    if (warp != 0) return;
+    choose_experts(score, choice, rule, correction, chosen + (size_t)token * rule.top, weights + (size_t)token * rule.top, counts);
+}
+
+// The choice alone, from router logits that a matrix product has made: z float32 [N, experts (+ 1 for the gate)].  One
+// warp per token.
 __global__ void moe_select_kernel(const float* __restrict__ logits, const float* __restrict__ correction, int* __restrict__ chosen,
-                                  float* __restrict__ weights, int n_tokens, int experts, int top, float scale) {
+                                  float* __restrict__ weights, int n_tokens, RouteRule rule, float* __restrict__ gate_out) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float select_shared[];      // per warp: [experts] scores, [experts] choice scores
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
     const int token = blockIdx.x * warps + warp;
     if (token >= n_tokens) return;
-    float* score = select_shared + (size_t)warp * 2 * experts;
-    float* choice = score + experts;
-    for (int e = lane; e < experts; e += 32) {
-        const float s = 1.0f / (1.0f + expf(-logits[(size_t)token * experts + e]));
-        score[e] = s;
-        choice[e] = s + (correction ? correction[e] : 0.0f);
-    }
+    float* score = select_shared + (size_t)warp * 2 * rule.experts;
+    const float* z = logits + (size_t)token * (rule.experts + (gate_out ? 1 : 0));
+    for (int e = lane; e < rule.experts; e += 32) score[e] = z[e];
+    if (gate_out && lane == 0) gate_out[token] = 1.0f / (1.0f + expf(-z[rule.experts]));
     __syncwarp();
-    for (int j = 0; j < top; ++j) {
-        float best = -INFINITY;
-        int best_index = 0x7fffffff;
-        for (int e = lane; e < experts; e += 32) {
-            const float c = choice[e];
-            if (c > best) {
-                best = c;
-                best_index = e;
-            }
-        }
-#pragma unroll
-        for (int offset = 16; offset > 0; offset >>= 1) {
-            const float other = __shfl_xor_sync(0xffffffffu, best, offset);
-            const int other_index = __shfl_xor_sync(0xffffffffu, best_index, offset);
-            if (other > best || (other == best && other_index < best_index)) {
-                best = other;
-                best_index = other_index;
-            }
-        }
-        if (best_index == 0x7fffffff) best_index = 0;
-        if (lane == 0) {
-            chosen[(size_t)token * top + j] = best_index;
-            weights[(size_t)token * top + j] = score[best_index] * scale;
-            choice[best_index] = -INFINITY;
-        }
-        __syncwarp();
-    }
+    choose_experts(score, score + rule.experts, rule, correction, chosen + (size_t)token * rule.top, weights + (size_t)token * rule.top, nullptr);
 }
 
 __device__ __forceinline__ float gated_activation(float gate, float up, float limit, float alpha, float up_shift = 1.0f) {
@@ -190,7 +229,7 @@ __global__ void indexed_linear_kernel(const T* __restrict__ in, const T* __restr
 
 template <typename T>
 __global__ void moe_combine_kernel(const float* __restrict__ down, const float* __restrict__ weights, const T* __restrict__ shared_out,
-                                   T* __restrict__ out, int width, int top, size_t total) {
+                                   const float* __restrict__ shared_gate, T* __restrict__ out, int width, int top, size_t total) {
     pdl_trigger();
     pdl_wait();
     for (size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x; e < total; e += (size_t)gridDim.x * blockDim.x) {
@@ -199,7 +238,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ down, const float* 
         float sum = 0.0f;
         for (int j = 0; j < top; ++j)
             sum = fmaf(weights[token * top + j], down[(token * top + j) * width + column], sum);
-        if (shared_out) sum += Num<T>::load(shared_out + e);
+        if (shared_out) sum = fmaf(shared_gate ? shared_gate[token] : 1.0f, Num<T>::load(shared_out + e), sum);
         Num<T>::store(out + e, sum);
     }
 }
@@ -247,14 +286,25 @@ __global__ void clamped_glu_vec_kernel(const T* __restrict__ gate_up, T* __restr
     }
 }
 
-LLM_EXPORT int llm_moe_route(const void* x, const float* router, const float* correction, int* chosen, float* weights,
-                             int* counts, int n_tokens, int width, int experts, int top, float scale, int dtype,
-                             cudaStream_t stream) {
-    if (n_tokens == 0) return LLM_OK;
-    if (top <= 0 || top > experts || top > MOE_MAX_TOP) {
-        llm_set_error("moe_route: top %d must lie in 1..min(%d experts, %d)", top, experts, MOE_MAX_TOP);
+static int check_rule(const char* what, const RouteRule& rule) {
+    if (rule.top <= 0 || rule.top > rule.experts || rule.top > MOE_MAX_TOP) {
+        llm_set_error("%s: top %d must lie in 1..min(%d experts, %d)", what, rule.top, rule.experts, MOE_MAX_TOP);
         return LLM_REFUSED;
     }
+    if (rule.groups < 0 || (rule.groups > 0 && (rule.experts % rule.groups || rule.keep <= 0 || rule.keep > rule.groups ||
+                                                rule.top > rule.keep * (rule.experts / rule.groups)))) {
+        llm_set_error("%s: %d experts in %d groups of which %d are kept cannot give %d choices", what, rule.experts, rule.groups, rule.keep, rule.top);
+        return LLM_REFUSED;
+    }
+    return LLM_OK;
+}
+
+LLM_EXPORT int llm_moe_route(const void* x, const float* router, const float* correction, int* chosen, float* weights,
+                             int* counts, int n_tokens, int width, int experts, int top, float scale, int softmax, int groups, int keep,
+                             int renormalise, float* gate_out, int dtype, cudaStream_t stream) {
+    if (n_tokens == 0) return LLM_OK;
+    const RouteRule rule = {experts, top, softmax, groups, keep, renormalise, scale};
+    if (const int refused = check_rule("moe_route", rule)) return refused;
     const size_t shared = ((size_t)width + 2 * (size_t)experts) * sizeof(float);
     if (shared > 200 * 1024) {
         llm_set_error("moe_route: width %d and %d experts need %zu bytes of shared memory", width, experts, shared);
@@ -266,18 +316,17 @@ LLM_EXPORT int llm_moe_route(const void* x, const float* router, const float* co
             if (status != LLM_OK) return status;
         }
         llm_launch(moe_route_kernel<T>, n_tokens, 256, shared, stream, (const T*)x, router, correction, chosen, weights,
-                   counts, width, experts, top, scale);
+                   counts, width, rule, gate_out);
     });
     return llm_check_launch("moe_route");
 }
 
 LLM_EXPORT int llm_moe_select(const float* logits, const float* correction, int* chosen, float* weights, int n_tokens,
-                              int experts, int top, float scale, cudaStream_t stream) {
+                              int experts, int top, float scale, int softmax, int groups, int keep, int renormalise, float* gate_out,
+                              cudaStream_t stream) {
     if (n_tokens == 0) return LLM_OK;
-    if (top <= 0 || top > experts || top > MOE_MAX_TOP) {
-        llm_set_error("moe_select: top %d must lie in 1..min(%d experts, %d)", top, experts, MOE_MAX_TOP);
-        return LLM_REFUSED;
-    }
+    const RouteRule rule = {experts, top, softmax, groups, keep, renormalise, scale};
+    if (const int refused = check_rule("moe_select", rule)) return refused;
     const int warps = 4;
     const size_t shared = (size_t)warps * 2 * experts * sizeof(float);
     if (shared > 40 * 1024) {
@@ -285,7 +334,7 @@ LLM_EXPORT int llm_moe_select(const float* logits, const float* correction, int*
         return LLM_REFUSED;
     }
     llm_launch(moe_select_kernel, (n_tokens + warps - 1) / warps, warps * 32, shared, stream, logits, correction, chosen, weights,
-               n_tokens, experts, top, scale);
+               n_tokens, rule, gate_out);
     return llm_check_launch("moe_select");
 }
 
@@ -330,14 +379,14 @@ LLM_EXPORT int llm_indexed_linear(const void* in, const void* weight, const int*
     return llm_check_launch("indexed_linear");
 }
 
-LLM_EXPORT int llm_moe_combine(const float* down, const float* weights, const void* shared_out, void* out, int n_tokens,
+LLM_EXPORT int llm_moe_combine(const float* down, const float* weights, const void* shared_out, const float* shared_gate, void* out, int n_tokens,
                                int width, int top, int dtype, cudaStream_t stream) {
     if (n_tokens == 0) return LLM_OK;
     const size_t total = (size_t)n_tokens * width;
     size_t blocks = (total + 255) / 256;
     if (blocks > 148 * 16) blocks = 148 * 16;
     LLM_DISPATCH_DTYPE(dtype, (llm_launch(moe_combine_kernel<T>, (unsigned)blocks, 256, 0, stream, down, weights,
-                                  (const T*)shared_out, (T*)out, width, top, total)));
+                                  (const T*)shared_out, shared_gate, (T*)out, width, top, total)));
     return llm_check_launch("moe_combine");
 }
 

@@ -228,14 +228,15 @@ __global__ void __launch_bounds__(kGemmThreads) moe_grouped_kernel(const __nv_bf
     }
 }
 
-// out[t] = sum_j weight[t, j] * down[row_of_pair[t * top + j]] (+ shared[t]), 32-bit, slots in order.
+// out[t] = sum_j weight[t, j] * down[row_of_pair[t * top + j]] (+ gate[t] * shared[t]), 32-bit, slots in order.
 template <typename T>
 __global__ void moe_combine_rows_kernel(const float* __restrict__ down, const int* __restrict__ row_of_pair,
-                                        const float* __restrict__ weights, const T* __restrict__ shared_out, T* __restrict__ out,
-                                        int width, int top) {
+                                        const float* __restrict__ weights, const T* __restrict__ shared_out,
+                                        const float* __restrict__ shared_gate, T* __restrict__ out, int width, int top) {
     pdl_trigger();
     pdl_wait();
     const size_t token = blockIdx.x;
+    const float gate = shared_gate ? shared_gate[token] : 1.0f;
     for (int column = threadIdx.x * 4; column < width; column += blockDim.x * 4) {
         float sum[4] = {0.0f, 0.0f, 0.0f, 0.0f};
         for (int j = 0; j < top; ++j) {
@@ -248,7 +249,7 @@ __global__ void moe_combine_rows_kernel(const float* __restrict__ down, const in
         }
 #pragma unroll
         for (int v = 0; v < 4; ++v) {
-            if (shared_out) sum[v] += Num<T>::load(shared_out + token * width + column + v);
+            if (shared_out) sum[v] = fmaf(gate, Num<T>::load(shared_out + token * width + column + v), sum[v]);
             Num<T>::store(out + token * width + column + v, sum[v]);
         }
     }
@@ -308,13 +309,13 @@ LLM_EXPORT int llm_moe_grouped(const void* a, const void* w, const int* tiles, c
 }
 
 LLM_EXPORT int llm_moe_combine_rows(const float* down, const int* row_of_pair, const float* weights, const void* shared_out,
-                                    void* out, int n_tokens, int width, int top, int dtype, cudaStream_t stream) {
+                                    const float* shared_gate, void* out, int n_tokens, int width, int top, int dtype, cudaStream_t stream) {
     if (n_tokens == 0) return LLM_OK;
     if (width % 4) {
         llm_set_error("moe_combine_rows: the width %d is no multiple of 4", width);
         return LLM_REFUSED;
     }
     LLM_DISPATCH_DTYPE(dtype, (llm_launch(moe_combine_rows_kernel<T>, n_tokens, 256, 0, stream, down, row_of_pair, weights,
-                                  (const T*)shared_out, (T*)out, width, top)));
+                                  (const T*)shared_out, shared_gate, (T*)out, width, top)));
     return llm_check_launch("moe_combine_rows");
 }

@@ -455,3 +455,84 @@ LLM_EXPORT int llm_scaled_add_rmsnorm(float* residual, const void* a, const floa
     });
     return llm_check_launch("scaled_add_rmsnorm");
 }
+
+// RMS norm of 32-bit rows in `parts` equal pieces, each by its own root mean square:
+//   out[r][c] = x[r][c] * rsqrt(mean over c's piece of x[r]^2 + eps) * weight[c]
+// One warp per (row, piece); the order of the sum depends on the piece's size only.
+template <typename T, typename W, bool VEC>
+__global__ void grouped_rmsnorm_kernel(const float* __restrict__ x, const W* __restrict__ weight, T* __restrict__ out, int n_rows,
+                                       int parts, int size, float eps) {
+    pdl_trigger();
+    pdl_wait();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+    const long long item = (long long)blockIdx.x * warps + warp;
+    if (item >= (long long)n_rows * parts) return;
+    const int part = (int)(item % parts);
+    const float* src = x + item * size;
+    const W* w = weight + (size_t)part * size;
+    T* dst = out + item * size;
+    float squares = 0.0f;
+    if (VEC) {
+        for (int c = lane * 8; c < size; c += 256) {
+            float v[8];
+            load8<float>(src + c, v);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) squares = fmaf(v[j], v[j], squares);
+        }
+    } else {
+        for (int c = lane; c < size; c += 32) squares = fmaf(src[c], src[c], squares);
+    }
+    const float inverse = rsqrtf(warp_sum(squares) / (float)size + eps);
+    if (VEC) {
+        for (int c = lane * 8; c < size; c += 256) {
+            float v[8], scale[8];
+            load8<float>(src + c, v);
+            load8<W>(w + c, scale);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[j] = v[j] * inverse * scale[j];
+            store8<T>(dst + c, v);
+        }
+    } else {
+        for (int c = lane; c < size; c += 32) Num<T>::store(dst + c, src[c] * inverse * Num<W>::load(w + c));
+    }
+}
+
+// The same with one block per (row, piece), for steps with fewer pieces than fill the GPU with single warps and for long
+// pieces; a piece's elements stay in the L1 between the two passes.
+template <typename T, typename W>
+__global__ void grouped_rmsnorm_block_kernel(const float* __restrict__ x, const W* __restrict__ weight, T* __restrict__ out, int parts,
+                                             int size, float eps) {
+    pdl_trigger();
+    pdl_wait();
+    __shared__ float scratch[33];
+    const int part = blockIdx.x % parts;
+    const float* src = x + (size_t)blockIdx.x * size;
+    const W* w = weight + (size_t)part * size;
+    T* dst = out + (size_t)blockIdx.x * size;
+    float squares = 0.0f;
+    for (int c = threadIdx.x; c < size; c += blockDim.x) squares = fmaf(src[c], src[c], squares);
+    const float inverse = rsqrtf(block_sum(squares, scratch) / (float)size + eps);
+    for (int c = threadIdx.x; c < size; c += blockDim.x) Num<T>::store(dst + c, src[c] * inverse * Num<W>::load(w + c));
+}
+
+LLM_EXPORT int llm_grouped_rmsnorm(const float* x, const void* weight, void* out, int n_rows, int parts, int size, float eps, int dtype,
+                                   int weight_dtype, cudaStream_t stream) {
+    if (n_rows == 0) return LLM_OK;
+    if (parts <= 0 || size <= 0) {
+        llm_set_error("grouped_rmsnorm: %d pieces of %d elements must both be positive", parts, size);
+        return LLM_REFUSED;
+    }
+    if (size > 1024) {      // the choice depends on the piece's size only, so a row's result does not depend on the batch
+        LLM_DISPATCH_DTYPE_WEIGHT(dtype, weight_dtype, (llm_launch(grouped_rmsnorm_block_kernel<T, W>, (unsigned)n_rows * parts, 256, 0, stream,
+                                                                   x, (const W*)weight, (T*)out, parts, size, eps)));
+        return llm_check_launch("grouped_rmsnorm");
+    }
+    const int warps = 8;
+    const unsigned blocks = (unsigned)(((long long)n_rows * parts + warps - 1) / warps);
+    const bool vec = size % 8 == 0 && aligned16(x) && aligned16(weight) && aligned16(out);
+    LLM_DISPATCH_DTYPE_WEIGHT(dtype, weight_dtype, {
+        if (vec) llm_launch(grouped_rmsnorm_kernel<T, W, true>, blocks, warps * 32, 0, stream, x, (const W*)weight, (T*)out, n_rows, parts, size, eps);
+        else llm_launch(grouped_rmsnorm_kernel<T, W, false>, blocks, warps * 32, 0, stream, x, (const W*)weight, (T*)out, n_rows, parts, size, eps);
+    });
+    return llm_check_launch("grouped_rmsnorm");
+}

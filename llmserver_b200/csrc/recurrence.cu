@@ -5,7 +5,7 @@
 //     token of a step, zeros for the first token of a sequence), out[s] = h + (h' - h) * mu[s] for each of M mixing
 //     vectors.  The stored row is replaced by the kernel of (3), behind every read of it.
 //
-// (2) Short convolution (`llm_short_conv_units`): y_t[c] = silu(sum_j w[c][j] * x_(t - taps + 1 + j)[c]), zeros before the
+// (2) Short convolution (`llm_short_conv_units`): y_t[c] = silu(sum_j w[c][j] * x_(t - taps + 1 + j)[c] + bias[c]), zeros before the
 //     sequence's start, the last taps - 1 inputs of every sequence carried in its state slot; channels come in units (a
 //     head's query, key or value channels); the first `n_unit_norm` units are then made unit vectors,
 //     y / sqrt(sum(y^2) + norm_eps), and the first `n_scaled` of those multiplied by `scale`.  Results are 32-bit.  A block
@@ -17,6 +17,12 @@
 //       delta   S <- g_t S;  d = beta_t (v_t - S^T k_t);  S <- S + k_t d^T;  o_t = S^T q_t
 //               g_t = exp(-exp(A) softplus(a_t + dt)),  beta_t = sigmoid(b_t)
 //     followed by out = o / sqrt(mean(o^2) + eps) * weight * silu(gate).
+//     Two more share one plain form, a single decay per head and token (`llm_retention_recurrent`, `llm_ssd_recurrent`):
+//       S <- g_t S + k_t v_t^T;  o_t = S_t^T q_t
+//       retention   g a constant of the head, q and k rotated by the token's position, k scaled, as they are staged;
+//                   followed by out = o / sqrt(mean(o^2) + eps) * silu(gate)
+//       ssd         (Dao and Gu, "Transformers are SSMs") g_t = exp(-exp(A) dt_t), dt_t = softplus(z_t + bias), q = C_t and
+//                   k = dt_t B_t shared by a group of heads, v = x_t; followed by out = (o + D x) * silu(gate), in 32-bit
 //
 // One block per (sequence, head).  A warp covers 32 / P value channels (columns of S) with P row partitions side by
 // side in its lanes; a thread owns R rows of one column in registers, so a sum over the rows is R multiply-adds and
@@ -25,9 +31,9 @@
 // and stored by one warp per token.  The order of every sum depends on the sizes alone, so a token's result does not
 // depend on how its prompt was cut or on what else is in the batch.
 //
-// Long portions can also be walked segment by segment in parallel (a segment length given to the launchers).  Both
+// Long portions can also be walked segment by segment in parallel (a segment length given to the launchers).  All the
 // recurrences are linear in S: behind a segment, S_out = M S_in + L, where L is what the segment leaves from a zero state
-// and M its transition: diag(prod_t w_t) for wkv; for the delta rule the product of the g_t (I - beta_t k_t k_t^T), a
+// and M its transition: diag(prod_t w_t) for wkv; prod_t g_t for the two with one decay per head; for the delta rule the product of the g_t (I - beta_t k_t k_t^T), a
 // dim x dim matrix, which the same walk yields column by column when it starts from the identity with values of zero.
 // Pass A runs every segment but the last from zero (delta: also `dim` more columns from the identity) and leaves L and M;
 // a scan gives every segment the state it starts from, S_in(k + 1) = M_k S_in(k) + L_k; pass C runs the segments again
@@ -78,12 +84,13 @@ struct ConvArgs {
     float* out;             // [N, channels]
     int channels;
     int n_unit_norm, unit_dim, n_scaled;   // units 0 .. n_unit_norm - 1 have unit_dim channels and are made unit vectors
-    int n_plain, plain_dim;                // the units behind them
+    int n_plain, plain_dim;                // the units behind them (the last may be cut short by `channels`)
     float norm_eps, scale;
+    const float* bias;                     // [channels] or null
 };
 
 #define CONV_MAX_PER_LANE 16    // a unit has at most 32 * 16 channels
-#define CONV_MAX_TAPS 8
+#define CONV_MAX_TAPS 64
 #define CONV_CHUNK 64           // tokens per block; more than CONV_MAX_TAPS - 1, so only a sequence's first block reads stored inputs
 
 template <typename T>
@@ -95,8 +102,8 @@ __global__ void __launch_bounds__(256) short_conv_units_kernel(ConvArgs a) {
     const int chunk_begin = begin + blockIdx.z * CONV_CHUNK, chunk_end = min(end, chunk_begin + CONV_CHUNK);
     if (chunk_begin >= end) return;
     const bool normed = unit < a.n_unit_norm;
-    const int size = normed ? a.unit_dim : a.plain_dim;
     const int first = normed ? unit * a.unit_dim : a.n_unit_norm * a.unit_dim + (unit - a.n_unit_norm) * a.plain_dim;
+    const int size = normed ? a.unit_dim : min(a.plain_dim, a.channels - first);
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
     const int history = a.taps - 1;
     const T* x = (const T*)a.x + a.column + first;
@@ -109,7 +116,7 @@ __global__ void __launch_bounds__(256) short_conv_units_kernel(ConvArgs a) {
             const int c = lane + 32 * u;
             y[u] = 0.0f;
             if (c < size) {
-                float sum = 0.0f;
+                float sum = a.bias ? a.bias[first + c] : 0.0f;
                 for (int j = 0; j < a.taps; ++j) {
                     const int source = t - history + j;      // on the step's token axis; before `begin`: the stored inputs
                     const float value = source >= begin ? Num<T>::load(x + (size_t)source * a.row_width + c)
@@ -147,9 +154,16 @@ __global__ void __launch_bounds__(256) short_conv_units_kernel(ConvArgs a) {
 
 LLM_EXPORT int llm_short_conv_units(const void* x, int row_width, int column, const float* taps_w, int taps, float* state,
                                     const int* state_slots, const int* q_start, float* out, int n_seqs, int longest, int n_unit_norm,
-                                    int unit_dim, int n_scaled, int n_plain, int plain_dim, float norm_eps, float scale, int dtype,
-                                    cudaStream_t stream) {
+                                    int unit_dim, int n_scaled, int n_plain, int plain_dim, float norm_eps, float scale,
+                                    const float* bias, int channels, int dtype, cudaStream_t stream) {
     if (n_seqs == 0 || longest <= 0) return LLM_OK;
+    // the plain units cover the channels behind the normalised ones, only the last of them cut short
+    const int plain = channels - n_unit_norm * unit_dim;
+    if (plain < 0 || plain > n_plain * plain_dim || (n_plain > 0 && plain <= (n_plain - 1) * plain_dim)) {
+        llm_set_error("short_conv_units: %d channels are not %d units of %d and %d units of up to %d", channels, n_unit_norm, unit_dim,
+                      n_plain, plain_dim);
+        return LLM_REFUSED;
+    }
     if (taps < 1 || taps > CONV_MAX_TAPS || unit_dim > 32 * CONV_MAX_PER_LANE || plain_dim > 32 * CONV_MAX_PER_LANE ||
         n_unit_norm < 0 || n_plain < 0 || n_unit_norm + n_plain == 0) {
         llm_set_error("short_conv_units: %d taps (1 to %d) over units of %d and %d channels (up to %d) are not supported", taps,
@@ -159,7 +173,7 @@ LLM_EXPORT int llm_short_conv_units(const void* x, int row_width, int column, co
     ConvArgs a;
     a.x = x; a.row_width = row_width; a.column = column; a.taps_w = taps_w; a.taps = taps; a.state = state;
     a.state_slots = state_slots; a.q_start = q_start; a.out = out;
-    a.channels = n_unit_norm * unit_dim + n_plain * plain_dim;
+    a.channels = channels; a.bias = bias;
     a.n_unit_norm = n_unit_norm; a.unit_dim = unit_dim; a.n_scaled = n_scaled; a.n_plain = n_plain; a.plain_dim = plain_dim;
     a.norm_eps = norm_eps; a.scale = scale;
     LLM_DISPATCH_DTYPE(dtype, (llm_launch(short_conv_units_kernel<T>, dim3(n_seqs, n_unit_norm + n_plain, (longest + CONV_CHUNK - 1) / CONV_CHUNK), 256, 0, stream, a)));
@@ -174,17 +188,23 @@ struct RecArgs {
     // inputs in 32-bit
     const float* pre;       // delta: [N, pre_width] convolved q | k | v (q and k heads of `dim`, v heads of `vdim`)
     int pre_width, q_col, k_col, v_col, qk_heads;
-    const float* wide;      // wkv: z [N, heads * dim]; delta: [N, 2 heads] = b | a
+    const float* wide;      // wkv: z [N, heads * dim]; delta: [N, 2 heads] = b | a; ssd: [N, heads], dt before its bias
     const float* w0;        // wkv: [heads * dim]
     const float* bonus;     // wkv: u [heads, dim]
-    const float* a_log;     // delta: [heads]
-    const float* dt_bias;   // delta: [heads]
+    const float* a_log;     // delta, ssd: [heads]
+    const float* dt_bias;   // delta, ssd: [heads]
+    const float* head_decay;    // retention: [heads]
+    const float* skip;          // ssd: D [heads]
+    const int* positions;       // retention: [N]
+    const float* inv_freq;      // retention: [rotary_dim / 2]; null: nothing rotates
+    int rotary_dim;
+    float k_scale;              // retention: what a key is multiplied by behind its rotation
     const void* weight;     // norm weight, [vdim] (weight_stride 0) or [heads, vdim] (weight_stride vdim)
     int weight_stride;
     float* state;           // [slots, heads, dim, vdim]
     const int* state_slots;
     const int* q_start;
-    void* out;              // [N, heads * vdim]
+    void* out;              // [N, heads * vdim] in the activation type; ssd: float32
     int heads, dim, vdim, partitions, stride_rows;     // stride_rows: floats from one partition's staged rows to the next's
     float eps;
     // wkv: the row that the next step's token shift reads
@@ -195,15 +215,16 @@ struct RecArgs {
     int segment, max_segments;  // tokens per segment, segments the scratch has room for per sequence
     int groups;                 // delta, pass A: blocks per (segment, head): one for the value columns + those for the transition's
     float* segment_state;       // [S, max_segments, heads, dim, vdim]: pass A leaves L there, the scan S_in
-    float* segment_move;        // wkv: [S, max_segments, heads, dim], the products of the decays; delta: [.., heads, dim, dim]
+    float* segment_move;        // [S, max_segments, heads, dim], the products of the decays; delta: [.., heads, dim, dim]
 };
 
-enum : int { REC_WKV = 0, REC_DELTA = 1 };
+enum : int { REC_WKV = 0, REC_DELTA = 1, REC_RETENTION = 2, REC_SSD = 3 };
 // PASS 0: a sequence's tokens in one pass, from and into its state slot.  1: pass A of the segmented form.  3: pass C.
 enum : int { REC_ONE_PASS = 0, REC_LOCAL = 1, REC_OUTPUT = 3 };
 
 template <typename T, typename W, int R, int MODE, int PASS>
 __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) matrix_recurrence_kernel(RecArgs a) {
+    constexpr bool PLAIN = MODE == REC_RETENTION || MODE == REC_SSD;      // one decay per head and token
     pdl_trigger();
     pdl_wait();
     extern __shared__ float4 rec_shared_raw[];
@@ -233,7 +254,7 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) matrix_recurrence_kernel(
     float* w_s = k_s + REC_TOKENS * padded;            // wkv only: the decays
     float* v_s = w_s + (MODE == REC_WKV ? REC_TOKENS * padded : 0);     // [REC_TOKENS][vdim]
     float* o_s = v_s + REC_TOKENS * vdim;              // [REC_TOKENS][vdim]
-    float* scalar_s = o_s + REC_TOKENS * vdim;         // [REC_TOKENS][2]: wkv: the bonus term; delta: g and beta
+    float* scalar_s = o_s + REC_TOKENS * vdim;         // [REC_TOKENS][2]: wkv: the bonus term; delta: g and beta; else: g
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
     const int per_warp = 32 / P;                       // columns of S per warp
     const int part = lane / per_warp, column = warp * per_warp + lane % per_warp;
@@ -254,8 +275,9 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) matrix_recurrence_kernel(
         else S[i] = (owner && row0 + i < dim) ? source[(size_t)(row0 + i) * vdim + column] : 0.0f;
         if (PASS == REC_LOCAL && MODE == REC_WKV) decay[i] = 1.0f;
     }
+    float move = 1.0f;      // pass A with one decay per head: the product of the segment's decays
 
-    const int qk_head = MODE == REC_DELTA ? head / (a.heads / a.qk_heads) : head;
+    const int qk_head = MODE == REC_DELTA || MODE == REC_SSD ? head / (a.heads / a.qk_heads) : head;
     for (int first = begin; first < end; first += REC_TOKENS) {
         const int count = min(REC_TOKENS, end - first);
         __syncthreads();      // the staged values of the tokens before have been read
@@ -263,7 +285,40 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) matrix_recurrence_kernel(
         for (int t = warp; t < count; t += warps) {
             const size_t token = (size_t)(first + t);
             float bonus = 0.0f;
-            for (int i = lane; i < P * R; i += 32) {
+            float dt = 0.0f;
+            if (MODE == REC_SSD) {
+                const float z = a.wide[token * a.heads + head] + a.dt_bias[head];
+                dt = z > 20.0f ? z : log1pf(expf(z));
+                if (lane == 0) scalar_s[2 * t] = expf(-expf(a.a_log[head]) * dt);
+            }
+            if (MODE == REC_RETENTION) {
+                if (lane == 0) scalar_s[2 * t] = a.head_decay[head];
+                const T* row = proj + token * a.row_width;
+                const T* q_row = row + a.r_offset + head * dim;
+                const T* k_row = row + a.k_offset + head * dim;
+                const int half = a.inv_freq ? a.rotary_dim >> 1 : 0;
+                const float position = (float)a.positions[token];
+                for (int i = lane; i < half; i += 32) {      // element i turns with element i + half
+                    float s, c;
+                    sincosf(position * a.inv_freq[i], &s, &c);
+                    const int at = t * padded + (i / R) * a.stride_rows + i % R;
+                    const int at2 = t * padded + ((i + half) / R) * a.stride_rows + (i + half) % R;
+                    const float ku = Num<T>::load(k_row + i), kv = Num<T>::load(k_row + i + half);
+                    k_s[at] = (ku * c - kv * s) * a.k_scale;
+                    k_s[at2] = (kv * c + ku * s) * a.k_scale;
+                    if (PASS != REC_LOCAL) {
+                        const float qu = Num<T>::load(q_row + i), qv = Num<T>::load(q_row + i + half);
+                        q_s[at] = qu * c - qv * s;
+                        q_s[at2] = qv * c + qu * s;
+                    }
+                }
+                for (int i = 2 * half + lane; i < P * R; i += 32) {
+                    const int at = t * padded + (i / R) * a.stride_rows + i % R;
+                    k_s[at] = i < dim ? Num<T>::load(k_row + i) * a.k_scale : 0.0f;
+                    q_s[at] = PASS != REC_LOCAL && i < dim ? Num<T>::load(q_row + i) : 0.0f;
+                }
+            }
+            for (int i = lane; i < (MODE == REC_RETENTION ? 0 : P * R); i += 32) {
                 float qv = 0.0f, kv = 0.0f, wv = 0.0f;
                 if (i < dim) {
                     if (MODE == REC_WKV) {
@@ -277,6 +332,7 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) matrix_recurrence_kernel(
                     } else {
                         if (PASS != REC_LOCAL) qv = a.pre[token * a.pre_width + a.q_col + qk_head * dim + i];
                         kv = a.pre[token * a.pre_width + a.k_col + qk_head * dim + i];
+                        if (MODE == REC_SSD) kv *= dt;
                     }
                 }
                 const int at = t * padded + (i / R) * a.stride_rows + i % R;
@@ -286,12 +342,12 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) matrix_recurrence_kernel(
             }
             for (int j = lane; j < vdim; j += 32)
                 v_s[t * vdim + j] = group > 0 ? 0.0f
-                                    : MODE == REC_WKV ? Num<T>::load(proj + token * a.row_width + a.v_offset + head * vdim + j)
+                                    : MODE == REC_WKV || MODE == REC_RETENTION ? Num<T>::load(proj + token * a.row_width + a.v_offset + head * vdim + j)
                                                       : a.pre[token * a.pre_width + a.v_col + head * vdim + j];
             if (MODE == REC_WKV) {
                 bonus = warp_sum(bonus);
                 if (lane == 0) scalar_s[2 * t] = bonus;
-            } else if (lane == 0) {
+            } else if (MODE == REC_DELTA && lane == 0) {
                 const float b = a.wide[token * 2 * a.heads + head], z = a.wide[token * 2 * a.heads + a.heads + head] + a.dt_bias[head];
                 const float softplus = z > 20.0f ? z : log1pf(expf(z));
                 scalar_s[2 * t] = expf(-expf(a.a_log[head]) * softplus);
@@ -337,6 +393,35 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) matrix_recurrence_kernel(
                 }
                 for (int offset = per_warp; offset < 32; offset <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, offset);
                 o = fmaf(scalar_s[2 * t], vj, sum);
+            } else if (PLAIN) {
+                const float g = scalar_s[2 * t];
+                if (PASS == REC_LOCAL) {
+#pragma unroll
+                    for (int i = 0; i < R / 4; ++i) {
+                        const float4 kk = k4[i];
+                        S[4 * i + 0] = fmaf(g, S[4 * i + 0], kk.x * vj);
+                        S[4 * i + 1] = fmaf(g, S[4 * i + 1], kk.y * vj);
+                        S[4 * i + 2] = fmaf(g, S[4 * i + 2], kk.z * vj);
+                        S[4 * i + 3] = fmaf(g, S[4 * i + 3], kk.w * vj);
+                    }
+                    move *= g;
+                    continue;
+                }
+                float sum = 0.0f;
+#pragma unroll
+                for (int i = 0; i < R / 4; ++i) {
+                    const float4 qq = q4[i], kk = k4[i];
+                    S[4 * i + 0] = fmaf(g, S[4 * i + 0], kk.x * vj);
+                    S[4 * i + 1] = fmaf(g, S[4 * i + 1], kk.y * vj);
+                    S[4 * i + 2] = fmaf(g, S[4 * i + 2], kk.z * vj);
+                    S[4 * i + 3] = fmaf(g, S[4 * i + 3], kk.w * vj);
+                    sum = fmaf(S[4 * i + 0], qq.x, sum);
+                    sum = fmaf(S[4 * i + 1], qq.y, sum);
+                    sum = fmaf(S[4 * i + 2], qq.z, sum);
+                    sum = fmaf(S[4 * i + 3], qq.w, sum);
+                }
+                for (int offset = per_warp; offset < 32; offset <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, offset);
+                o = sum;
             } else {
                 const float g = scalar_s[2 * t], beta = scalar_s[2 * t + 1];
                 float read = 0.0f;
@@ -384,6 +469,16 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) matrix_recurrence_kernel(
         __syncthreads();
         // ---- head norm, gate, store: a warp per token
         for (int t = warp; t < count; t += warps) {
+            if (MODE == REC_SSD) {      // no norm yet: what is normalised together spans several heads
+                const T* g_row = proj + (size_t)(first + t) * a.row_width + a.g_offset + head * vdim;
+                float* dst = (float*)a.out + ((size_t)(first + t) * a.heads + head) * vdim;
+                const float skip = a.skip[head];
+                for (int j = lane; j < vdim; j += 32) {
+                    const float g = Num<T>::load(g_row + j);
+                    dst[j] = fmaf(skip, v_s[t * vdim + j], o_s[t * vdim + j]) * (g / (1.0f + expf(-g)));
+                }
+                continue;
+            }
             float squares = 0.0f;
             for (int j = lane; j < vdim; j += 32) squares = fmaf(o_s[t * vdim + j], o_s[t * vdim + j], squares);
             const float inverse = rsqrtf(warp_sum(squares) / (float)vdim + a.eps);
@@ -392,7 +487,7 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) matrix_recurrence_kernel(
             const W* weight = (const W*)a.weight + (size_t)head * a.weight_stride;
             for (int j = lane; j < vdim; j += 32) {
                 const float g = Num<T>::load(g_row + j);
-                Num<T>::store(dst + j, o_s[t * vdim + j] * inverse * Num<W>::load(weight + j) * (g / (1.0f + expf(-g))));
+                Num<T>::store(dst + j, o_s[t * vdim + j] * inverse * (MODE == REC_RETENTION ? 1.0f : Num<W>::load(weight + j)) * (g / (1.0f + expf(-g))));
             }
         }
     }
@@ -408,10 +503,10 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) matrix_recurrence_kernel(
             for (int i = 0; i < R; ++i)
                 if (row0 + i < dim) move[(size_t)(row0 + i) * dim + move_column] = S[i];
         }
-        if (MODE == REC_WKV && column == 0) {
+        if ((MODE == REC_WKV || PLAIN) && column == 0) {
 #pragma unroll
             for (int i = 0; i < R; ++i)
-                if (row0 + i < dim) a.segment_move[segment_index * dim + row0 + i] = decay[i % (sizeof(decay) / sizeof(float))];
+                if (row0 + i < dim) a.segment_move[segment_index * dim + row0 + i] = PLAIN ? move : decay[i % (sizeof(decay) / sizeof(float))];
         }
         return;
     }
@@ -705,7 +800,7 @@ static int rec_launch(RecArgs& a, int mode, int n_seqs, int dtype, int weight_dt
             REC_LAUNCH_PASS(R, MODE, REC_ONE_PASS, dim3(n_seqs, a.heads));                                                 \
         } else {                                                                                                           \
             REC_LAUNCH_PASS(R, MODE, REC_LOCAL, dim3(n_seqs, a.heads, a.max_segments * (MODE == REC_DELTA ? a.groups : 1))); \
-            if (MODE == REC_WKV)                                                                                           \
+            if (MODE != REC_DELTA)                                                                                         \
                 llm_launch(rec_scan_diagonal_kernel, dim3(n_seqs, a.heads, (a.dim * a.vdim + 255) / 256), 256, 0, stream, a); \
             else if (staged_scan) {                                                                                        \
                 const int status = rec_launch_staged_scan(a, n_seqs, stream);                                              \
@@ -725,7 +820,9 @@ static int rec_launch(RecArgs& a, int mode, int n_seqs, int dtype, int weight_dt
     } while (0)
     LLM_DISPATCH_DTYPE_WEIGHT(dtype, weight_dtype, {
         if (mode == REC_WKV) REC_LAUNCH_ROWS(REC_WKV);
-        else REC_LAUNCH_ROWS(REC_DELTA);
+        else if (mode == REC_DELTA) REC_LAUNCH_ROWS(REC_DELTA);
+        else if (mode == REC_RETENTION) REC_LAUNCH_ROWS(REC_RETENTION);
+        else REC_LAUNCH_ROWS(REC_SSD);
     });
 #undef REC_LAUNCH_ROWS
 #undef REC_LAUNCH
@@ -764,4 +861,39 @@ LLM_EXPORT int llm_delta_rule_recurrent(const void* proj, int row_width, int g_o
     a.weight_stride = 0; a.state = state; a.state_slots = state_slots; a.q_start = q_start; a.out = out; a.heads = heads;
     a.dim = dim; a.vdim = vdim; a.eps = eps;
     return rec_launch(a, REC_DELTA, n_seqs, dtype, weight_dtype, stream);
+}
+
+LLM_EXPORT int llm_retention_recurrent(const void* proj, int row_width, int q_offset, int k_offset, int v_offset, int g_offset,
+                                       const float* head_decay, const int* positions, const float* inv_freq, int rotary_dim,
+                                       float k_scale, float* state, const int* state_slots, const int* q_start, void* out, int n_seqs,
+                                       int heads, int dim, int vdim, float eps, int dtype, int segment, int max_segments,
+                                       float* segment_state, float* segment_move, cudaStream_t stream) {
+    if (inv_freq && (rotary_dim < 0 || rotary_dim % 2 || rotary_dim > dim)) {
+        llm_set_error("retention_recurrent: %d rotating elements must be an even number of at most %d", rotary_dim, dim);
+        return LLM_REFUSED;
+    }
+    RecArgs a = {};
+    a.segment = segment; a.max_segments = max_segments; a.segment_state = segment_state; a.segment_move = segment_move;
+    a.proj = proj; a.row_width = row_width; a.r_offset = q_offset; a.k_offset = k_offset; a.v_offset = v_offset; a.g_offset = g_offset;
+    a.head_decay = head_decay; a.positions = positions; a.inv_freq = inv_freq; a.rotary_dim = rotary_dim; a.k_scale = k_scale;
+    a.state = state; a.state_slots = state_slots; a.q_start = q_start; a.out = out; a.heads = heads; a.dim = dim; a.vdim = vdim;
+    a.eps = eps; a.qk_heads = heads;
+    return rec_launch(a, REC_RETENTION, n_seqs, dtype, dtype, stream);
+}
+
+LLM_EXPORT int llm_ssd_recurrent(const void* proj, int row_width, int g_offset, const float* pre, int pre_width, int v_col, int k_col,
+                                 int q_col, const float* wide, const float* a_log, const float* dt_bias, const float* skip,
+                                 float* state, const int* state_slots, const int* q_start, float* out, int n_seqs, int heads,
+                                 int groups, int dim, int vdim, int dtype, int segment, int max_segments, float* segment_state,
+                                 float* segment_move, cudaStream_t stream) {
+    if (groups <= 0 || heads % groups) {
+        llm_set_error("ssd_recurrent: %d heads are no multiple of %d groups", heads, groups);
+        return LLM_REFUSED;
+    }
+    RecArgs a = {};
+    a.segment = segment; a.max_segments = max_segments; a.segment_state = segment_state; a.segment_move = segment_move;
+    a.proj = proj; a.row_width = row_width; a.g_offset = g_offset; a.pre = pre; a.pre_width = pre_width; a.v_col = v_col;
+    a.k_col = k_col; a.q_col = q_col; a.qk_heads = groups; a.wide = wide; a.a_log = a_log; a.dt_bias = dt_bias; a.skip = skip;
+    a.state = state; a.state_slots = state_slots; a.q_start = q_start; a.out = out; a.heads = heads; a.dim = dim; a.vdim = vdim;
+    return rec_launch(a, REC_SSD, n_seqs, dtype, dtype, stream);
 }

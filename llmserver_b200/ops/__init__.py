@@ -22,7 +22,8 @@ __all__ = ["KernelError", "embedding", "add_rmsnorm", "rmsnorm", "silu_mul", "sa
            "clamped_glu", "gemm_f32", "linear", "linear_wide", "qkv_projection", "gate_up_silu", "interleave_gate_up", "require_device", "library", "launch_count",
            "RowScaled", "StreamSink", "STREAM_ROWS", "unscaled_rows_supported", "norm_rope_units", "rotate_units", "attention_diff", "gla_supported",
            "gla_recurrent", "head_linear", "relu_squared", "tanh_narrow", "softcap_", "scaled_sum", "token_shift_mix",
-           "short_conv_units", "matrix_recurrence_supported", "wkv_recurrent", "delta_rule_recurrent"]
+           "short_conv_units", "matrix_recurrence_supported", "wkv_recurrent", "delta_rule_recurrent", "retention_recurrent", "ssd_recurrent",
+           "gelu_mul", "grouped_rmsnorm", "conv_norm_kv"]
 
 
 def embedding(table: torch.Tensor, ids: torch.Tensor, out: Optional[torch.Tensor] = None, scale: float = 1.0) -> torch.Tensor:
@@ -88,15 +89,23 @@ def silu_mul(gate_up: torch.Tensor, out: Optional[torch.Tensor] = None, group: i
     """out[n, i] = silu(gate_up[n, i]) * gate_up[n, I + i]; gate_up is [N, 2 I], gate half first.  With ``group`` > 0
     gate and up columns are interleaved in groups of that many: output i finds its gate value at column
     (i // group) * 2 * group + i % group and its up value ``group`` columns further."""
+    return _glu("llm_silu_mul", gate_up, out, group)
+
+
+def gelu_mul(gate_up: torch.Tensor, out: Optional[torch.Tensor] = None, group: int = 0) -> torch.Tensor:
+    """``silu_mul`` with gelu in its tanh form, 0.5 x (1 + tanh(sqrt(2 / pi) (x + 0.044715 x^3))), in silu's place."""
+    return _glu("llm_gelu_mul", gate_up, out, group)
+
+
+def _glu(launcher: str, gate_up: torch.Tensor, out: Optional[torch.Tensor], group: int) -> torch.Tensor:
     check(gate_up, "gate_up")
     rows, doubled = gate_up.shape
     if doubled % 2:
         raise KernelError(f"gate_up's last dimension must be even, got {doubled}")
     if out is None:
         out = torch.empty((rows, doubled // 2), dtype=gate_up.dtype, device=gate_up.device)
-    check(out, "silu_mul output", gate_up.dtype, doubled // 2)
-    call("llm_silu_mul", gate_up.data_ptr(), out.data_ptr(), rows, doubled // 2, int(group), dtype_code(gate_up.dtype),
-         stream_handle())
+    check(out, "the activation's output", gate_up.dtype, doubled // 2)
+    call(launcher, gate_up.data_ptr(), out.data_ptr(), rows, doubled // 2, int(group), dtype_code(gate_up.dtype), stream_handle())
     return out
 
 
@@ -196,10 +205,13 @@ def attention_generic(q: torch.Tensor, q_stride: int, k_pages: torch.Tensor, v_p
                       block_tables: torch.Tensor, seq_of_token: torch.Tensor, positions: torch.Tensor,
                       n_q_heads: int, n_kv_heads: int, head_dim: int, scale: float, window: int = 0,
                       out: Optional[torch.Tensor] = None, error_flag: Optional[torch.Tensor] = None,
-                      value_dim: Optional[int] = None, sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
+                      value_dim: Optional[int] = None, sinks: Optional[torch.Tensor] = None, chunk: int = 0,
+                      bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal (optionally windowed) attention of every token over its sequence's pages, 32-bit
     arithmetic.  ``q`` holds head h of token n at q[n * q_stride + h * D]; returns [N, Hq * Dv], Dv = ``value_dim``
-    (default D).  ``sinks`` (float32 [Hq]): one more term exp(sinks[h]) in each head's softmax denominator.  A
+    (default D).  ``sinks`` (float32 [Hq]): one more term exp(sinks[h]) in each head's softmax denominator.  ``chunk`` > 0:
+    a query sees the keys of its own chunk of that many positions only.  ``bias`` (float32 [Hq, L]): bias[h, min(n, L - 1)]
+    is added to the scaled score of the key n positions back.  A
     block-table entry that names no page of the pool is not followed: page 0 is read instead and ``error_flag``
     (default: the device's shared flag) is set to 5."""
     check(q, "q")
@@ -216,16 +228,24 @@ def attention_generic(q: torch.Tensor, q_stride: int, k_pages: torch.Tensor, v_p
         check(sinks, "sinks", torch.float32)
         if sinks.numel() != n_q_heads:
             raise KernelError(f"sinks must hold one number per query head ({n_q_heads}), got {sinks.numel()}")
+    _check_bias(bias, n_q_heads)
     if out is None:
         out = torch.empty((tokens, n_q_heads * value_dim), dtype=q.dtype, device=q.device)
     check(out, "attention output", q.dtype, n_q_heads * value_dim)
     call("llm_attention_generic", q.data_ptr(), q_stride, k_pages.data_ptr(), v_pages.data_ptr(),
          block_tables.data_ptr(), block_tables.shape[-1], seq_of_token.data_ptr(), positions.data_ptr(),
          out.data_ptr(), tokens, n_q_heads, n_kv_heads, head_dim, value_dim, k_pages.shape[2], k_pages.shape[0],
-         float(scale), int(window), pointer(sinks),
+         float(scale), int(window), pointer(sinks), int(chunk), pointer(bias), 0 if bias is None else bias.shape[1],
          (error_flag if error_flag is not None else wait_error_flag(q.device)).data_ptr(), dtype_code(q.dtype),
          stream_handle())
     return out
+
+
+def _check_bias(bias: Optional[torch.Tensor], n_q_heads: int) -> None:
+    if bias is not None:
+        check(bias, "distance bias", torch.float32)
+        if bias.dim() != 2 or bias.shape[0] != n_q_heads or bias.shape[1] == 0:
+            raise KernelError(f"the distance bias must be [{n_q_heads}, distances], got {tuple(bias.shape)}")
 
 
 def rope_kv_write_split(qkv: torch.Tensor, inv_freq: Optional[torch.Tensor], magnitude: float, positions: torch.Tensor,
@@ -553,20 +573,24 @@ def token_shift_mix(h: torch.Tensor, shift_state: torch.Tensor, batch, mu: torch
 
 
 def short_conv_units(x: torch.Tensor, column: int, taps_w: torch.Tensor, state: torch.Tensor, batch, n_unit_norm: int,
-                     unit_dim: int, n_scaled: int, n_plain: int, plain_dim: int, norm_eps: float, scale: float) -> torch.Tensor:
+                     unit_dim: int, n_scaled: int, n_plain: int, plain_dim: int, norm_eps: float, scale: float,
+                     bias: Optional[torch.Tensor] = None, channels: Optional[int] = None) -> torch.Tensor:
     """A short causal convolution over time, channel by channel, then SiLU:
 
-        y_t[c] = silu(sum_j taps_w[c, j] * x_(t - taps + 1 + j)[c])        zeros before a sequence's start
+        y_t[c] = silu(sum_j taps_w[c, j] * x_(t - taps + 1 + j)[c] + bias[c])      zeros before a sequence's start
 
     over the channels that start at ``column`` of ``x`` [N, row]; ``taps_w`` is float32 [channels, taps], the last column
     the current token's.  Channels come in units: first ``n_unit_norm`` units of ``unit_dim`` channels, each made a unit
     vector y / sqrt(sum(y^2) + norm_eps), the first ``n_scaled`` of them multiplied by ``scale``; then ``n_plain`` units of
-    ``plain_dim`` channels that stay as they are.  A sequence's last taps - 1 inputs live in its slot of ``state``
+    ``plain_dim`` channels that stay as they are (the last of them cut short where ``channels`` says so).  ``bias`` (float32
+    [channels]) may be absent.  A sequence's last taps - 1 inputs live in its slot of ``state``
     (float32 [slots, max(taps - 1, 1), channels]) and are brought up to date.  Returns float32 [N, channels]."""
     check(x, "x")
     tokens, row_width = x.shape
-    channels = n_unit_norm * unit_dim + n_plain * plain_dim
+    channels = n_unit_norm * unit_dim + n_plain * plain_dim if channels is None else int(channels)
     taps = taps_w.shape[1]
+    if bias is not None:
+        check(bias, "convolution bias", torch.float32, channels)
     check(taps_w, "convolution weights", torch.float32)
     if taps_w.shape[0] != channels or column < 0 or column + channels > row_width:
         raise KernelError(f"{channels} channels from column {column} do not fit rows of {row_width} or weights {tuple(taps_w.shape)}")
@@ -576,7 +600,66 @@ def short_conv_units(x: torch.Tensor, column: int, taps_w: torch.Tensor, state: 
     out = torch.empty((tokens, channels), dtype=torch.float32, device=x.device)
     call("llm_short_conv_units", x.data_ptr(), row_width, int(column), taps_w.data_ptr(), int(taps), state.data_ptr(),
          batch.state_slots.data_ptr(), batch.q_start.data_ptr(), out.data_ptr(), batch.n_seqs, int(batch.max_q_len), int(n_unit_norm),
-         int(unit_dim), int(n_scaled), int(n_plain), int(plain_dim), float(norm_eps), float(scale), dtype_code(x.dtype), stream_handle())
+         int(unit_dim), int(n_scaled), int(n_plain), int(plain_dim), float(norm_eps), float(scale), pointer(bias), channels, dtype_code(x.dtype),
+         stream_handle())
+    return out
+
+
+def conv_norm_kv(x: torch.Tensor, taps_w: Optional[torch.Tensor], state: Optional[torch.Tensor], batch, block_tables: torch.Tensor,
+                 k_pages: torch.Tensor, v_pages: torch.Tensor, n_q_heads: int, n_kv_heads: int, key_dim: int, value_dim: int,
+                 q_weight: Optional[torch.Tensor] = None, k_weight: Optional[torch.Tensor] = None, eps: float = 0.0,
+                 write_cache: bool = True) -> torch.Tensor:
+    """From a packed projection ``x`` [N, >= Hq D + Hkv D + Hkv Dv] to attention's inputs: a causal convolution over time on
+    every channel of q, k and v (``taps_w`` float32 [taps, channels], the last row the current token's; None: no
+    convolution), then RMS norms over all query channels and over all key channels of a token (``q_weight`` [Hq D],
+    ``k_weight`` [Hkv D]; None: no norm), then k and v into the pages [page, Hkv, slot, D | Dv].  A sequence's last taps - 1
+    rows of ``x`` live in its slot of ``state`` (float32 [slots, max(taps - 1, 1), channels]) and are brought up to date.
+    Returns the queries [N, Hq D] in x's type; everything in between is 32-bit."""
+    check(x, "packed projection")
+    tokens, row_width = x.shape
+    channels = (n_q_heads + n_kv_heads) * key_dim + n_kv_heads * value_dim
+    taps = 1
+    if taps_w is not None:
+        check(taps_w, "convolution weights", torch.float32, channels)
+        taps = taps_w.shape[0]
+        if taps > 1:
+            check(state, "convolution state", torch.float32, channels)
+            if state.dim() != 3 or state.shape[1] != taps - 1:
+                raise KernelError(f"the convolution state must be [slots, {taps - 1}, {channels}], got {tuple(state.shape)}")
+    weight_dtype = x.dtype
+    for name, tensor, size in (("q norm weight", q_weight, n_q_heads * key_dim), ("k norm weight", k_weight, n_kv_heads * key_dim)):
+        if tensor is not None:
+            check(tensor, name, last_dim=size)
+            weight_dtype = tensor.dtype
+    if q_weight is not None and k_weight is not None and q_weight.dtype != k_weight.dtype:
+        raise KernelError("q and k norm weights must share a dtype")
+    check(block_tables, "block_tables", torch.int32)
+    check(k_pages, "k pages", x.dtype, key_dim)
+    check(v_pages, "v pages", x.dtype, value_dim)
+    if k_pages.dim() != 4 or k_pages.shape[1] != n_kv_heads or k_pages.shape[:-1] != v_pages.shape[:-1]:
+        raise KernelError(f"pages must be [pages, {n_kv_heads}, page_size, {key_dim} | {value_dim}], got "
+                          f"{tuple(k_pages.shape)} and {tuple(v_pages.shape)}")
+    q_out = torch.empty((tokens, n_q_heads * key_dim), dtype=x.dtype, device=x.device)
+    call("llm_conv_norm_kv", x.data_ptr(), row_width, pointer(taps_w), int(taps), pointer(state) if taps > 1 else 0,
+         batch.state_slots.data_ptr(), batch.q_start.data_ptr(), batch.positions.data_ptr(), block_tables.data_ptr(),
+         block_tables.shape[-1], pointer(q_weight), pointer(k_weight), float(eps), q_out.data_ptr(), k_pages.data_ptr(),
+         v_pages.data_ptr(), batch.n_seqs, int(batch.max_q_len), n_q_heads, n_kv_heads, int(key_dim), int(value_dim), k_pages.shape[2],
+         k_pages.shape[0], int(write_cache), batch.error_flag.data_ptr(), dtype_code(x.dtype), dtype_code(weight_dtype),
+         stream_handle())
+    return q_out
+
+
+def grouped_rmsnorm(x: torch.Tensor, weight: torch.Tensor, parts: int, eps: float, act_dtype: torch.dtype) -> torch.Tensor:
+    """RMS norm of 32-bit rows in ``parts`` equal pieces, each divided by its own root mean square, times ``weight`` [width];
+    the result in the activation type."""
+    check(x, "x", torch.float32)
+    rows, width = x.shape
+    check(weight, "norm weight", last_dim=width)
+    if parts <= 0 or width % parts:
+        raise KernelError(f"rows of {width} do not divide into {parts} equal pieces")
+    out = torch.empty((rows, width), dtype=act_dtype, device=x.device)
+    call("llm_grouped_rmsnorm", x.data_ptr(), weight.data_ptr(), out.data_ptr(), rows, int(parts), width // int(parts), float(eps),
+         dtype_code(act_dtype), dtype_code(weight.dtype), stream_handle())
     return out
 
 
@@ -698,6 +781,78 @@ def delta_rule_recurrent(proj: torch.Tensor, g_column: int, pre: torch.Tensor, w
     return out
 
 
+def _check_matrix_state(state: torch.Tensor, heads: int, dim: int, value_dim: int) -> None:
+    check(state, "recurrent state", torch.float32, value_dim)
+    if state.dim() != 4 or tuple(state.shape[1:]) != (heads, dim, value_dim):
+        raise KernelError(f"the state must be [slots, {heads}, {dim}, {value_dim}], got {tuple(state.shape)}")
+
+
+def retention_recurrent(proj: torch.Tensor, q_column: int, k_column: int, v_column: int, g_column: int, decay: torch.Tensor,
+                        inv_freq: Optional[torch.Tensor], state: torch.Tensor, batch, heads: int, dim: int, value_dim: int,
+                        k_scale: float, eps: float, segment: Optional[int] = None) -> torch.Tensor:
+    """Retention, sequence by sequence, from and into each sequence's slot of ``state`` (float32 [slots, heads, dim, value_dim]):
+
+        S <- decay_h S + k v^T;  o = S^T q;  out = o / sqrt(mean(o^2) + eps) * silu(g)        per head
+
+    q, k (heads * dim columns each), v and g (heads * value_dim) start at the given columns of ``proj``; q and k are rotated
+    by the token's position as they are read (the first 2 * len(inv_freq) elements of each head, element i with element
+    i + len(inv_freq); ``inv_freq`` None: nothing rotates), k is then multiplied by ``k_scale``; ``decay`` float32 [heads].
+    Returns [N, heads * value_dim] in the activation type; rotation and recurrence are 32-bit.  ``segment`` as for
+    ``delta_rule_recurrent``."""
+    check(proj, "packed projection")
+    tokens, row_width = proj.shape
+    check(decay, "decays", torch.float32, heads)
+    if inv_freq is not None:
+        check(inv_freq, "inv_freq", torch.float32)
+    _check_matrix_state(state, heads, dim, value_dim)
+    for column, size in ((q_column, heads * dim), (k_column, heads * dim), (v_column, heads * value_dim), (g_column, heads * value_dim)):
+        if column < 0 or column + size > row_width:
+            raise KernelError(f"columns {column}..{column + size} lie outside a row of {row_width}")
+    out = torch.empty((tokens, heads * value_dim), dtype=proj.dtype, device=proj.device)
+    segment, segments, segment_state, segment_move = _recurrence_segments(batch, proj, segment, heads, dim, value_dim, 1)
+    call("llm_retention_recurrent", proj.data_ptr(), row_width, int(q_column), int(k_column), int(v_column), int(g_column),
+         decay.data_ptr(), batch.positions.data_ptr(), pointer(inv_freq), 0 if inv_freq is None else 2 * inv_freq.numel(),
+         float(k_scale), state.data_ptr(), batch.state_slots.data_ptr(), batch.q_start.data_ptr(), out.data_ptr(), batch.n_seqs,
+         int(heads), int(dim), int(value_dim), float(eps), dtype_code(proj.dtype), segment, segments, pointer(segment_state),
+         pointer(segment_move), stream_handle())
+    return out
+
+
+def ssd_recurrent(proj: torch.Tensor, g_column: int, pre: torch.Tensor, v_column: int, k_column: int, q_column: int,
+                  wide: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor, skip: torch.Tensor, state: torch.Tensor, batch,
+                  heads: int, groups: int, dim: int, value_dim: int, segment: Optional[int] = None) -> torch.Tensor:
+    """The state-space recurrence with one decay per head and token, from and into each sequence's slot of ``state`` (float32
+    [slots, heads, dim, value_dim]):
+
+        dt = softplus(wide + dt_bias);  S <- exp(-exp(A) dt) S + dt B x^T;  o = S^T C;  out = (o + D x) * silu(g)    per head
+
+    ``pre`` float32 holds x (heads * value_dim columns from ``v_column``), B and C (groups * dim columns each from ``k_column``
+    and ``q_column``; head h reads group h // (heads / groups)); ``wide`` float32 [N, heads]; ``a_log`` (A), ``dt_bias`` and
+    ``skip`` (D) float32 [heads]; the gate's pre-activation is heads * value_dim columns of ``proj`` from ``g_column``.  Returns
+    float32 [N, heads * value_dim] (what is normalised next spans heads).  ``segment`` as for ``delta_rule_recurrent``."""
+    check(proj, "packed projection")
+    tokens, row_width = proj.shape
+    if g_column < 0 or g_column + heads * value_dim > row_width:
+        raise KernelError(f"the gate's columns {g_column}..{g_column + heads * value_dim} lie outside a row of {row_width}")
+    check(pre, "convolved x, B, C", torch.float32)
+    for column, size in ((v_column, heads * value_dim), (k_column, groups * dim), (q_column, groups * dim)):
+        if column < 0 or column + size > pre.shape[1]:
+            raise KernelError(f"columns {column}..{column + size} lie outside a row of {pre.shape[1]}")
+    check(wide, "dt", torch.float32, heads)
+    for name, tensor in (("A", a_log), ("dt bias", dt_bias), ("D", skip)):
+        check(tensor, name, torch.float32, heads)
+    _check_matrix_state(state, heads, dim, value_dim)
+    if pre.shape[0] != tokens or wide.shape[0] != tokens:
+        raise KernelError("every input needs one row per token")
+    out = torch.empty((tokens, heads * value_dim), dtype=torch.float32, device=proj.device)
+    segment, segments, segment_state, segment_move = _recurrence_segments(batch, proj, segment, heads, dim, value_dim, 1)
+    call("llm_ssd_recurrent", proj.data_ptr(), row_width, int(g_column), pre.data_ptr(), pre.shape[1], int(v_column), int(k_column),
+         int(q_column), wide.data_ptr(), a_log.data_ptr(), dt_bias.data_ptr(), skip.data_ptr(), state.data_ptr(),
+         batch.state_slots.data_ptr(), batch.q_start.data_ptr(), out.data_ptr(), batch.n_seqs, int(heads), int(groups), int(dim),
+         int(value_dim), dtype_code(proj.dtype), segment, segments, pointer(segment_state), pointer(segment_move), stream_handle())
+    return out
+
+
 def head_linear(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
     """out[n, h, :] = weight[h] x[n, h, :] for ``x`` [N, H * K] and ``weight`` [H, R, K]: every head has a matrix of its
     own.  Returns [N, H * R] in the activation type.  Steps of many rows in bfloat16 go to the library's batched product;
@@ -718,37 +873,61 @@ def head_linear(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
 HEAD_LINEAR_ROWS = 32     # up to this many tokens a bfloat16 step multiplies row by row
 
 
+def _route_rule(experts: int, scores: str, groups: Optional[tuple], renormalise: bool):
+    """(softmax, groups, keep, renormalise) as the launchers take them."""
+    if scores not in ("sigmoid", "softmax"):
+        raise KernelError(f"router scores are 'sigmoid' or 'softmax', not {scores!r}")
+    count, keep = (int(groups[0]), int(groups[1])) if groups else (0, 0)
+    if groups and experts % count:
+        raise KernelError(f"{experts} experts do not form {count} equal groups")
+    return int(scores == "softmax"), count, keep, int(bool(renormalise))
+
+
 def moe_route(x: torch.Tensor, router: torch.Tensor, correction: Optional[torch.Tensor], top: int, scale: float,
-              counts: Optional[torch.Tensor] = None):
+              counts: Optional[torch.Tensor] = None, scores: str = "sigmoid", groups: Optional[tuple] = None,
+              renormalise: bool = False, gate: bool = False):
     """Per token the ``top`` experts with the largest sigmoid(router x) + correction (ties: the lower index) and their
     weights sigmoid(router x) * scale: (chosen int32 [N, top], weights float32 [N, top]).  ``router`` [E, H] and
-    ``correction`` [E] are float32; with ``counts`` (int32 [E]) each choice also adds one to its expert's count."""
+    ``correction`` [E] are float32; with ``counts`` (int32 [E]) each choice also adds one to its expert's count.
+
+    ``scores`` "softmax": softmax over all experts in the sigmoid's place.  ``groups`` = (count, keep): only experts of the
+    ``keep`` best of ``count`` equal groups of neighbours can be chosen, a group's score being the largest in it.
+    ``renormalise``: the chosen weights are divided by their sum (+ 1e-20), then scaled.  ``gate``: the router has one more
+    row, [E + 1, H], and the sigmoid of its product is returned as a third result (float32 [N])."""
     check(x, "x")
     tokens, width = x.shape
     check(router, "router weight", torch.float32, width)
-    experts = router.shape[0]
+    experts = router.shape[0] - int(bool(gate))
+    rule = _route_rule(experts, scores, groups, renormalise)
     if correction is not None:
         check(correction, "router correction", torch.float32, experts)
     if counts is not None:
         check(counts, "expert counts", torch.int32, experts)
     chosen = torch.empty((tokens, top), dtype=torch.int32, device=x.device)
     weights = torch.empty((tokens, top), dtype=torch.float32, device=x.device)
+    gate_out = torch.empty((tokens,), dtype=torch.float32, device=x.device) if gate else None
     call("llm_moe_route", x.data_ptr(), router.data_ptr(), pointer(correction), chosen.data_ptr(), weights.data_ptr(),
-         pointer(counts), tokens, width, experts, int(top), float(scale), dtype_code(x.dtype), stream_handle())
-    return chosen, weights
+         pointer(counts), tokens, width, experts, int(top), float(scale), *rule, pointer(gate_out), dtype_code(x.dtype),
+         stream_handle())
+    return (chosen, weights, gate_out) if gate else (chosen, weights)
 
 
-def moe_select(logits: torch.Tensor, correction: Optional[torch.Tensor], top: int, scale: float):
-    """``moe_route``'s choice from router logits that a product has already made: logits float32 [N, E]."""
+def moe_select(logits: torch.Tensor, correction: Optional[torch.Tensor], top: int, scale: float, scores: str = "sigmoid",
+               groups: Optional[tuple] = None, renormalise: bool = False, gate: bool = False):
+    """``moe_route``'s choice from router logits that a product has already made: logits float32 [N, E], or [N, E + 1] with
+    the ``gate``'s pre-activation last."""
     check(logits, "router logits", torch.float32)
     tokens, experts = logits.shape
+    experts -= int(bool(gate))
+    rule = _route_rule(experts, scores, groups, renormalise)
     if correction is not None:
         check(correction, "router correction", torch.float32, experts)
     chosen = torch.empty((tokens, top), dtype=torch.int32, device=logits.device)
     weights = torch.empty((tokens, top), dtype=torch.float32, device=logits.device)
+    gate_out = torch.empty((tokens,), dtype=torch.float32, device=logits.device) if gate else None
     call("llm_moe_select", logits.data_ptr(), pointer(correction), chosen.data_ptr(), weights.data_ptr(), tokens, experts,
-         int(top), float(scale), stream_handle())
-    return chosen, weights
+         int(top), float(scale), *rule, pointer(gate_out), stream_handle())
+    return (chosen, weights, gate_out) if gate else (chosen, weights)
 
 
 def indexed_linear(x: torch.Tensor, weight: torch.Tensor, index: Optional[torch.Tensor], pairs: int, in_div: int = 1,
@@ -796,8 +975,17 @@ def _gate_constants(gated: Optional[tuple]):
     return float(gated[0]), float(gated[1]), float(gated[2]) if len(gated) > 2 else 1.0
 
 
-def moe_combine(down: torch.Tensor, weights: torch.Tensor, shared_out: Optional[torch.Tensor], act_dtype: torch.dtype) -> torch.Tensor:
-    """out[t] = sum_j weights[t, j] * down[t * top + j] (+ shared_out[t]); ``down`` float32 [N * top, H]."""
+def _check_shared_gate(shared_gate: Optional[torch.Tensor], tokens: int) -> None:
+    if shared_gate is not None:
+        check(shared_gate, "shared expert gate", torch.float32)
+        if shared_gate.numel() != tokens:
+            raise KernelError(f"the shared expert's gate has {shared_gate.numel()} numbers for {tokens} tokens")
+
+
+def moe_combine(down: torch.Tensor, weights: torch.Tensor, shared_out: Optional[torch.Tensor], act_dtype: torch.dtype,
+                shared_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """out[t] = sum_j weights[t, j] * down[t * top + j] (+ shared_gate[t] * shared_out[t]); ``down`` float32 [N * top, H],
+    ``shared_gate`` float32 [N] (absent: 1)."""
     check(down, "expert outputs", torch.float32)
     check(weights, "routing weights", torch.float32)
     tokens, top = weights.shape
@@ -806,8 +994,9 @@ def moe_combine(down: torch.Tensor, weights: torch.Tensor, shared_out: Optional[
         raise KernelError(f"{down.shape[0]} expert outputs for {tokens} tokens with {top} experts each")
     if shared_out is not None:
         check(shared_out, "shared expert output", act_dtype, width)
+    _check_shared_gate(shared_gate, tokens)
     out = torch.empty((tokens, width), dtype=act_dtype, device=down.device)
-    call("llm_moe_combine", down.data_ptr(), weights.data_ptr(), pointer(shared_out), out.data_ptr(), tokens, width, top,
+    call("llm_moe_combine", down.data_ptr(), weights.data_ptr(), pointer(shared_out), pointer(shared_gate), out.data_ptr(), tokens, width, top,
          dtype_code(act_dtype), stream_handle())
     return out
 
@@ -889,17 +1078,19 @@ def moe_grouped(x: torch.Tensor, weight: torch.Tensor, plan: ExpertPlan, gather_
 
 
 def moe_combine_rows(down: torch.Tensor, plan: ExpertPlan, weights: torch.Tensor, shared_out: Optional[torch.Tensor],
-                     act_dtype: torch.dtype) -> torch.Tensor:
-    """out[t] = sum_j weights[t, j] * down[row_of_pair[t * top + j]] (+ shared_out[t]); ``down`` float32 in the plan's order."""
+                     act_dtype: torch.dtype, shared_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """out[t] = sum_j weights[t, j] * down[row_of_pair[t * top + j]] (+ shared_gate[t] * shared_out[t]); ``down`` float32 in
+    the plan's order, ``shared_gate`` float32 [N] (absent: 1)."""
     check(down, "expert outputs", torch.float32)
     check(weights, "routing weights", torch.float32)
     tokens, top = weights.shape
     width = down.shape[-1]
     if shared_out is not None:
         check(shared_out, "shared expert output", act_dtype, width)
+    _check_shared_gate(shared_gate, tokens)
     out = torch.empty((tokens, width), dtype=act_dtype, device=down.device)
     call("llm_moe_combine_rows", down.data_ptr(), plan.row_of_pair.data_ptr(), weights.data_ptr(), pointer(shared_out),
-         out.data_ptr(), tokens, width, top, dtype_code(act_dtype), stream_handle())
+         pointer(shared_gate), out.data_ptr(), tokens, width, top, dtype_code(act_dtype), stream_handle())
     return out
 
 
@@ -992,25 +1183,31 @@ def qkv_projection(x, weight: torch.Tensor, q_weight: Optional[torch.Tensor], k_
 def attention(qkv: torch.Tensor, batch, block_tables: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
               n_q_heads: int, n_kv_heads: int, head_dim: int, scale: float, window: int = 0,
               value_dim: Optional[int] = None, sinks: Optional[torch.Tensor] = None, precise: bool = False,
-              q_stride: Optional[int] = None) -> torch.Tensor:
+              q_stride: Optional[int] = None, chunk: int = 0, bias: Optional[torch.Tensor] = None,
+              bias_log2: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of a step's tokens over the paged cache; ``qkv`` is the packed projection whose Q
     heads have been normalised and rotated in place (``q_stride``: elements from one token's queries to the next's,
     where they are not such a packed row).  Chooses the kernel by dtype, head size and the
-    shape of the batch; every choice computes the same function.  ``value_dim`` (default: head_dim) and ``sinks`` as
-    in ``attention_generic``.  ``precise``: the attention weights may not be rounded to bfloat16 on their way into the
+    shape of the batch; every choice computes the same function.  ``value_dim`` (default: head_dim) and ``sinks``,
+    ``chunk`` and ``bias`` as in ``attention_generic``; ``bias_log2``: the bias times log2(e), which the tensor-core kernels
+    take (made here when it is not given).  ``precise``: the attention weights may not be rounded to bfloat16 on their way into the
     P V product (the tensor-core kernels then carry each as two bfloat16 numbers)."""
     value_dim = head_dim if value_dim is None else int(value_dim)
     if q_stride is None:
         q_stride = (n_q_heads + n_kv_heads) * head_dim + n_kv_heads * value_dim
     if qkv.dtype == torch.bfloat16:
         from . import attention_bf16
-        if value_dim == head_dim and sinks is None and not precise:
+        if value_dim == head_dim and sinks is None and not precise and not chunk and bias is None:
             result = attention_bf16.try_attention(qkv, q_stride, batch, block_tables, k_pages, v_pages, n_q_heads,
                                                   n_kv_heads, head_dim, scale, window)
         else:
             result = attention_bf16.try_attention_precise(qkv, q_stride, batch, block_tables, k_pages, v_pages, n_q_heads,
-                                                          n_kv_heads, head_dim, value_dim, scale, window, sinks)
+                                                          n_kv_heads, head_dim, value_dim, scale, window, sinks, chunk,
+                                                          bias_log2 if bias_log2 is not None or bias is None else bias * LOG2E)
         if result is not None:
             return result
     return attention_generic(qkv, q_stride, k_pages, v_pages, block_tables, batch.seq_of_token, batch.positions,
-                             n_q_heads, n_kv_heads, head_dim, scale, window, value_dim=value_dim, sinks=sinks)
+                             n_q_heads, n_kv_heads, head_dim, scale, window, value_dim=value_dim, sinks=sinks, chunk=chunk, bias=bias)
+
+
+LOG2E = 1.4426950408889634

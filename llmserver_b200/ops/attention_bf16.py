@@ -73,13 +73,14 @@ def supported(head_dim: int, n_q_heads: int, n_kv_heads: int) -> bool:
     return bool(library().llm_attention_mma_supports(head_dim, n_q_heads, n_kv_heads))
 
 
-def plan(batch, group: int, n_kv_heads: int, device=None, blocks_per_sm: int = DECODE_BLOCKS_PER_SM, cluster: bool = None):
+def plan(batch, group: int, n_kv_heads: int, device=None, blocks_per_sm: int = DECODE_BLOCKS_PER_SM, cluster: bool = None,
+         span: int = None):
     """Launch shape of a batch, derived once per step from its host-side lengths (and the number of SMs: the split
     count fixes the order of the partial sums, so it is a function of the batch and the GPU model only).
     ``blocks_per_sm``: decode blocks an SM holds at a time; ``cluster``: whether splits merge inside a cluster (which
-    bounds their number) or through the merge kernel."""
+    bounds their number) or through the merge kernel; ``span``: the most keys a query sees, where that is bounded."""
     cluster = CLUSTER_MERGE if cluster is None else cluster
-    key = ("attention_mma", group, n_kv_heads, blocks_per_sm, cluster)
+    key = ("attention_mma", group, n_kv_heads, blocks_per_sm, cluster, span)
     cached = batch.scratch.get(key)
     if cached is not None:
         return cached
@@ -91,6 +92,8 @@ def plan(batch, group: int, n_kv_heads: int, device=None, blocks_per_sm: int = D
     split_len, max_splits = MIN_SPLIT, 1
     if run_decode:
         longest = max(context for context, length in zip(batch.context_lens, batch.q_lens) if length == 1)
+        if span is not None:
+            longest = min(longest, span + TILE)     # + TILE: the first visible key may lie inside a tile
         # As many equal splits of the longest context as give about one wave of blocks (two per SM); with a
         # wave's worth of (sequence, kv head) pairs already, no split at all.  Measured on the 8B head shape:
         # equal splits beat ragged ones, and one wave beats one and a half.
@@ -192,10 +195,11 @@ PRECISE_DECODE_BLOCKS_PER_SM = int(os.environ.get("LLMSERVER_B200_PRECISE_DECODE
 
 
 def try_attention_precise(qkv, q_stride, batch, block_tables, k_pages, v_pages, n_q_heads, n_kv_heads, head_dim, value_dim,
-                          scale, window, sinks):
+                          scale, window, sinks, chunk=0, bias_log2=None):
     """The tensor-core kernels in the form that keeps attention weights at 16 significant bits through the P V product,
-    takes value heads of another size than key heads and adds exp(sinks[h]) to each softmax denominator; None when the
-    sizes are not ones it takes (64 or 128 each)."""
+    takes value heads of another size than key heads and adds exp(sinks[h]) to each softmax denominator; with ``chunk`` a
+    query sees the keys of its own chunk of positions, with ``bias_log2`` (float32 [Hq, distances], times log2(e)) scores get
+    a bias by distance.  None when the sizes are not ones it takes (64 or 128 each)."""
     if not library().llm_attention_mma_sinks_supports(head_dim, value_dim, n_q_heads, n_kv_heads):
         return None
     check(qkv, "qkv", torch.bfloat16)
@@ -204,10 +208,15 @@ def try_attention_precise(qkv, q_stride, batch, block_tables, k_pages, v_pages, 
     check(block_tables, "block_tables", torch.int32)
     if sinks is not None:
         check(sinks, "sinks", torch.float32, n_q_heads)
+    if bias_log2 is not None:
+        check(bias_log2, "distance bias", torch.float32)
+        if bias_log2.dim() != 2 or bias_log2.shape[0] != n_q_heads:
+            raise ValueError(f"the distance bias must be [{n_q_heads}, distances], got {tuple(bias_log2.shape)}")
     # the cp.async decode kernel keeps two tiles in flight per block: three blocks an SM (its shared memory allows them)
     # and splits without the cluster's bound keep more bytes in flight
     run_portions, tiles, run_decode, split_len, max_splits = plan(batch, n_q_heads // n_kv_heads, n_kv_heads, qkv.device,
-                                                                  blocks_per_sm=PRECISE_DECODE_BLOCKS_PER_SM, cluster=False)
+                                                                  blocks_per_sm=PRECISE_DECODE_BLOCKS_PER_SM, cluster=False,
+                                                                  span=int(chunk) or None)
     out = torch.empty((batch.n_tokens, n_q_heads * value_dim), dtype=torch.bfloat16, device=qkv.device)
     partial_out = partial_ml = None
     if run_decode and max_splits > 1:
@@ -219,7 +228,7 @@ def try_attention_precise(qkv, q_stride, batch, block_tables, k_pages, v_pages, 
             batch.scratch[key] = scratch
         partial_out, partial_ml = scratch
     page_size = k_pages.shape[2]
-    if run_portions and value_dim == head_dim and PRECISE_PREFILL_KERNEL == "tcgen05" and \
+    if run_portions and value_dim == head_dim and PRECISE_PREFILL_KERNEL == "tcgen05" and not chunk and bias_log2 is None and \
             prefill_tcgen05_supported(head_dim, n_q_heads, n_kv_heads, page_size):
         # prompt portions on the 128-row tcgen05 kernel in its form with two-part weights; single tokens, if any, below
         group = n_q_heads // n_kv_heads
@@ -241,7 +250,8 @@ def try_attention_precise(qkv, q_stride, batch, block_tables, k_pages, v_pages, 
     call("llm_attention_mma_sinks", qkv.data_ptr(), q_stride, k_pages.data_ptr(), v_pages.data_ptr(), block_tables.data_ptr(),
          block_tables.shape[-1], batch.q_start.data_ptr(), batch.context_len.data_ptr(), out.data_ptr(), batch.n_seqs,
          n_q_heads, n_kv_heads, head_dim, value_dim, k_pages.shape[2], k_pages.shape[0], float(scale), int(window),
-         0 if sinks is None else sinks.data_ptr(), int(run_portions), tiles, int(run_decode), split_len, max_splits,
+         0 if sinks is None else sinks.data_ptr(), int(chunk), 0 if bias_log2 is None else bias_log2.data_ptr(),
+         0 if bias_log2 is None else bias_log2.shape[1], int(run_portions), tiles, int(run_decode), split_len, max_splits,
          0 if partial_out is None else partial_out.data_ptr(), 0 if partial_ml is None else partial_ml.data_ptr(),
          wait_error_flag(qkv.device).data_ptr(), stream_handle())
     return out

@@ -3,14 +3,32 @@ positions and a sliding window."""
 from __future__ import annotations
 
 import functools
+import math
 
 import torch
 
 from .. import ops
-from ..cache.manager import KVPagesNeed
+from ..cache.manager import KVPagesNeed, StateNeed
 from ..weights.declare import NORM, WIDE, WeightDecl
 from .base import Mixer
 from .registry import MIXERS
+
+
+def distance_buckets(count: int, largest: float, distances: int) -> list:
+    """The bucket of each distance 0 .. distances - 1 among ``count`` buckets: with half = count / 2, distance n < half has a
+    bucket of its own, and farther ones share buckets whose borders grow geometrically up to ``largest``,
+
+        half + floor(ln(n / half) / ln(largest / half) * (count - half)),  at most count - 1."""
+    half = count // 2
+    if count < 2 or largest <= half:
+        raise ValueError(f"{count} buckets need a largest distance above {half}, got {largest}")
+    found = []
+    for n in range(distances):
+        if n < half:
+            found.append(n)
+        else:
+            found.append(min(count - 1, half + int(math.floor(math.log(n / half) / math.log(largest / half) * (count - half)))))
+    return found
 
 
 @MIXERS.register("gqa_attention")
@@ -32,8 +50,14 @@ class GQAttention(Mixer):
     projection, a head's key as projected (and normalised and rotated, where the layer does that) is also its value; the
     cache then keeps keys alone.  ``unit_sink`` (bool): every softmax denominator holds one more 1 (a sink whose score is
     0, without a learned number).  ``query_temperature`` = (coef, every): the query at position p is multiplied by
-    1 + coef * ln(floor((p + 1) / every) + 1).  ``names``: pairs (role, tensor name behind the prefix) for checkpoints that call the
-    tensors otherwise; roles are q, k, v, o, q_norm, k_norm, sinks.
+    1 + coef * ln(floor((p + 1) / every) + 1).  ``conv`` (taps): q, k and v pass a causal convolution over time per channel
+    right behind their projections (weights: the projection's name with ".conv" added, [channels, taps], the last column
+    the current token's); the last taps - 1 projected rows of every request are kept in its state slot.  ``qk_norm``
+    "projection": one RMS norm over all of q and one over all of k, weights as long as they, in place of the norms per
+    head.  ``chunk``: a query at position p reads keys floor(p / chunk) * chunk .. p.  ``distance_bias`` = (buckets, largest):
+    a learned number per head and bucket of the distance between query and key (``rel`` [buckets, heads]; see
+    ``distance_buckets``; buckets None: as many as the tensor has rows) is added to the scaled score.  ``names``: pairs (role, tensor name behind the prefix) for checkpoints that call the
+    tensors otherwise; roles are q, k, v, o, q_norm, k_norm, sinks, rel.
 
     How positions are encoded comes from the position encoding the layer names (``attach``): its inverse
     frequencies, how many elements of a head rotate (``rotary_dim``, at most head_dim) and how they pair
@@ -43,9 +67,10 @@ class GQAttention(Mixer):
     such heads go through the kernel for heads made of units (pairing "halves" only)."""
 
     KNOWN_PARAMS = ("hidden", "heads", "kv_heads", "head_dim", "scale", "qk_norm", "eps", "window", "bias", "softcap",
-                    "value_dim", "sinks", "names", "precise_weights", "values_are_keys", "unit_sink", "query_temperature")
+                    "value_dim", "sinks", "names", "precise_weights", "values_are_keys", "unit_sink", "query_temperature",
+                    "conv", "chunk", "distance_bias")
     NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
-             "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "sinks": "sinks"}
+             "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "sinks": "sinks", "rel": "rel"}
 
     @classmethod
     def names(cls, params) -> dict:
@@ -69,6 +94,20 @@ class GQAttention(Mixer):
         temperature = params.get("query_temperature")
         if temperature and (len(temperature) != 2 or int(temperature[1]) <= 0):
             raise ValueError("gqa_attention: query_temperature is (coef, every) with a positive period")
+        if params.get("qk_norm") not in (None, True, False, "projection"):
+            raise ValueError(f"gqa_attention: qk_norm is a truth value or 'projection', not {params['qk_norm']!r}")
+        if cls.by_rows(params) and (params.get("values_are_keys") or params.get("query_temperature")):
+            raise ValueError("gqa_attention: convolutions and norms over whole projections come with a value projection and "
+                             "without a query temperature")
+        if params.get("chunk") and (int(params["chunk"]) <= 0 or params.get("window")):
+            raise ValueError("gqa_attention: keys are bounded by a window or by chunks of a positive size, not by both")
+        if params.get("distance_bias") and params["distance_bias"][0] is not None:
+            distance_buckets(int(params["distance_bias"][0]), float(params["distance_bias"][1]), 1)
+
+    @classmethod
+    def by_rows(cls, params) -> bool:
+        """Whether whole rows of the projection are convolved or normalised before they become heads."""
+        return bool(params.get("conv")) or params.get("qk_norm") == "projection"
 
     @classmethod
     def declare_weights(cls, params):
@@ -82,8 +121,14 @@ class GQAttention(Mixer):
         if params.get("values_are_keys"):
             del wanted[name["v"]]
         if params.get("qk_norm"):
-            wanted[name["q_norm"]] = WeightDecl((dim,), NORM)
-            wanted[name["k_norm"]] = WeightDecl((dim,), NORM)
+            whole = params["qk_norm"] == "projection"
+            wanted[name["q_norm"]] = WeightDecl((heads * dim if whole else dim,), NORM)
+            wanted[name["k_norm"]] = WeightDecl((kv_heads * dim if whole else dim,), NORM)
+        if params.get("conv"):
+            for role in ("q", "k", "v"):
+                wanted[name[role] + ".conv"] = WeightDecl((wanted[name[role]].shape[0], int(params["conv"])), WIDE)
+        if params.get("distance_bias"):
+            wanted[name["rel"]] = WeightDecl((int(params["distance_bias"][0]) if params["distance_bias"][0] else -1, heads), WIDE)
         if params.get("sinks"):
             wanted[name["sinks"]] = WeightDecl((heads,), WIDE)
         return wanted
@@ -92,8 +137,14 @@ class GQAttention(Mixer):
     def cache_need(cls, params):
         if params.get("values_are_keys"):
             return KVPagesNeed(int(params["kv_heads"]), int(params["head_dim"]), params.get("window"), None, keys_only=True)
-        return KVPagesNeed(int(params["kv_heads"]), int(params["head_dim"]), params.get("window"),
-                           int(params["value_dim"]) if params.get("value_dim") else None)
+        pages = KVPagesNeed(int(params["kv_heads"]), int(params["head_dim"]), params.get("window"),
+                            int(params["value_dim"]) if params.get("value_dim") else None,
+                            chunk=int(params["chunk"]) if params.get("chunk") else None)
+        if int(params.get("conv") or 1) == 1:
+            return pages
+        kv_heads, dim = int(params["kv_heads"]), int(params["head_dim"])
+        channels = (int(params["heads"]) + kv_heads) * dim + kv_heads * int(params.get("value_dim") or dim)
+        return (pages, StateNeed((int(params["conv"]) - 1, channels), "float32"))
 
     def __init__(self, params, weights, runtime):
         super().__init__(params, weights, runtime)
@@ -120,12 +171,31 @@ class GQAttention(Mixer):
         # keys that are their own values and queries with a temperature go through the kernel for heads made of units
         self.by_units = self.values_are_keys or self.temperature is not None
         self.inv_freq, self.rotary_dim, self.interleaved, self.magnitude = None, self.head_dim, False, 1.0
+        self.rows_first = self.by_rows(params)
+        self.taps = None
+        if params.get("conv"):
+            self.taps = torch.cat([weights[name[role] + ".conv"].to(torch.float32) for role in ("q", "k", "v")], dim=0).t().contiguous()
+        self.chunk = int(params.get("chunk") or 0)
+        self.bias = self.bias_log2 = None
+        if params.get("distance_bias"):
+            # the table by distance, made once: a chunk or the window bounds the distances, and from the largest one on
+            # every distance falls into the last bucket
+            table = weights[name["rel"]].to(torch.float32)
+            count, largest = table.shape[0], float(params["distance_bias"][1])
+            reach = math.ceil(largest) + 1
+            for bound in (self.chunk, self.window):
+                reach = min(reach, bound) if bound else reach
+            buckets = torch.tensor(distance_buckets(count, largest, reach), dtype=torch.long, device=table.device)
+            self.bias = table[buckets].t().contiguous()
+            self.bias_log2 = (self.bias * ops.LOG2E).contiguous()
 
     def attach(self, position):
         """``position``: None (no rotation) or an encoding with ``inv_freq`` (float32 [rotary_dim / 2] on the device)
         and, optionally, ``rotary_dim``, ``pairing`` ("halves" | "interleaved") and ``attention_factor``."""
         if position is None:
             return
+        if self.rows_first:
+            raise ValueError("gqa_attention: the kernel that convolves and normalises whole projections does not rotate heads")
         inv_freq = getattr(position, "inv_freq", None)
         if inv_freq is None:
             raise ValueError(f"gqa_attention rotates queries and keys: the position encoding {type(position).__name__} "
@@ -154,9 +224,18 @@ class GQAttention(Mixer):
 
     @functools.cached_property
     def takes_unscaled(self):
-        return not self.split and not self.by_units and ops.unscaled_rows_supported(self.qkv)
+        return not self.split and not self.by_units and not self.rows_first and ops.unscaled_rows_supported(self.qkv)
 
     def forward(self, x, batch, cache, sink=None):
+        if self.rows_first:
+            pages, history = cache, None
+            if cache.parts:
+                pages, history = cache.parts[0], cache.parts[1].state
+            tables = batch.block_tables[pages.group]
+            queries = ops.conv_norm_kv(ops.linear(x, self.qkv), self.taps, history, batch, tables, pages.k_pages, pages.v_pages,
+                                       self.heads, self.kv_heads, self.head_dim, self.value_dim, self.q_norm, self.k_norm, self.eps,
+                                       write_cache=pages.writes)
+            return ops.linear(self._attend(queries, batch, tables, pages, queries.shape[1]), self.out, sink=sink)
         tables = batch.block_tables[cache.group]
         if self.by_units:
             # one unit per head: norms, temperature, rotation and the cache write in one kernel; without a value projection
@@ -169,10 +248,7 @@ class GQAttention(Mixer):
                                 q_weight=self.q_norm, k_weight=self.k_norm, eps=self.eps, inv_freq=self.inv_freq,
                                 rotary_dim=rotating, write_cache=cache.writes, interleaved=self.interleaved,
                                 q_temp=self.temperature)
-            attended = ops.attention(qkv, batch, tables, cache.k_pages, cache.v_pages, self.heads, self.kv_heads, self.head_dim,
-                                     self.scale, self.window, value_dim=self.value_dim, sinks=self.sinks,
-                                     precise=bool(self.params.get("precise_weights")), q_stride=qkv.shape[1])
-            return ops.linear(attended, self.out, sink=sink)
+            return ops.linear(self._attend(qkv, batch, tables, cache, qkv.shape[1]), self.out, sink=sink)
         if self.split and self.q_norm is not None:
             # heads with a norm whose values have another size than their keys: the kernel for heads made of units, one
             # unit per head
@@ -191,7 +267,10 @@ class GQAttention(Mixer):
             qkv = ops.qkv_projection(x, self.qkv, self.q_norm, self.k_norm, self.inv_freq, batch.positions, batch.seq_of_token,
                                      tables, cache.k_pages, cache.v_pages, self.heads, self.kv_heads, self.head_dim, self.eps,
                                      cache.writes, batch.error_flag, self.rotary_dim, self.interleaved)
-        attended = ops.attention(qkv, batch, tables, cache.k_pages, cache.v_pages, self.heads, self.kv_heads,
-                                 self.head_dim, self.scale, self.window, value_dim=self.value_dim, sinks=self.sinks,
-                                 precise=bool(self.params.get("precise_weights")))
-        return ops.linear(attended, self.out, sink=sink)
+        return ops.linear(self._attend(qkv, batch, tables, cache), self.out, sink=sink)
+
+    def _attend(self, queries, batch, tables, pages, q_stride=None):
+        return ops.attention(queries, batch, tables, pages.k_pages, pages.v_pages, self.heads, self.kv_heads, self.head_dim,
+                             self.scale, self.window, value_dim=self.value_dim, sinks=self.sinks,
+                             precise=bool(self.params.get("precise_weights")), q_stride=q_stride, chunk=self.chunk, bias=self.bias,
+                             bias_log2=self.bias_log2)

@@ -1,4 +1,4 @@
-"""Dense feed-forwards: SwiGLU, a gated layer with clamped values, and a layer without a gate."""
+"""Dense feed-forwards: SwiGLU, the gated layer with gelu, one with clamped values, and a layer without a gate."""
 from __future__ import annotations
 
 import functools
@@ -52,6 +52,36 @@ class SwiGLU(FeedForward):
 
     def forward(self, x, sink=None):
         return ops.linear(ops.gate_up_silu(x, self.gate_up, self.group), self.down, sink=sink)
+
+
+@FEED_FORWARDS.register("gelu_glu")
+class GeluGLU(FeedForward):
+    """A dense gated feed-forward: y = W_down (gelu(W_gate x) * (W_up x)), gelu in its tanh form, no biases.  Parameters:
+    ``hidden``, ``intermediate``; ``names``: pairs (role, tensor name behind the prefix) for the roles gate, up and down.
+    gate and up are one [2 I, H] matrix, gate rows first; the activation is formed in 32-bit and rounded once."""
+
+    KNOWN_PARAMS = ("hidden", "intermediate", "names")
+    NAMES = {"gate": "gate", "up": "up", "down": "down"}
+
+    @classmethod
+    def names(cls, params) -> dict:
+        return {**cls.NAMES, **dict(params.get("names") or ())}
+
+    @classmethod
+    def declare_weights(cls, params):
+        hidden, intermediate = int(params["hidden"]), int(params["intermediate"])
+        name = cls.names(params)
+        return {name["gate"]: WeightDecl((intermediate, hidden)), name["up"]: WeightDecl((intermediate, hidden)),
+                name["down"]: WeightDecl((hidden, intermediate))}
+
+    def __init__(self, params, weights, runtime):
+        super().__init__(params, weights, runtime)
+        name = self.names(params)
+        self.gate_up = torch.cat([weights[name["gate"]], weights[name["up"]]], dim=0).contiguous()
+        self.down = weights[name["down"]].contiguous()
+
+    def forward(self, x):
+        return ops.linear(ops.gelu_mul(ops.linear(x, self.gate_up)), self.down)
 
 
 @FEED_FORWARDS.register("clamped_glu")

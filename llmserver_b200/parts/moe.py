@@ -25,14 +25,19 @@ class RoutedExperts(FeedForward):
     into its expert instead of what comes out, y = sum_e expert_e(w_e * x): the pair's row is scaled as the first product
     reads it, and the experts' outputs are summed as they are.
 
+    ``scores`` "softmax": s = softmax(z) over all experts.  ``groups`` = (count, keep): the experts form ``count`` equal groups
+    of neighbours and only those of the ``keep`` best groups can be chosen, a group's score being the largest in it.
+    ``renormalise``: the chosen experts' weights are divided by their sum (+ 1e-20).  ``shared_gate``: the shared expert's
+    output is multiplied by sigmoid(W_sg x), one number per token; W_sg is one more row of the router's product.
+
     Parameters: ``hidden``, ``experts``, ``top``, ``intermediate``, ``limit``, ``route_scale``; ``alpha`` (default
     1.702); ``correction`` (default True: the router has one); ``shared_intermediate`` and ``shared_limit`` (absent: no
     shared expert).  Tensors behind the part's prefix: ``e<i>.gate``, ``e<i>.up`` [intermediate, hidden], ``e<i>.down``
     [hidden, intermediate], ``router`` [experts, hidden], ``correction`` [experts], ``shared.gate`` / ``.up`` /
-    ``.down``.  Router and correction are held in float32 in either path."""
+    ``.down``, ``shared.sg`` [1, hidden].  Router and correction are held in float32 in either path."""
 
     KNOWN_PARAMS = ("hidden", "experts", "top", "intermediate", "limit", "route_scale", "alpha", "correction",
-                    "shared_intermediate", "shared_limit", "activation", "weight_on")
+                    "shared_intermediate", "shared_limit", "activation", "weight_on", "scores", "groups", "renormalise", "shared_gate")
     ACTIVATIONS = ("clamped_swish", "silu")
 
     @classmethod
@@ -43,12 +48,22 @@ class RoutedExperts(FeedForward):
         activation = params.get("activation", "clamped_swish")
         if activation not in cls.ACTIVATIONS:
             raise ValueError(f"routed_experts: unknown activation {activation!r} (known: {', '.join(cls.ACTIVATIONS)})")
-        if activation == "silu" and (params.get("limit") is not None or params.get("alpha") is not None or params.get("shared_intermediate")):
-            raise ValueError("routed_experts: the plain silu activation takes no limit or alpha, and has no shared expert")
+        if activation == "silu" and (params.get("limit") is not None or params.get("alpha") is not None or params.get("shared_limit") is not None):
+            raise ValueError("routed_experts: the plain silu activation takes no limit or alpha")
         if activation != "silu" and params.get("limit") is None:
             raise ValueError("routed_experts: the clamped activation needs its limit")
         if params.get("weight_on", "output") not in ("output", "input"):
             raise ValueError(f"routed_experts: weight_on is 'output' or 'input', not {params.get('weight_on')!r}")
+        if params.get("scores", "sigmoid") not in ("sigmoid", "softmax"):
+            raise ValueError(f"routed_experts: scores are 'sigmoid' or 'softmax', not {params.get('scores')!r}")
+        if params.get("groups"):
+            count, keep = (int(value) for value in params["groups"])
+            if count <= 0 or int(params["experts"]) % count or not 0 < keep <= count:
+                raise ValueError(f"routed_experts: {params['experts']} experts do not form {count} equal groups of which {keep} are kept")
+            if int(params["top"]) > keep * (int(params["experts"]) // count):
+                raise ValueError(f"routed_experts: {keep} groups hold fewer than top {params['top']} experts")
+        if params.get("shared_gate") and not params.get("shared_intermediate"):
+            raise ValueError("routed_experts: a gate on the shared expert needs a shared expert")
 
     @classmethod
     def declare_weights(cls, params):
@@ -66,6 +81,8 @@ class RoutedExperts(FeedForward):
             wanted["shared.gate"] = WeightDecl((shared, hidden))
             wanted["shared.up"] = WeightDecl((shared, hidden))
             wanted["shared.down"] = WeightDecl((hidden, shared))
+            if params.get("shared_gate"):
+                wanted["shared.sg"] = WeightDecl((1, hidden), WIDE)
         return wanted
 
     def __init__(self, params, weights, runtime):
@@ -84,6 +101,10 @@ class RoutedExperts(FeedForward):
                                     for e in range(self.experts)]).contiguous()
         self.down = torch.stack([weights[f"e{e}.down"] for e in range(self.experts)]).contiguous()
         self.router = weights["router"].to(torch.float32).contiguous()
+        self.rule = {"scores": params.get("scores", "sigmoid"), "groups": tuple(params["groups"]) if params.get("groups") else None,
+                     "renormalise": bool(params.get("renormalise")), "gate": bool(params.get("shared_gate"))}
+        if self.rule["gate"]:
+            self.router = torch.cat([self.router, weights["shared.sg"].to(torch.float32)], dim=0).contiguous()
         # A router whose weights are bfloat16 numbers (what a bfloat16 checkpoint holds) can be multiplied on the tensor
         # cores without leaving 32-bit arithmetic: products of two bfloat16 numbers are exact in 32-bit, and the sums
         # are 32-bit.  Any other router, and the 32-bit path, use the FMA kernel that makes the choice as well.
@@ -91,8 +112,13 @@ class RoutedExperts(FeedForward):
         self.router_narrow = narrow.contiguous() if runtime.dtype == torch.bfloat16 and bool((narrow.float() == self.router).all()) else None
         self.correction = weights["correction"].to(torch.float32).contiguous() if params.get("correction", True) else None
         self.shared_gate_up = self.shared_down = None
+        self.shared_group = 0
         if params.get("shared_intermediate"):
-            self.shared_gate_up = torch.cat([weights["shared.gate"], weights["shared.up"]], dim=0).contiguous()
+            gate, up = weights["shared.gate"], weights["shared.up"]
+            # a plain silu layer in bfloat16: rows interleaved so that the product kernel for few rows applies the gate itself
+            if params.get("activation") == "silu" and gate.dtype == torch.bfloat16 and gate.shape[0] % ops.GATE_UP_GROUP == 0:
+                self.shared_group = ops.GATE_UP_GROUP
+            self.shared_gate_up = ops.interleave_gate_up(gate, up) if self.shared_group else torch.cat([gate, up], dim=0).contiguous()
             self.shared_down = weights["shared.down"].contiguous()
             self.shared_limit = float(params.get("shared_limit", self.limit))
 
@@ -108,11 +134,14 @@ class RoutedExperts(FeedForward):
         tokens = x.shape[0]
         if self.router_narrow is not None:
             logits = ops.linear_wide(x, self.router_narrow)
-            chosen, weights = ops.moe_select(logits, self.correction, self.top, self.route_scale)
+            chosen, weights, *gate = ops.moe_select(logits, self.correction, self.top, self.route_scale, **self.rule)
         else:
-            chosen, weights = ops.moe_route(x, self.router, self.correction, self.top, self.route_scale)
+            chosen, weights, *gate = ops.moe_route(x, self.router, self.correction, self.top, self.route_scale, **self.rule)
+        shared_gate = gate[0] if gate else None
         shared = None
-        if self.shared_gate_up is not None:
+        if self.shared_gate_up is not None and self.params.get("activation") == "silu":
+            shared = ops.linear(ops.gate_up_silu(x, self.shared_gate_up, self.shared_group), self.shared_down)
+        elif self.shared_gate_up is not None:
             shared = ops.linear(ops.clamped_glu(ops.linear(x, self.shared_gate_up), self.shared_limit, self.alpha),
                                 self.shared_down)
         on_input = weights.view(-1) if self.weight_on_input else None
@@ -122,12 +151,12 @@ class RoutedExperts(FeedForward):
             plan = ops.moe_plan(chosen, self.experts)
             hidden = ops.moe_grouped(x, self.gate_up, plan, gather_div=self.top, gated=self.gate, pair_scale=on_input)
             down = ops.moe_grouped(hidden, self.down, plan)
-            return ops.moe_combine_rows(down, plan, weights, shared, self.runtime.dtype)
+            return ops.moe_combine_rows(down, plan, weights, shared, self.runtime.dtype, shared_gate)
         pairs = tokens * self.top
         index = chosen.view(-1)
         hidden = ops.indexed_linear(x, self.gate_up, index, pairs, in_div=self.top, gated=self.gate, in_scale=on_input)
         down = ops.indexed_linear(hidden, self.down, index, pairs, out_dtype=torch.float32)
-        return ops.moe_combine(down, weights, shared, self.runtime.dtype)
+        return ops.moe_combine(down, weights, shared, self.runtime.dtype, shared_gate)
 
     def _ones(self, like):
         """Unit weights of ``like``'s shape (kept: a step's shapes repeat, and a captured step must not allocate anew)."""

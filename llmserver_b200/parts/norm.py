@@ -50,20 +50,24 @@ class RMSNorm(Norm):
     (1 + weight); no bias.  Parameters: ``width``, ``eps``; ``tensor``: the weight's name behind the part's prefix
     (default "weight"; "" when the prefix is the whole name); ``one_plus`` (default False): the tensor holds the weight's
     distance from one, y = (1 + w) * x / rms: the sum is made once, in 32-bit, when the model is built (in bfloat16 it
-    would round the small w away), and the kernels read that 32-bit weight.  Fused with the residual add that precedes
+    would round the small w away), and the kernels read that 32-bit weight.  ``scalar`` (default False): the tensor is one
+    number for all coordinates, laid out as a weight when the model is built.  Fused with the residual add that precedes
     it, as the reference's add_rms_norm (utils/fused_ops.py:145-155)."""
 
-    KNOWN_PARAMS = ("width", "eps", "tensor", "one_plus")
+    KNOWN_PARAMS = ("width", "eps", "tensor", "one_plus", "scalar")
 
     @classmethod
     def declare_weights(cls, params):
-        return {params.get("tensor", "weight"): WeightDecl((params["width"],), OFFSET if params.get("one_plus") else NORM)}
+        shape = () if params.get("scalar") else (params["width"],)
+        return {params.get("tensor", "weight"): WeightDecl(shape, OFFSET if params.get("one_plus") else NORM)}
 
     def __init__(self, params, weights, runtime):
         super().__init__(params, weights, runtime)
         self.weight = weights[params.get("tensor", "weight")].contiguous()
         if params.get("one_plus"):
             self.weight = (self.weight.to(torch.float32) + 1.0).contiguous()
+        if params.get("scalar"):
+            self.weight = self.weight.to(torch.float32).expand(int(params["width"])).contiguous()
         self.eps = float(params["eps"])
 
     def add_norm(self, residual, delta, rows=None, unscaled=False):
