@@ -618,3 +618,108 @@ def zeridra_step_cost(size: dict, layers: int, tokens: int, sequences: int, cont
         total_bytes += 2.0 * weights
         flops += 2.0 * tokens * weights
     return total_bytes, flops
+
+
+# ---------------------------------------------------------------------------------------------------------------------
+# Dozotar beside the closest design of each of its layers at equal size: Gefarax for attention with routed experts (the
+# same heads, the same experts with a shared one), Dikusun's gated linear attention for the two recurrences (as many
+# cells of state and value channels, a dense gated feed-forward)
+# ---------------------------------------------------------------------------------------------------------------------
+def _dozotar_mixers(width, heads, kv_heads):
+    """Mixers of one width: attention with heads of 128 in chunks of 2048 positions (a prompt of 2048 tokens is causal), a
+    bias over 32 buckets and convolutions of 4 taps; retention with keys half as wide as the stream and values as wide;
+    the state-space form with twice the stream's width in heads of 64, a state of 128 and one group."""
+    return (dict(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, conv=4, scale=128 ** -0.5, bias_max=128, buckets=32,
+                 mask={"size": 2048}),
+            dict(heads=width // 128, dim=64, vdim=128, decay=[1.0 - 2.0 ** -(5.0 + 4.0 * h / (width // 128)) for h in range(width // 128)],
+                 rot={"base": 10000.0, "dims": 64}),
+            dict(heads=width // 32, vdim=64, state=128, groups=1, conv=4, norm_groups=1))
+
+
+# Layer sizes that resemble served models: four layers of one kind of mixer, or attention, state space, retention, state
+# space.  Attention layers and the mix have routed experts with a shared one, the recurrences alone a dense feed-forward
+# three times as wide as the stream.
+DOZOTAR_SIZES = {}
+for _width, _heads, _kv, _experts, _top, _ff in ((2048, 16, 4, 32, 4, 768), (4096, 32, 8, 64, 6, 1792)):
+    _a, _r, _s = _dozotar_mixers(_width, _heads, _kv)
+    for _label, _kinds in (("attention", ("attention",) * 4), ("retention", ("retention",) * 4), ("mamba2", ("mamba2",) * 4),
+                           ("mixed", ("attention", "mamba2", "retention", "mamba2"))):
+        DOZOTAR_SIZES[f"w{_width}-{_label}"] = dict(width=_width, attention=_a, retention=_r, mamba2=_s, experts=_experts, top=_top,
+                                                    ff=_ff, shared_ff=2 * _ff, groups=8, keep=4, dense_ff=3 * _width,
+                                                    moe=_label in ("attention", "mixed"), kinds=_kinds)
+
+
+def _dozotar_kinds(size: dict, layers: int):
+    return [size["kinds"][index % len(size["kinds"])] for index in range(layers)]
+
+
+def dozotar_config(size: dict, layers: int = None):
+    from llmserver_b200.config import DozotarConfig
+    mlp = {"kind": "dense", "ff": size["dense_ff"]}
+    if size["moe"]:
+        mlp = {"kind": "moe", "router": {"experts": size["experts"], "top": size["top"],
+                                         "groups": {"count": size["groups"], "keep": size["keep"]}},
+               "expert": {"ff": size["ff"]}, "shared": {"ff": size["shared_ff"]}}
+    return DozotarConfig.from_dict({"architecture": "Dozotar", "vocab": COMPARE_VOCAB, "width": size["width"], "norm": {"eps": 1e-6},
+                                    "layers": [{"type": kind, "mixer": size[kind], "mlp": mlp}
+                                               for kind in _dozotar_kinds(size, layers or len(size["kinds"]))]})
+
+
+def dozotar_twin(size: dict, layers: int):
+    """(label, size, configuration, cost function) of the closest design at equal size; None for a mix of kinds."""
+    kinds = set(size["kinds"])
+    if len(kinds) > 1:
+        return None
+    width = size["width"]
+    if kinds == {"attention"}:
+        a = size["attention"]
+        twin = _gefarax_size(width, a["heads"], a["kv_heads"], a["dim"], a["vdim"], size["experts"], size["top"], size["ff"], size["shared_ff"])
+
+        def cost(sizes, layers, tokens, sequences, context):
+            per_sequence = tokens / sequences
+            pairs = sequences * (per_sequence * context + per_sequence * (per_sequence + 1) / 2)
+            return gefarax_step_cost(sizes, layers, tokens, sequences * (context + per_sequence), pairs)
+
+        return "gefarax", twin, gefarax_config(twin, layers), cost
+    gla = dict(heads=width // 128, dim=64, vdim=128, tau=8.0, a_rank=32)
+    if kinds == {"mamba2"}:
+        gla = dict(heads=width // 64, dim=128, vdim=128, tau=8.0, a_rank=32)
+    twin = _dikusun_size(width, size["dense_ff"], None, None, gla, ("gla",) * len(size["kinds"]))
+    return "dikusun", twin, dikusun_config(twin, layers), dikusun_step_cost
+
+
+def dozotar_step_cost(size: dict, layers: int, tokens: int, sequences: int, context: float):
+    """(bytes, FLOPs) of one step in which each of ``sequences`` requests brings tokens / sequences new tokens behind
+    ``context`` cached ones: bytes = every weight the step touches once (of the routed experts the expected number of
+    distinct ones its tokens choose) + the chunk's cached rows + the states read and written; FLOPs = the products of the
+    tokens + attention per (query, key) pair + the recurrences' multiply-adds (a decay, a write and a read per cell)."""
+    width, experts, top, ff, shared = size["width"], size["experts"], size["top"], size["ff"], size["shared_ff"]
+    per_sequence = tokens / sequences
+    total_bytes = COMPARE_VOCAB * width * 2.0
+    flops = 0.0
+    distinct = experts * (1.0 - (1.0 - top / experts) ** tokens)
+    for kind in _dozotar_kinds(size, layers):
+        m = size[kind]
+        if size["moe"]:
+            total_bytes += 2.0 * 3 * width * (distinct * ff + shared) + 2.0 * (experts + 1) * width
+            flops += 2.0 * tokens * (3 * width * (top * ff + shared) + (experts + 1) * width)
+        else:
+            total_bytes += 2.0 * 3 * width * size["dense_ff"]
+            flops += 2.0 * tokens * 3 * width * size["dense_ff"]
+        if kind == "attention":
+            heads, kv, dim, vdim, chunk = m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["mask"]["size"]
+            weights = (heads * dim + kv * dim + kv * vdim) * width + width * heads * vdim
+            total_bytes += sequences * ((context + per_sequence - 1) % chunk + 1) * kv * (dim + vdim) * 2.0
+            pairs = sequences * sum((context + i) % chunk + 1 for i in range(int(per_sequence)))
+            flops += 2.0 * heads * (dim + vdim) * pairs
+        else:
+            heads, dim, vdim = m["heads"], m.get("dim", m.get("state")), m["vdim"]
+            if kind == "retention":
+                weights = (2 * heads * dim + 2 * heads * vdim) * width + width * heads * vdim
+            else:
+                weights = (2 * heads * vdim + 2 * m["groups"] * dim + heads) * width + width * heads * vdim
+            total_bytes += sequences * heads * dim * vdim * 4.0 * 2
+            flops += tokens * heads * dim * vdim * 5.0
+        total_bytes += 2.0 * weights
+        flops += 2.0 * tokens * weights
+    return total_bytes, flops

@@ -43,6 +43,8 @@ constexpr uint32_t kQBytes = kRows * kDim * 2;        // 32 KiB
 constexpr uint32_t kKVBytes = kKeys * kDim * 2;       // 16 KiB per K or V tile
 constexpr uint32_t kColS0 = 0, kColS1 = 64, kColO = 128, kTmemCols = 256;
 
+// The form with a bias by distance gives one K stage up for the group's rows of the bias.
+constexpr uint32_t kBiasBytes = kKVBytes;
 constexpr uint32_t kTileBytes = kQBytes + (kKStages + kVStages) * kKVBytes;   // 112 KiB
 constexpr uint32_t kControlBytes = 256;
 constexpr uint32_t kSharedBytes = 113 * 1024;
@@ -69,7 +71,27 @@ struct PrefillParams {
     int pairing;
     int* error_flag;
     const float* sinks;  // [Hq] or null: exp(sinks[h]) joins head h's softmax denominator (no key, no value, not scaled)
+    int chunk = 0;                  // > 0: the query at position p sees keys (p / chunk) * chunk .. p only
+    const float* bias = nullptr;    // BIAS: [Hq, bias_len], times log2(e): added to the score of the key n positions back, n at
+    int bias_len = 0;               // most bias_len - 1 (farther keys: the last entry)
+    int bias_stride = 0;            // floats between two heads' staged rows
 };
+
+// The first key that the query at `position` may see.
+__device__ __forceinline__ int first_visible(const PrefillParams& p, int position) {
+    int low = p.window > 0 ? max(0, position - p.window + 1) : 0;
+    if (p.chunk > 0) low = max(low, position / p.chunk * p.chunk);
+    return low;
+}
+
+// BIAS: a head's staged row holds kKeys zeros, its bias_len distances and kKeys copies of the last one, so that a thread
+// reads the 64 distances of a tile without looking at each: those in front of distance 0 belong to masked keys.
+__host__ __device__ constexpr int bias_row_floats(int bias_len) { return bias_len + 2 * kKeys; }
+// Heads of a group lie so far apart that the 32 rows of a warp (token, head of the group) read different banks.
+inline int bias_row_stride(int bias_len, int group) {
+    const int apart = (32 + group - 1) / group % 32;
+    return (bias_row_floats(bias_len) + 31) / 32 * 32 + apart;
+}
 
 using tma::mbar_arrive;
 using tma::mbar_expect_tx;
@@ -83,7 +105,7 @@ using namespace tc5;
 // S_b and the rounding of what that left over in the other 32 (the softmax thread holds all 64 scores of its row in
 // registers by then, so S_b's own columns are free), and the P V product is two MMAs per 16 keys: 16 significant bits
 // for models whose attention weights have to stay 32-bit.
-template <bool PRECISE>
+template <bool PRECISE, bool BIAS = false>
 __global__ void __launch_bounds__(kThreads, 2) attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q,
                                                                              const __grid_constant__ CUtensorMap map_k,
                                                                              const __grid_constant__ CUtensorMap map_v,
@@ -100,7 +122,9 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_tcgen05_kernel(
         if (threadIdx.x == 0 && p.error_flag) atomicExch(p.error_flag, 5);
         return;
     }
-    const uint32_t q_smem = base, k_smem = base + kQBytes, v_smem = k_smem + kKStages * kKVBytes;
+    constexpr int KS = BIAS ? kKStages - 1 : kKStages;
+    const uint32_t q_smem = base, k_smem = base + kQBytes, v_smem = k_smem + KS * kKVBytes;
+    float* bias_shared = reinterpret_cast<float*>(shared_raw + (v_smem + kVStages * kKVBytes - raw));
     Control& control = *reinterpret_cast<Control*>(shared_raw + (kSharedBytes - kControlBytes));
     uint64_t& q_full = control.q_full;
     uint64_t (&k_full)[kKStages] = control.k_full;
@@ -140,6 +164,13 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_tcgen05_kernel(
     const int* table = p.block_tables + (size_t)seq * p.max_blocks;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
+    if (BIAS) {
+        const int row_floats = bias_row_floats(p.bias_len);
+        for (int e = threadIdx.x; e < group * row_floats; e += kThreads) {
+            const int h = e / row_floats, n = e % row_floats - kKeys;
+            bias_shared[h * p.bias_stride + n + kKeys] = n < 0 ? 0.0f : p.bias[(size_t)(kv_head * group + h) * p.bias_len + min(n, p.bias_len - 1)];
+        }
+    }
     if (threadIdx.x == 0) failed = 0;
     if (warp == 5) {
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_slot)), "r"(kTmemCols));
@@ -154,8 +185,7 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_tcgen05_kernel(
     const int tile = pass == 0 ? first_tile : second_tile;
     const int first_token = tile * tokens_per_tile;
     const int high_key = base_position + min(first_token + tokens_per_tile, q_len) - 1;
-    int low_key = 0;
-    if (p.window > 0) low_key = max(0, base_position + first_token - p.window + 1);
+    const int low_key = first_visible(p, base_position + first_token);
     const int first_tile_key = (low_key / kKeys) * kKeys;
     const int n_tiles = (high_key - first_tile_key) / kKeys + 1;
 
@@ -195,8 +225,8 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_tcgen05_kernel(
         for (int step = 0; step < n_tiles + 2; ++step) {
             bool ok = true;
             if (step < n_tiles) {
-                const int t = step, s = t % kKStages;
-                if (t >= kKStages) ok = mbar_wait(smem_u32(&k_free[s]), ((t / kKStages) - 1) & 1);
+                const int t = step, s = t % KS;
+                if (t >= KS) ok = mbar_wait(smem_u32(&k_free[s]), ((t / KS) - 1) & 1);
                 if (ok) {
                     if (lane == 0) mbar_expect_tx(smem_u32(&k_full[s]), kKVBytes);
                     __syncwarp();
@@ -238,8 +268,8 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_tcgen05_kernel(
             bool ok = mbar_wait(smem_u32(&q_full), 0);
             for (int j = 0; j <= n_tiles && ok; ++j) {
                 if (j < n_tiles) {        // S_b = Q K_j^T
-                    const int s = j % kKStages, b = j & 1;
-                    ok = mbar_wait(smem_u32(&k_full[s]), (j / kKStages) & 1);
+                    const int s = j % KS, b = j & 1;
+                    ok = mbar_wait(smem_u32(&k_full[s]), (j / KS) & 1);
                     if (!ok) break;
                     fence_after();
 #pragma unroll
@@ -279,7 +309,8 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_tcgen05_kernel(
         const int token = first_token + row / group, head = kv_head * group + row % group;
         const bool exists = row < tokens_per_tile * group && token < q_len;
         const int position = exists ? base_position + token : -1;
-        const int low = (exists && p.window > 0) ? max(0, position - p.window + 1) : 0;
+        const int low = exists ? first_visible(p, position) : 0;
+        const float* bias_row = BIAS ? bias_shared + (row % group) * p.bias_stride + kKeys : nullptr;      // distance 0 of this row's head
         const uint32_t lane_base = tmem + ((uint32_t)(warp * 32) << 16);
         float reference = -INFINITY;     // what is subtracted in the exponent (a stale maximum)
         float row_sum = 0.0f;
@@ -292,6 +323,19 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_tcgen05_kernel(
             uint32_t raw[64];
             tmem_load_64(s_address, raw);
             const int tile_key = first_tile_key + j * kKeys;
+            if (BIAS) {      // scores leave here as they enter the exponent: scaled, with their bias, times log2(e)
+                const int back = position - tile_key;      // distance of the tile's first key; its last one is kKeys - 1 nearer
+                if (back - (kKeys - 1) >= p.bias_len - 1) {      // the whole tile lies beyond the last distance
+                    const float far = bias_row[p.bias_len - 1];
+#pragma unroll
+                    for (int c = 0; c < 64; ++c) raw[c] = __float_as_uint(fmaf(__uint_as_float(raw[c]), p.scale_log2, far));
+                } else {
+                    // rows that see nothing of this tile (and rows that do not exist) read their head's first entries
+                    const float* at = bias_row + max(back, -1);
+#pragma unroll
+                    for (int c = 0; c < 64; ++c) raw[c] = __float_as_uint(fmaf(__uint_as_float(raw[c]), p.scale_log2, at[-c]));
+                }
+            }
             // only tiles that touch the diagonal, the window's edge or the end of the rows need the mask
             if (tile_key + kKeys - 1 > position || tile_key < low) {
 #pragma unroll
@@ -310,7 +354,7 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_tcgen05_kernel(
 #pragma unroll
             for (int c = 4; c < 32; ++c) running[c & 3] = max3(running[c & 3], __uint_as_float(raw[2 * c]), __uint_as_float(raw[2 * c + 1]));
             const float raw_max = fmaxf(fmaxf(running[0], running[1]), fmaxf(running[2], running[3]));
-            const float tile_max = raw_max * p.scale_log2;
+            const float tile_max = BIAS ? raw_max : raw_max * p.scale_log2;
             // the reference moves only when the maximum has outgrown it by the threshold (or nothing was seen yet)
             float factor = 1.0f;
             if (tile_max > reference + kRescaleThreshold || (reference == -INFINITY && tile_max > -INFINITY)) {
@@ -318,7 +362,7 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_tcgen05_kernel(
                 reference = tile_max;
             }
             const float subtract = reference == -INFINITY ? 0.0f : reference;
-            const uint64_t scale_pair = pair_of(p.scale_log2, p.scale_log2), minus_pair = pair_of(-subtract, -subtract);
+            const uint64_t scale_pair = BIAS ? pair_of(1.0f, 1.0f) : pair_of(p.scale_log2, p.scale_log2), minus_pair = pair_of(-subtract, -subtract);
             float weight[64];
 #pragma unroll
             for (int c = 0; c < 32; ++c)
@@ -426,13 +470,20 @@ LLM_EXPORT int llm_attention_prefill_tcgen05_supports(int head_dim, int n_q_head
     return page_size == 8 || page_size == 16 || page_size == 32 || page_size == 64;
 }
 
+// Whether the rows of a bias over `bias_len` distances fit beside the tiles for groups of `group` heads.
+LLM_EXPORT int llm_attention_prefill_tcgen05_bias_fits(int bias_len, int group) {
+    return bias_len > 0 && bias_len < 65536 && group > 0 &&
+           (size_t)group * bias_row_stride(bias_len, group) * sizeof(float) <= kBiasBytes;
+}
+
 // total_pairs: the number of CTAs: with pairing, the sum over the sequences it handles of ceil(ceil(q_len * group / 128) / 2)
 // (each CTA takes a row tile and its mirror, which evens out the work of a causal prompt); without, one CTA per tile; sequences of one token are skipped when skip_single is set (the decode kernel takes them).
 static int launch_prefill_tcgen05(const void* q, int q_stride, int n_tokens, const void* k_pages, const void* v_pages,
                                   const int* block_tables, int max_blocks, const int* q_start,
                                   const int* context_len, void* out, int n_seqs, int n_q_heads, int n_kv_heads,
                                   int head_dim, int page_size, int num_pages, float scale, int window, int skip_single, int pairing,
-                                  int total_pairs, int* error_flag, const float* sinks, bool precise, cudaStream_t stream) {
+                                  int total_pairs, int* error_flag, const float* sinks, bool precise, int chunk, const float* bias,
+                                  int bias_len, cudaStream_t stream) {
     if (total_pairs <= 0) return LLM_OK;
     if (num_pages <= 0) {
         llm_set_error("attention_prefill_tcgen05: the page pool has %d pages", num_pages);
@@ -478,9 +529,21 @@ static int launch_prefill_tcgen05(const void* q, int q_stride, int n_tokens, con
     p.pairing = pairing;
     p.error_flag = error_flag;
     p.sinks = sinks;
+    p.chunk = chunk;
+    p.bias = bias;
+    p.bias_len = bias_len;
+    if (chunk < 0 || (bias && (!precise || !llm_attention_prefill_tcgen05_bias_fits(bias_len, group)))) {
+        llm_set_error("attention_prefill_tcgen05: chunks of %d positions or a bias of %d distances for groups of %d heads are not supported",
+                      chunk, bias_len, group);
+        return LLM_REFUSED;
+    }
+    p.bias_stride = bias ? bias_row_stride(bias_len, group) : 0;
     const size_t shared = kSharedBytes;
     dim3 grid(total_pairs, n_kv_heads);
-    if (precise) {
+    if (bias) {
+        if (int limit_status = llm_raise_shared_limit(reinterpret_cast<const void*>(attention_prefill_tcgen05_kernel<true, true>), shared, "attention_prefill_tcgen05", true)) return limit_status;
+        llm_launch(attention_prefill_tcgen05_kernel<true, true>, grid, kThreads, shared, stream, map_q, map_k, map_v, p);
+    } else if (precise) {
         if (int limit_status = llm_raise_shared_limit(reinterpret_cast<const void*>(attention_prefill_tcgen05_kernel<true>), shared, "attention_prefill_tcgen05", true)) return limit_status;
         llm_launch(attention_prefill_tcgen05_kernel<true>, grid, kThreads, shared, stream, map_q, map_k, map_v, p);
     } else {
@@ -497,18 +560,21 @@ LLM_EXPORT int llm_attention_prefill_tcgen05(const void* q, int q_stride, int n_
                                              int total_pairs, int* error_flag, cudaStream_t stream) {
     return launch_prefill_tcgen05(q, q_stride, n_tokens, k_pages, v_pages, block_tables, max_blocks, q_start, context_len, out, n_seqs,
                                   n_q_heads, n_kv_heads, head_dim, page_size, num_pages, scale, window, skip_single, pairing,
-                                  total_pairs, error_flag, nullptr, false, stream);
+                                  total_pairs, error_flag, nullptr, false, 0, nullptr, 0, stream);
 }
 
 // The same with attention weights of 16 significant bits in the P V product and, with `sinks` (float32 [Hq], may be
-// null), one more term exp(sinks[h]) in every row's softmax denominator.
+// null), one more term exp(sinks[h]) in every row's softmax denominator.  `chunk` > 0: a query sees the keys of its own
+// chunk of positions only.  `bias` (float32 [Hq, bias_len], given times log2(e); may be null): what is added to the score
+// of the key n positions back, at min(n, bias_len - 1).
 LLM_EXPORT int llm_attention_prefill_tcgen05_precise(const void* q, int q_stride, int n_tokens, const void* k_pages, const void* v_pages,
                                                      const int* block_tables, int max_blocks, const int* q_start,
                                                      const int* context_len, void* out, int n_seqs, int n_q_heads, int n_kv_heads,
                                                      int head_dim, int page_size, int num_pages, float scale, int window,
                                                      int skip_single, int pairing, int total_pairs, int* error_flag,
-                                                     const float* sinks, cudaStream_t stream) {
+                                                     const float* sinks, int chunk, const float* bias, int bias_len,
+                                                     cudaStream_t stream) {
     return launch_prefill_tcgen05(q, q_stride, n_tokens, k_pages, v_pages, block_tables, max_blocks, q_start, context_len, out, n_seqs,
                                   n_q_heads, n_kv_heads, head_dim, page_size, num_pages, scale, window, skip_single, pairing,
-                                  total_pairs, error_flag, sinks, true, stream);
+                                  total_pairs, error_flag, sinks, true, chunk, bias, bias_len, stream);
 }

@@ -228,7 +228,8 @@ def try_attention_precise(qkv, q_stride, batch, block_tables, k_pages, v_pages, 
             batch.scratch[key] = scratch
         partial_out, partial_ml = scratch
     page_size = k_pages.shape[2]
-    if run_portions and value_dim == head_dim and PRECISE_PREFILL_KERNEL == "tcgen05" and not chunk and bias_log2 is None and \
+    if run_portions and value_dim == head_dim and PRECISE_PREFILL_KERNEL == "tcgen05" and \
+            (bias_log2 is None or library().llm_attention_prefill_tcgen05_bias_fits(bias_log2.shape[1], n_q_heads // n_kv_heads)) and \
             prefill_tcgen05_supported(head_dim, n_q_heads, n_kv_heads, page_size):
         # prompt portions on the 128-row tcgen05 kernel in its form with two-part weights; single tokens, if any, below
         group = n_q_heads // n_kv_heads
@@ -243,7 +244,8 @@ def try_attention_precise(qkv, q_stride, batch, block_tables, k_pages, v_pages, 
              block_tables.data_ptr(), block_tables.shape[-1], batch.q_start.data_ptr(), batch.context_len.data_ptr(),
              out.data_ptr(), batch.n_seqs, n_q_heads, n_kv_heads, head_dim, page_size, k_pages.shape[0], float(scale), int(window),
              int(run_decode), int(pairing), paired if pairing else sum(tile_counts), wait_error_flag(qkv.device).data_ptr(),
-             0 if sinks is None else sinks.data_ptr(), stream_handle())
+             0 if sinks is None else sinks.data_ptr(), int(chunk), 0 if bias_log2 is None else bias_log2.data_ptr(),
+             0 if bias_log2 is None else bias_log2.shape[1], stream_handle())
         run_portions = False
         if not run_decode:
             return out

@@ -62,7 +62,8 @@ SIGNATURES = {
     "llm_attention_mma_sinks": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _P, _P, _P, _S],
     "llm_attention_prefill_tcgen05_supports": [_I, _I, _I, _I],
     "llm_attention_prefill_tcgen05": [_P, _I, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _I, _P, _S],
-    "llm_attention_prefill_tcgen05_precise": [_P, _I, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _I, _P, _P, _S],
+    "llm_attention_prefill_tcgen05_bias_fits": [_I, _I],
+    "llm_attention_prefill_tcgen05_precise": [_P, _I, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _I, _P, _P, _I, _P, _I, _S],
     "llm_attention_prefill_wide_supports": [_I, _I, _I, _I],
     "llm_attention_prefill_wide": [_P, _I, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _I, _P, _S],
     "llm_gemm_small_m_supports": [_I, _I, _I],
