@@ -138,6 +138,18 @@ __device__ __forceinline__ void store8(T* p, const float (&v)[8]) {
     }
 }
 
+// Eight elements as they lie in memory: fetched (through the read-only path) well before they are widened, so that
+// several are in flight at a time.
+template <typename T>
+struct Raw8 {
+    uint4 words[sizeof(T) / 2];
+    __device__ __forceinline__ void fetch(const T* p) {
+#pragma unroll
+        for (int i = 0; i < (int)(sizeof(T) / 2); ++i) words[i] = __ldg(reinterpret_cast<const uint4*>(p) + i);
+    }
+    __device__ __forceinline__ void widen(float (&v)[8]) const { load8<T>(reinterpret_cast<const T*>(words), v); }
+};
+
 __host__ __device__ __forceinline__ bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
 
 __device__ __forceinline__ float warp_sum(float v) {

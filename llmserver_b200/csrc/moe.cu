@@ -142,10 +142,10 @@ __global__ void moe_route_kernel(const T* __restrict__ x, const float* __restric
     choose_experts(score, choice, rule, correction, chosen + (size_t)token * rule.top, weights + (size_t)token * rule.top, counts);
 }
 
-// The choice alone, from router logits that a matrix product has made: z float32 [N, experts (+ 1 for the gate)].  One
-// warp per token.
+// The choice alone, from router logits that a matrix product has made: z float32, `stride` numbers per token, the experts'
+// first and then the gate's.  One warp per token.
 __global__ void moe_select_kernel(const float* __restrict__ logits, const float* __restrict__ correction, int* __restrict__ chosen,
-                                  float* __restrict__ weights, int n_tokens, RouteRule rule, float* __restrict__ gate_out) {
+                                  float* __restrict__ weights, int n_tokens, RouteRule rule, int stride, float* __restrict__ gate_out) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float select_shared[];      // per warp: [experts] scores, [experts] choice scores
@@ -153,7 +153,7 @@ __global__ void moe_select_kernel(const float* __restrict__ logits, const float*
     const int token = blockIdx.x * warps + warp;
     if (token >= n_tokens) return;
     float* score = select_shared + (size_t)warp * 2 * rule.experts;
-    const float* z = logits + (size_t)token * (rule.experts + (gate_out ? 1 : 0));
+    const float* z = logits + (size_t)token * stride;
     for (int e = lane; e < rule.experts; e += 32) score[e] = z[e];
     if (gate_out && lane == 0) gate_out[token] = 1.0f / (1.0f + expf(-z[rule.experts]));
     __syncwarp();
@@ -322,11 +322,15 @@ LLM_EXPORT int llm_moe_route(const void* x, const float* router, const float* co
 }
 
 LLM_EXPORT int llm_moe_select(const float* logits, const float* correction, int* chosen, float* weights, int n_tokens,
-                              int experts, int top, float scale, int softmax, int groups, int keep, int renormalise, float* gate_out,
-                              cudaStream_t stream) {
+                              int experts, int top, float scale, int softmax, int groups, int keep, int renormalise, int stride,
+                              float* gate_out, cudaStream_t stream) {
     if (n_tokens == 0) return LLM_OK;
     const RouteRule rule = {experts, top, softmax, groups, keep, renormalise, scale};
     if (const int refused = check_rule("moe_select", rule)) return refused;
+    if (stride < experts + (gate_out ? 1 : 0)) {
+        llm_set_error("moe_select: %d numbers per token for %d experts", stride, experts);
+        return LLM_REFUSED;
+    }
     const int warps = 4;
     const size_t shared = (size_t)warps * 2 * experts * sizeof(float);
     if (shared > 40 * 1024) {
@@ -334,7 +338,7 @@ LLM_EXPORT int llm_moe_select(const float* logits, const float* correction, int*
         return LLM_REFUSED;
     }
     llm_launch(moe_select_kernel, (n_tokens + warps - 1) / warps, warps * 32, shared, stream, logits, correction, chosen, weights,
-               n_tokens, rule, gate_out);
+               n_tokens, rule, stride, gate_out);
     return llm_check_launch("moe_select");
 }
 

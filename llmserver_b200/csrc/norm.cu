@@ -515,6 +515,42 @@ __global__ void grouped_rmsnorm_block_kernel(const float* __restrict__ x, const 
     for (int c = threadIdx.x; c < size; c += blockDim.x) Num<T>::store(dst + c, src[c] * inverse * Num<W>::load(w + c));
 }
 
+// The same with 16-byte accesses and the piece held in registers between the passes (sizes that are a multiple of 8, up to
+// blockDim * 32).
+template <typename T, typename W>
+__global__ void grouped_rmsnorm_vec_kernel(const float* __restrict__ x, const W* __restrict__ weight, T* __restrict__ out, int parts,
+                                           int size, float eps) {
+    pdl_trigger();
+    pdl_wait();
+    __shared__ float scratch[33];
+    const int part = blockIdx.x % parts, chunks = size / kChunk;
+    const float* src = x + (size_t)blockIdx.x * size;
+    const W* w = weight + (size_t)part * size;
+    T* dst = out + (size_t)blockIdx.x * size;
+    float values[kMaxChunks][kChunk], squares = 0.0f;
+#pragma unroll
+    for (int i = 0; i < kMaxChunks; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        if (c < chunks) {
+            load8<float>(src + c * kChunk, values[i]);
+#pragma unroll
+            for (int j = 0; j < kChunk; ++j) squares = fmaf(values[i][j], values[i][j], squares);
+        }
+    }
+    const float inverse = rsqrtf(block_sum(squares, scratch) / (float)size + eps);
+#pragma unroll
+    for (int i = 0; i < kMaxChunks; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        if (c < chunks) {
+            float scale[kChunk];
+            load8<W>(w + c * kChunk, scale);
+#pragma unroll
+            for (int j = 0; j < kChunk; ++j) scale[j] = values[i][j] * inverse * scale[j];
+            store8<T>(dst + c * kChunk, scale);
+        }
+    }
+}
+
 LLM_EXPORT int llm_grouped_rmsnorm(const float* x, const void* weight, void* out, int n_rows, int parts, int size, float eps, int dtype,
                                    int weight_dtype, cudaStream_t stream) {
     if (n_rows == 0) return LLM_OK;
@@ -522,7 +558,15 @@ LLM_EXPORT int llm_grouped_rmsnorm(const float* x, const void* weight, void* out
         llm_set_error("grouped_rmsnorm: %d pieces of %d elements must both be positive", parts, size);
         return LLM_REFUSED;
     }
-    if (size > 1024) {      // the choice depends on the piece's size only, so a row's result does not depend on the batch
+    // the choices depend on the piece's size only, so a row's result does not depend on the batch
+    if (size > 1024 && size % kChunk == 0 && size <= 512 * kChunk * kMaxChunks && aligned16(x) && aligned16(weight) && aligned16(out)) {
+        int threads = (size / kChunk + 31) / 32 * 32;
+        if (threads > 512) threads = 512;
+        LLM_DISPATCH_DTYPE_WEIGHT(dtype, weight_dtype, (llm_launch(grouped_rmsnorm_vec_kernel<T, W>, (unsigned)n_rows * parts, threads, 0, stream,
+                                                                   x, (const W*)weight, (T*)out, parts, size, eps)));
+        return llm_check_launch("grouped_rmsnorm");
+    }
+    if (size > 1024) {
         LLM_DISPATCH_DTYPE_WEIGHT(dtype, weight_dtype, (llm_launch(grouped_rmsnorm_block_kernel<T, W>, (unsigned)n_rows * parts, 256, 0, stream,
                                                                    x, (const W*)weight, (T*)out, parts, size, eps)));
         return llm_check_launch("grouped_rmsnorm");

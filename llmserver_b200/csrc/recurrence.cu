@@ -17,12 +17,6 @@
 //       delta   S <- g_t S;  d = beta_t (v_t - S^T k_t);  S <- S + k_t d^T;  o_t = S^T q_t
 //               g_t = exp(-exp(A) softplus(a_t + dt)),  beta_t = sigmoid(b_t)
 //     followed by out = o / sqrt(mean(o^2) + eps) * weight * silu(gate).
-//     Two more share one plain form, a single decay per head and token (`llm_retention_recurrent`, `llm_ssd_recurrent`):
-//       S <- g_t S + k_t v_t^T;  o_t = S_t^T q_t
-//       retention   g a constant of the head, q and k rotated by the token's position, k scaled, as they are staged;
-//                   followed by out = o / sqrt(mean(o^2) + eps) * silu(gate)
-//       ssd         (Dao and Gu, "Transformers are SSMs") g_t = exp(-exp(A) dt_t), dt_t = softplus(z_t + bias), q = C_t and
-//                   k = dt_t B_t shared by a group of heads, v = x_t; followed by out = (o + D x) * silu(gate), in 32-bit
 //
 // One block per (sequence, head).  A warp covers 32 / P value channels (columns of S) with P row partitions side by
 // side in its lanes; a thread owns R rows of one column in registers, so a sum over the rows is R multiply-adds and
@@ -31,9 +25,9 @@
 // and stored by one warp per token.  The order of every sum depends on the sizes alone, so a token's result does not
 // depend on how its prompt was cut or on what else is in the batch.
 //
-// Long portions can also be walked segment by segment in parallel (a segment length given to the launchers).  All the
+// Long portions can also be walked segment by segment in parallel (a segment length given to the launchers).  Both
 // recurrences are linear in S: behind a segment, S_out = M S_in + L, where L is what the segment leaves from a zero state
-// and M its transition: diag(prod_t w_t) for wkv; prod_t g_t for the two with one decay per head; for the delta rule the product of the g_t (I - beta_t k_t k_t^T), a
+// and M its transition: diag(prod_t w_t) for wkv; for the delta rule the product of the g_t (I - beta_t k_t k_t^T), a
 // dim x dim matrix, which the same walk yields column by column when it starts from the identity with values of zero.
 // Pass A runs every segment but the last from zero (delta: also `dim` more columns from the identity) and leaves L and M;
 // a scan gives every segment the state it starts from, S_in(k + 1) = M_k S_in(k) + L_k; pass C runs the segments again
@@ -152,6 +146,78 @@ __global__ void __launch_bounds__(256) short_conv_units_kernel(ConvArgs a) {
     }
 }
 
+// Plain channels alone (no unit vectors), in vectors of eight with a number of taps known at compile time: a thread walks
+// a vector's tokens with the inputs in its registers.  The thread that has a sequence's first tokens of a vector is the
+// only one that reads and renews the vector's stored inputs (CONV_ROLL tokens are more than any history it takes).
+#define CONV_ROLL 16
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128) short_conv_roll_kernel(ConvArgs a) {
+    pdl_trigger();
+    pdl_wait();
+    const int seq = blockIdx.z;
+    const int begin = a.q_start[seq], end = a.q_start[seq + 1];
+    const int first = begin + blockIdx.x * CONV_ROLL, last = min(end, first + CONV_ROLL);
+    const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8;
+    if (first >= end || c >= a.channels) return;
+    constexpr int history = TAPS - 1;
+    const T* x = (const T*)a.x + a.column + c;
+    float* state = a.state + (size_t)a.state_slots[seq] * history * a.channels + c;
+    float w[TAPS][8], v[TAPS][8], bias[8];      // v[j]: the input that tap j meets
+    {
+        float rows[8 * TAPS];      // the vector's weights lie one behind the other
+#pragma unroll
+        for (int i = 0; i < TAPS; ++i) load8<float>(a.taps_w + (size_t)c * TAPS + 8 * i, reinterpret_cast<float (&)[8]>(rows[8 * i]));
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) w[j][i] = rows[i * TAPS + j];
+            bias[i] = 0.0f;
+        }
+        if (a.bias) load8<float>(a.bias + c, bias);
+    }
+#pragma unroll
+    for (int j = 0; j < history; ++j) {
+        const int source = first - history + j;
+        if (source >= begin) load8<T>(x + (size_t)source * a.row_width, v[j + 1]);
+        else load8<float>(state + (size_t)(history + source - begin) * a.channels, v[j + 1]);
+    }
+    constexpr int FETCH = 4;
+    for (int t0 = first; t0 < last; t0 += FETCH) {
+        Raw8<T> raw[FETCH];
+#pragma unroll
+        for (int u = 0; u < FETCH; ++u) raw[u].fetch(x + (size_t)min(t0 + u, last - 1) * a.row_width);
+#pragma unroll
+        for (int u = 0; u < FETCH; ++u) {
+            if (t0 + u < last) {
+#pragma unroll
+                for (int j = 0; j < history; ++j)
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) v[j][i] = v[j + 1][i];
+                raw[u].widen(v[TAPS - 1]);
+                float y[8];
+#pragma unroll
+                for (int i = 0; i < 8; ++i) {
+                    float sum = bias[i];
+#pragma unroll
+                    for (int j = 0; j < TAPS; ++j) sum = fmaf(w[j][i], v[j][i], sum);
+                    y[i] = sizeof(T) == 2 ? __fdividef(sum, 1.0f + __expf(-sum)) : sum / (1.0f + expf(-sum));
+                }
+                store8<float>(a.out + (size_t)(t0 + u) * a.channels + c, y);
+            }
+        }
+    }
+    if (blockIdx.x != 0) return;
+    const int length = end - begin;
+#pragma unroll
+    for (int r = 0; r < history; ++r) {      // oldest first: a row is read before it is overwritten
+        const int source = length - history + r;
+        float kept[8];
+        if (source >= 0) load8<T>(x + (size_t)(begin + source) * a.row_width, kept);
+        else load8<float>(state + (size_t)(history + source) * a.channels, kept);
+        store8<float>(state + (size_t)r * a.channels, kept);
+    }
+}
+
 LLM_EXPORT int llm_short_conv_units(const void* x, int row_width, int column, const float* taps_w, int taps, float* state,
                                     const int* state_slots, const int* q_start, float* out, int n_seqs, int longest, int n_unit_norm,
                                     int unit_dim, int n_scaled, int n_plain, int plain_dim, float norm_eps, float scale,
@@ -176,6 +242,16 @@ LLM_EXPORT int llm_short_conv_units(const void* x, int row_width, int column, co
     a.channels = channels; a.bias = bias;
     a.n_unit_norm = n_unit_norm; a.unit_dim = unit_dim; a.n_scaled = n_scaled; a.n_plain = n_plain; a.plain_dim = plain_dim;
     a.norm_eps = norm_eps; a.scale = scale;
+    if (n_unit_norm == 0 && taps >= 2 && taps <= 4 && channels % 8 == 0 && column % 8 == 0 && row_width % 8 == 0 && aligned16(x) &&
+        aligned16(state) && aligned16(out) && aligned16(taps_w) && aligned16(bias)) {
+        const dim3 grid((longest + CONV_ROLL - 1) / CONV_ROLL, (channels / 8 + 127) / 128, n_seqs);
+        LLM_DISPATCH_DTYPE(dtype, {
+            if (taps == 2) llm_launch(short_conv_roll_kernel<T, 2>, grid, 128, 0, stream, a);
+            else if (taps == 3) llm_launch(short_conv_roll_kernel<T, 3>, grid, 128, 0, stream, a);
+            else llm_launch(short_conv_roll_kernel<T, 4>, grid, 128, 0, stream, a);
+        });
+        return llm_check_launch("short_conv_units");
+    }
     LLM_DISPATCH_DTYPE(dtype, (llm_launch(short_conv_units_kernel<T>, dim3(n_seqs, n_unit_norm + n_plain, (longest + CONV_CHUNK - 1) / CONV_CHUNK), 256, 0, stream, a)));
     return llm_check_launch("short_conv_units");
 }
@@ -188,23 +264,17 @@ struct RecArgs {
     // inputs in 32-bit
     const float* pre;       // delta: [N, pre_width] convolved q | k | v (q and k heads of `dim`, v heads of `vdim`)
     int pre_width, q_col, k_col, v_col, qk_heads;
-    const float* wide;      // wkv: z [N, heads * dim]; delta: [N, 2 heads] = b | a; ssd: [N, heads], dt before its bias
+    const float* wide;      // wkv: z [N, heads * dim]; delta: [N, 2 heads] = b | a
     const float* w0;        // wkv: [heads * dim]
     const float* bonus;     // wkv: u [heads, dim]
-    const float* a_log;     // delta, ssd: [heads]
-    const float* dt_bias;   // delta, ssd: [heads]
-    const float* head_decay;    // retention: [heads]
-    const float* skip;          // ssd: D [heads]
-    const int* positions;       // retention: [N]
-    const float* inv_freq;      // retention: [rotary_dim / 2]; null: nothing rotates
-    int rotary_dim;
-    float k_scale;              // retention: what a key is multiplied by behind its rotation
+    const float* a_log;     // delta: [heads]
+    const float* dt_bias;   // delta: [heads]
     const void* weight;     // norm weight, [vdim] (weight_stride 0) or [heads, vdim] (weight_stride vdim)
     int weight_stride;
     float* state;           // [slots, heads, dim, vdim]
     const int* state_slots;
     const int* q_start;
-    void* out;              // [N, heads * vdim] in the activation type; ssd: float32
+    void* out;              // [N, heads * vdim]
     int heads, dim, vdim, partitions, stride_rows;     // stride_rows: floats from one partition's staged rows to the next's
     float eps;
     // wkv: the row that the next step's token shift reads
@@ -215,16 +285,15 @@ struct RecArgs {
     int segment, max_segments;  // tokens per segment, segments the scratch has room for per sequence
     int groups;                 // delta, pass A: blocks per (segment, head): one for the value columns + those for the transition's
     float* segment_state;       // [S, max_segments, heads, dim, vdim]: pass A leaves L there, the scan S_in
-    float* segment_move;        // [S, max_segments, heads, dim], the products of the decays; delta: [.., heads, dim, dim]
+    float* segment_move;        // wkv: [S, max_segments, heads, dim], the products of the decays; delta: [.., heads, dim, dim]
 };
 
-enum : int { REC_WKV = 0, REC_DELTA = 1, REC_RETENTION = 2, REC_SSD = 3 };
+enum : int { REC_WKV = 0, REC_DELTA = 1 };
 // PASS 0: a sequence's tokens in one pass, from and into its state slot.  1: pass A of the segmented form.  3: pass C.
 enum : int { REC_ONE_PASS = 0, REC_LOCAL = 1, REC_OUTPUT = 3 };
 
 template <typename T, typename W, int R, int MODE, int PASS>
 __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) matrix_recurrence_kernel(RecArgs a) {
-    constexpr bool PLAIN = MODE == REC_RETENTION || MODE == REC_SSD;      // one decay per head and token
     pdl_trigger();
     pdl_wait();
     extern __shared__ float4 rec_shared_raw[];
@@ -254,7 +323,7 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) matrix_recurrence_kernel(
     float* w_s = k_s + REC_TOKENS * padded;            // wkv only: the decays
     float* v_s = w_s + (MODE == REC_WKV ? REC_TOKENS * padded : 0);     // [REC_TOKENS][vdim]
     float* o_s = v_s + REC_TOKENS * vdim;              // [REC_TOKENS][vdim]
-    float* scalar_s = o_s + REC_TOKENS * vdim;         // [REC_TOKENS][2]: wkv: the bonus term; delta: g and beta; else: g
+    float* scalar_s = o_s + REC_TOKENS * vdim;         // [REC_TOKENS][2]: wkv: the bonus term; delta: g and beta
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
     const int per_warp = 32 / P;                       // columns of S per warp
     const int part = lane / per_warp, column = warp * per_warp + lane % per_warp;
@@ -275,9 +344,8 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) matrix_recurrence_kernel(
         else S[i] = (owner && row0 + i < dim) ? source[(size_t)(row0 + i) * vdim + column] : 0.0f;
         if (PASS == REC_LOCAL && MODE == REC_WKV) decay[i] = 1.0f;
     }
-    float move = 1.0f;      // pass A with one decay per head: the product of the segment's decays
 
-    const int qk_head = MODE == REC_DELTA || MODE == REC_SSD ? head / (a.heads / a.qk_heads) : head;
+    const int qk_head = MODE == REC_DELTA ? head / (a.heads / a.qk_heads) : head;
     for (int first = begin; first < end; first += REC_TOKENS) {
         const int count = min(REC_TOKENS, end - first);
         __syncthreads();      // the staged values of the tokens before have been read
@@ -285,40 +353,7 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) matrix_recurrence_kernel(
         for (int t = warp; t < count; t += warps) {
             const size_t token = (size_t)(first + t);
             float bonus = 0.0f;
-            float dt = 0.0f;
-            if (MODE == REC_SSD) {
-                const float z = a.wide[token * a.heads + head] + a.dt_bias[head];
-                dt = z > 20.0f ? z : log1pf(expf(z));
-                if (lane == 0) scalar_s[2 * t] = expf(-expf(a.a_log[head]) * dt);
-            }
-            if (MODE == REC_RETENTION) {
-                if (lane == 0) scalar_s[2 * t] = a.head_decay[head];
-                const T* row = proj + token * a.row_width;
-                const T* q_row = row + a.r_offset + head * dim;
-                const T* k_row = row + a.k_offset + head * dim;
-                const int half = a.inv_freq ? a.rotary_dim >> 1 : 0;
-                const float position = (float)a.positions[token];
-                for (int i = lane; i < half; i += 32) {      // element i turns with element i + half
-                    float s, c;
-                    sincosf(position * a.inv_freq[i], &s, &c);
-                    const int at = t * padded + (i / R) * a.stride_rows + i % R;
-                    const int at2 = t * padded + ((i + half) / R) * a.stride_rows + (i + half) % R;
-                    const float ku = Num<T>::load(k_row + i), kv = Num<T>::load(k_row + i + half);
-                    k_s[at] = (ku * c - kv * s) * a.k_scale;
-                    k_s[at2] = (kv * c + ku * s) * a.k_scale;
-                    if (PASS != REC_LOCAL) {
-                        const float qu = Num<T>::load(q_row + i), qv = Num<T>::load(q_row + i + half);
-                        q_s[at] = qu * c - qv * s;
-                        q_s[at2] = qv * c + qu * s;
-                    }
-                }
-                for (int i = 2 * half + lane; i < P * R; i += 32) {
-                    const int at = t * padded + (i / R) * a.stride_rows + i % R;
-                    k_s[at] = i < dim ? Num<T>::load(k_row + i) * a.k_scale : 0.0f;
-                    q_s[at] = PASS != REC_LOCAL && i < dim ? Num<T>::load(q_row + i) : 0.0f;
-                }
-            }
-            for (int i = lane; i < (MODE == REC_RETENTION ? 0 : P * R); i += 32) {
+            for (int i = lane; i < P * R; i += 32) {
                 float qv = 0.0f, kv = 0.0f, wv = 0.0f;
                 if (i < dim) {
                     if (MODE == REC_WKV) {
@@ -332,7 +367,6 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) matrix_recurrence_kernel(
                     } else {
                         if (PASS != REC_LOCAL) qv = a.pre[token * a.pre_width + a.q_col + qk_head * dim + i];
                         kv = a.pre[token * a.pre_width + a.k_col + qk_head * dim + i];
-                        if (MODE == REC_SSD) kv *= dt;
                     }
                 }
                 const int at = t * padded + (i / R) * a.stride_rows + i % R;
@@ -342,12 +376,12 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) matrix_recurrence_kernel(
             }
             for (int j = lane; j < vdim; j += 32)
                 v_s[t * vdim + j] = group > 0 ? 0.0f
-                                    : MODE == REC_WKV || MODE == REC_RETENTION ? Num<T>::load(proj + token * a.row_width + a.v_offset + head * vdim + j)
+                                    : MODE == REC_WKV ? Num<T>::load(proj + token * a.row_width + a.v_offset + head * vdim + j)
                                                       : a.pre[token * a.pre_width + a.v_col + head * vdim + j];
             if (MODE == REC_WKV) {
                 bonus = warp_sum(bonus);
                 if (lane == 0) scalar_s[2 * t] = bonus;
-            } else if (MODE == REC_DELTA && lane == 0) {
+            } else if (lane == 0) {
                 const float b = a.wide[token * 2 * a.heads + head], z = a.wide[token * 2 * a.heads + a.heads + head] + a.dt_bias[head];
                 const float softplus = z > 20.0f ? z : log1pf(expf(z));
                 scalar_s[2 * t] = expf(-expf(a.a_log[head]) * softplus);
@@ -393,35 +427,6 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) matrix_recurrence_kernel(
                 }
                 for (int offset = per_warp; offset < 32; offset <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, offset);
                 o = fmaf(scalar_s[2 * t], vj, sum);
-            } else if (PLAIN) {
-                const float g = scalar_s[2 * t];
-                if (PASS == REC_LOCAL) {
-#pragma unroll
-                    for (int i = 0; i < R / 4; ++i) {
-                        const float4 kk = k4[i];
-                        S[4 * i + 0] = fmaf(g, S[4 * i + 0], kk.x * vj);
-                        S[4 * i + 1] = fmaf(g, S[4 * i + 1], kk.y * vj);
-                        S[4 * i + 2] = fmaf(g, S[4 * i + 2], kk.z * vj);
-                        S[4 * i + 3] = fmaf(g, S[4 * i + 3], kk.w * vj);
-                    }
-                    move *= g;
-                    continue;
-                }
-                float sum = 0.0f;
-#pragma unroll
-                for (int i = 0; i < R / 4; ++i) {
-                    const float4 qq = q4[i], kk = k4[i];
-                    S[4 * i + 0] = fmaf(g, S[4 * i + 0], kk.x * vj);
-                    S[4 * i + 1] = fmaf(g, S[4 * i + 1], kk.y * vj);
-                    S[4 * i + 2] = fmaf(g, S[4 * i + 2], kk.z * vj);
-                    S[4 * i + 3] = fmaf(g, S[4 * i + 3], kk.w * vj);
-                    sum = fmaf(S[4 * i + 0], qq.x, sum);
-                    sum = fmaf(S[4 * i + 1], qq.y, sum);
-                    sum = fmaf(S[4 * i + 2], qq.z, sum);
-                    sum = fmaf(S[4 * i + 3], qq.w, sum);
-                }
-                for (int offset = per_warp; offset < 32; offset <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, offset);
-                o = sum;
             } else {
                 const float g = scalar_s[2 * t], beta = scalar_s[2 * t + 1];
                 float read = 0.0f;
@@ -469,16 +474,6 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) matrix_recurrence_kernel(
         __syncthreads();
         // ---- head norm, gate, store: a warp per token
         for (int t = warp; t < count; t += warps) {
-            if (MODE == REC_SSD) {      // no norm yet: what is normalised together spans several heads
-                const T* g_row = proj + (size_t)(first + t) * a.row_width + a.g_offset + head * vdim;
-                float* dst = (float*)a.out + ((size_t)(first + t) * a.heads + head) * vdim;
-                const float skip = a.skip[head];
-                for (int j = lane; j < vdim; j += 32) {
-                    const float g = Num<T>::load(g_row + j);
-                    dst[j] = fmaf(skip, v_s[t * vdim + j], o_s[t * vdim + j]) * (g / (1.0f + expf(-g)));
-                }
-                continue;
-            }
             float squares = 0.0f;
             for (int j = lane; j < vdim; j += 32) squares = fmaf(o_s[t * vdim + j], o_s[t * vdim + j], squares);
             const float inverse = rsqrtf(warp_sum(squares) / (float)vdim + a.eps);
@@ -487,7 +482,7 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) matrix_recurrence_kernel(
             const W* weight = (const W*)a.weight + (size_t)head * a.weight_stride;
             for (int j = lane; j < vdim; j += 32) {
                 const float g = Num<T>::load(g_row + j);
-                Num<T>::store(dst + j, o_s[t * vdim + j] * inverse * (MODE == REC_RETENTION ? 1.0f : Num<W>::load(weight + j)) * (g / (1.0f + expf(-g))));
+                Num<T>::store(dst + j, o_s[t * vdim + j] * inverse * Num<W>::load(weight + j) * (g / (1.0f + expf(-g))));
             }
         }
     }
@@ -503,10 +498,10 @@ __global__ void __launch_bounds__(512, R <= 8 ? 2 : 1) matrix_recurrence_kernel(
             for (int i = 0; i < R; ++i)
                 if (row0 + i < dim) move[(size_t)(row0 + i) * dim + move_column] = S[i];
         }
-        if ((MODE == REC_WKV || PLAIN) && column == 0) {
+        if (MODE == REC_WKV && column == 0) {
 #pragma unroll
             for (int i = 0; i < R; ++i)
-                if (row0 + i < dim) a.segment_move[segment_index * dim + row0 + i] = PLAIN ? move : decay[i % (sizeof(decay) / sizeof(float))];
+                if (row0 + i < dim) a.segment_move[segment_index * dim + row0 + i] = decay[i % (sizeof(decay) / sizeof(float))];
         }
         return;
     }
@@ -800,7 +795,7 @@ static int rec_launch(RecArgs& a, int mode, int n_seqs, int dtype, int weight_dt
             REC_LAUNCH_PASS(R, MODE, REC_ONE_PASS, dim3(n_seqs, a.heads));                                                 \
         } else {                                                                                                           \
             REC_LAUNCH_PASS(R, MODE, REC_LOCAL, dim3(n_seqs, a.heads, a.max_segments * (MODE == REC_DELTA ? a.groups : 1))); \
-            if (MODE != REC_DELTA)                                                                                         \
+            if (MODE == REC_WKV)                                                                                           \
                 llm_launch(rec_scan_diagonal_kernel, dim3(n_seqs, a.heads, (a.dim * a.vdim + 255) / 256), 256, 0, stream, a); \
             else if (staged_scan) {                                                                                        \
                 const int status = rec_launch_staged_scan(a, n_seqs, stream);                                              \
@@ -820,9 +815,7 @@ static int rec_launch(RecArgs& a, int mode, int n_seqs, int dtype, int weight_dt
     } while (0)
     LLM_DISPATCH_DTYPE_WEIGHT(dtype, weight_dtype, {
         if (mode == REC_WKV) REC_LAUNCH_ROWS(REC_WKV);
-        else if (mode == REC_DELTA) REC_LAUNCH_ROWS(REC_DELTA);
-        else if (mode == REC_RETENTION) REC_LAUNCH_ROWS(REC_RETENTION);
-        else REC_LAUNCH_ROWS(REC_SSD);
+        else REC_LAUNCH_ROWS(REC_DELTA);
     });
 #undef REC_LAUNCH_ROWS
 #undef REC_LAUNCH
@@ -861,39 +854,4 @@ LLM_EXPORT int llm_delta_rule_recurrent(const void* proj, int row_width, int g_o
     a.weight_stride = 0; a.state = state; a.state_slots = state_slots; a.q_start = q_start; a.out = out; a.heads = heads;
     a.dim = dim; a.vdim = vdim; a.eps = eps;
     return rec_launch(a, REC_DELTA, n_seqs, dtype, weight_dtype, stream);
-}
-
-LLM_EXPORT int llm_retention_recurrent(const void* proj, int row_width, int q_offset, int k_offset, int v_offset, int g_offset,
-                                       const float* head_decay, const int* positions, const float* inv_freq, int rotary_dim,
-                                       float k_scale, float* state, const int* state_slots, const int* q_start, void* out, int n_seqs,
-                                       int heads, int dim, int vdim, float eps, int dtype, int segment, int max_segments,
-                                       float* segment_state, float* segment_move, cudaStream_t stream) {
-    if (inv_freq && (rotary_dim < 0 || rotary_dim % 2 || rotary_dim > dim)) {
-        llm_set_error("retention_recurrent: %d rotating elements must be an even number of at most %d", rotary_dim, dim);
-        return LLM_REFUSED;
-    }
-    RecArgs a = {};
-    a.segment = segment; a.max_segments = max_segments; a.segment_state = segment_state; a.segment_move = segment_move;
-    a.proj = proj; a.row_width = row_width; a.r_offset = q_offset; a.k_offset = k_offset; a.v_offset = v_offset; a.g_offset = g_offset;
-    a.head_decay = head_decay; a.positions = positions; a.inv_freq = inv_freq; a.rotary_dim = rotary_dim; a.k_scale = k_scale;
-    a.state = state; a.state_slots = state_slots; a.q_start = q_start; a.out = out; a.heads = heads; a.dim = dim; a.vdim = vdim;
-    a.eps = eps; a.qk_heads = heads;
-    return rec_launch(a, REC_RETENTION, n_seqs, dtype, dtype, stream);
-}
-
-LLM_EXPORT int llm_ssd_recurrent(const void* proj, int row_width, int g_offset, const float* pre, int pre_width, int v_col, int k_col,
-                                 int q_col, const float* wide, const float* a_log, const float* dt_bias, const float* skip,
-                                 float* state, const int* state_slots, const int* q_start, float* out, int n_seqs, int heads,
-                                 int groups, int dim, int vdim, int dtype, int segment, int max_segments, float* segment_state,
-                                 float* segment_move, cudaStream_t stream) {
-    if (groups <= 0 || heads % groups) {
-        llm_set_error("ssd_recurrent: %d heads are no multiple of %d groups", heads, groups);
-        return LLM_REFUSED;
-    }
-    RecArgs a = {};
-    a.segment = segment; a.max_segments = max_segments; a.segment_state = segment_state; a.segment_move = segment_move;
-    a.proj = proj; a.row_width = row_width; a.g_offset = g_offset; a.pre = pre; a.pre_width = pre_width; a.v_col = v_col;
-    a.k_col = k_col; a.q_col = q_col; a.qk_heads = groups; a.wide = wide; a.a_log = a_log; a.dt_bias = dt_bias; a.skip = skip;
-    a.state = state; a.state_slots = state_slots; a.q_start = q_start; a.out = out; a.heads = heads; a.dim = dim; a.vdim = vdim;
-    return rec_launch(a, REC_SSD, n_seqs, dtype, dtype, stream);
 }

@@ -22,7 +22,7 @@ __all__ = ["KernelError", "embedding", "add_rmsnorm", "rmsnorm", "silu_mul", "sa
            "clamped_glu", "gemm_f32", "linear", "linear_wide", "qkv_projection", "gate_up_silu", "interleave_gate_up", "require_device", "library", "launch_count",
            "RowScaled", "StreamSink", "STREAM_ROWS", "unscaled_rows_supported", "norm_rope_units", "rotate_units", "attention_diff", "gla_supported",
            "gla_recurrent", "head_linear", "relu_squared", "tanh_narrow", "softcap_", "scaled_sum", "token_shift_mix",
-           "short_conv_units", "matrix_recurrence_supported", "wkv_recurrent", "delta_rule_recurrent", "retention_recurrent", "ssd_recurrent",
+           "short_conv_units", "matrix_recurrence_supported", "wkv_recurrent", "delta_rule_recurrent", "retention_recurrent", "ssd_recurrent", "decay_recurrence_supported",
            "gelu_mul", "grouped_rmsnorm", "conv_norm_kv"]
 
 
@@ -787,6 +787,42 @@ def _check_matrix_state(state: torch.Tensor, heads: int, dim: int, value_dim: in
         raise KernelError(f"the state must be [slots, {heads}, {dim}, {value_dim}], got {tuple(state.shape)}")
 
 
+def decay_recurrence_supported(dim: int, value_dim: int) -> bool:
+    return library().llm_decay_recurrence_threads(int(dim), int(value_dim)) > 0
+
+
+def _decay_segments(batch, activations: torch.Tensor, segment: Optional[int], heads: int, dim: int, value_dim: int):
+    """Segment length, segments per sequence and the scratch of the segmented form of ``retention_recurrent`` and
+    ``ssd_recurrent``: a state [dim, value_dim] and a decay per (sequence, segment, head).  ``segment`` None: chosen here for
+    bfloat16 steps whose longest portion spans two segments, such that the long portions' segments fill the GPU about once
+    (an SM holds 512 threads of the kernel), each at least REC_SEGMENT tokens; 0: the one-pass form."""
+    longest = int(batch.max_q_len)
+    if segment is None:
+        segment = 0
+        if activations.dtype == torch.bfloat16 and longest >= 2 * REC_SEGMENT:
+            per_sm = max(1, 512 // library().llm_decay_recurrence_threads(dim, value_dim))
+            long_portions = sum(1 for length in batch.q_lens if length >= 2 * REC_SEGMENT) or 1
+            most = min(REC_MAX_SEGMENTS, REC_SCRATCH_BYTES // max(batch.n_seqs * heads * dim * value_dim * 4, 1),
+                       _sm_count(activations.device) * per_sm // (long_portions * heads))
+            if most >= 2:
+                segment = max(REC_SEGMENT, -(-longest // most))
+    if not segment:
+        return 0, 0, None, None
+    segments = -(-longest // int(segment))
+    key = ("decay_recurrence_segments", batch.n_seqs, segments, heads, dim, value_dim)
+    scratch = batch.scratch.get(key)
+    if scratch is None:
+        scratch = (torch.empty((batch.n_seqs, segments, heads, dim, value_dim), dtype=torch.float32, device=activations.device),
+                   torch.empty((batch.n_seqs, segments, heads), dtype=torch.float32, device=activations.device))
+        batch.scratch[key] = scratch
+    return int(segment), segments, scratch[0], scratch[1]
+
+
+def _sm_count(device) -> int:
+    from . import attention_bf16
+    return attention_bf16._sm_count(device)
+
+
 def retention_recurrent(proj: torch.Tensor, q_column: int, k_column: int, v_column: int, g_column: int, decay: torch.Tensor,
                         inv_freq: Optional[torch.Tensor], state: torch.Tensor, batch, heads: int, dim: int, value_dim: int,
                         k_scale: float, eps: float, segment: Optional[int] = None) -> torch.Tensor:
@@ -809,7 +845,7 @@ def retention_recurrent(proj: torch.Tensor, q_column: int, k_column: int, v_colu
         if column < 0 or column + size > row_width:
             raise KernelError(f"columns {column}..{column + size} lie outside a row of {row_width}")
     out = torch.empty((tokens, heads * value_dim), dtype=proj.dtype, device=proj.device)
-    segment, segments, segment_state, segment_move = _recurrence_segments(batch, proj, segment, heads, dim, value_dim, 1)
+    segment, segments, segment_state, segment_move = _decay_segments(batch, proj, segment, heads, dim, value_dim)
     call("llm_retention_recurrent", proj.data_ptr(), row_width, int(q_column), int(k_column), int(v_column), int(g_column),
          decay.data_ptr(), batch.positions.data_ptr(), pointer(inv_freq), 0 if inv_freq is None else 2 * inv_freq.numel(),
          float(k_scale), state.data_ptr(), batch.state_slots.data_ptr(), batch.q_start.data_ptr(), out.data_ptr(), batch.n_seqs,
@@ -845,7 +881,7 @@ def ssd_recurrent(proj: torch.Tensor, g_column: int, pre: torch.Tensor, v_column
     if pre.shape[0] != tokens or wide.shape[0] != tokens:
         raise KernelError("every input needs one row per token")
     out = torch.empty((tokens, heads * value_dim), dtype=torch.float32, device=proj.device)
-    segment, segments, segment_state, segment_move = _recurrence_segments(batch, proj, segment, heads, dim, value_dim, 1)
+    segment, segments, segment_state, segment_move = _decay_segments(batch, proj, segment, heads, dim, value_dim)
     call("llm_ssd_recurrent", proj.data_ptr(), row_width, int(g_column), pre.data_ptr(), pre.shape[1], int(v_column), int(k_column),
          int(q_column), wide.data_ptr(), a_log.data_ptr(), dt_bias.data_ptr(), skip.data_ptr(), state.data_ptr(),
          batch.state_slots.data_ptr(), batch.q_start.data_ptr(), out.data_ptr(), batch.n_seqs, int(heads), int(groups), int(dim),
@@ -913,12 +949,12 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, correction: Optional[torch.
 
 
 def moe_select(logits: torch.Tensor, correction: Optional[torch.Tensor], top: int, scale: float, scores: str = "sigmoid",
-               groups: Optional[tuple] = None, renormalise: bool = False, gate: bool = False):
-    """``moe_route``'s choice from router logits that a product has already made: logits float32 [N, E], or [N, E + 1] with
-    the ``gate``'s pre-activation last."""
+               groups: Optional[tuple] = None, renormalise: bool = False, gate: bool = False, experts: Optional[int] = None):
+    """``moe_route``'s choice from router logits that a product has already made: logits float32 [N, E], with ``gate``
+    [N, E + 1], the gate's pre-activation last.  ``experts``: E, where the product's rows are longer (padded)."""
     check(logits, "router logits", torch.float32)
-    tokens, experts = logits.shape
-    experts -= int(bool(gate))
+    tokens, stride = logits.shape
+    experts = stride - int(bool(gate)) if experts is None else int(experts)
     rule = _route_rule(experts, scores, groups, renormalise)
     if correction is not None:
         check(correction, "router correction", torch.float32, experts)
@@ -926,7 +962,7 @@ def moe_select(logits: torch.Tensor, correction: Optional[torch.Tensor], top: in
     weights = torch.empty((tokens, top), dtype=torch.float32, device=logits.device)
     gate_out = torch.empty((tokens,), dtype=torch.float32, device=logits.device) if gate else None
     call("llm_moe_select", logits.data_ptr(), pointer(correction), chosen.data_ptr(), weights.data_ptr(), tokens, experts,
-         int(top), float(scale), *rule, pointer(gate_out), stream_handle())
+         int(top), float(scale), *rule, stride, pointer(gate_out), stream_handle())
     return (chosen, weights, gate_out) if gate else (chosen, weights)
 
 

@@ -23,6 +23,7 @@ SIGNATURES = {
     "llm_gelu_mul": [_P, _P, _I, _I, _I, _I, _S],
     "llm_grouped_rmsnorm": [_P, _P, _P, _I, _I, _I, _F, _I, _I, _S],
     "llm_conv_norm_kv": [_P, _I, _P, _I, _P, _P, _P, _P, _P, _I, _P, _P, _F, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _I, _S],
+    "llm_decay_recurrence_threads": [_I, _I],
     "llm_retention_recurrent": [_P, _I, _I, _I, _I, _I, _P, _P, _P, _I, _F, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _I, _P, _P, _S],
     "llm_ssd_recurrent": [_P, _I, _I, _P, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P, _S],
     "llm_sample": [_P, _P, _P, _P, _P, _I, _I, _P, _P, _S],
@@ -45,7 +46,7 @@ SIGNATURES = {
     "llm_wkv_recurrent": [_P, _I, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _F, _P, _P, _I, _I, _I, _I, _I, _P, _P, _S],
     "llm_delta_rule_recurrent": [_P, _I, _I, _P, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _I, _P, _P, _S],
     "llm_moe_route": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _I, _I, _P, _I, _S],
-    "llm_moe_select": [_P, _P, _P, _P, _I, _I, _I, _F, _I, _I, _I, _I, _P, _S],
+    "llm_moe_select": [_P, _P, _P, _P, _I, _I, _I, _F, _I, _I, _I, _I, _I, _P, _S],
     "llm_indexed_linear": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _I, _I, _I, _P, _F, _S],
     "llm_moe_combine": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _S],
     "llm_clamped_glu": [_P, _P, _I, _I, _F, _F, _I, _S],

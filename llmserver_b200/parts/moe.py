@@ -109,7 +109,9 @@ class RoutedExperts(FeedForward):
         # cores without leaving 32-bit arithmetic: products of two bfloat16 numbers are exact in 32-bit, and the sums
         # are 32-bit.  Any other router, and the 32-bit path, use the FMA kernel that makes the choice as well.
         narrow = self.router.to(torch.bfloat16)
-        self.router_narrow = narrow.contiguous() if runtime.dtype == torch.bfloat16 and bool((narrow.float() == self.router).all()) else None
+        if narrow.shape[0] % 8:      # the library's products want rows of whole 16-byte pieces; the padding is never looked at
+            narrow = torch.cat([narrow, narrow.new_zeros((8 - narrow.shape[0] % 8, narrow.shape[1]))], dim=0)
+        self.router_narrow = narrow.contiguous() if runtime.dtype == torch.bfloat16 and bool((narrow[:self.router.shape[0]].float() == self.router).all()) else None
         self.correction = weights["correction"].to(torch.float32).contiguous() if params.get("correction", True) else None
         self.shared_gate_up = self.shared_down = None
         self.shared_group = 0
@@ -134,7 +136,7 @@ class RoutedExperts(FeedForward):
         tokens = x.shape[0]
         if self.router_narrow is not None:
             logits = ops.linear_wide(x, self.router_narrow)
-            chosen, weights, *gate = ops.moe_select(logits, self.correction, self.top, self.route_scale, **self.rule)
+            chosen, weights, *gate = ops.moe_select(logits, self.correction, self.top, self.route_scale, experts=self.experts, **self.rule)
         else:
             chosen, weights, *gate = ops.moe_route(x, self.router, self.correction, self.top, self.route_scale, **self.rule)
         shared_gate = gate[0] if gate else None

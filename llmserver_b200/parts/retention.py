@@ -59,7 +59,7 @@ class Retention(Mixer):
         super().__init__(params, weights, runtime)
         self.heads, self.dim, self.value_dim = int(params["heads"]), int(params["dim"]), int(params["value_dim"])
         self.eps = float(params["eps"])
-        if not ops.matrix_recurrence_supported(self.dim, self.value_dim):
+        if not ops.decay_recurrence_supported(self.dim, self.value_dim):
             raise ValueError(f"retention: no kernel for heads of {self.dim} key and {self.value_dim} value channels")
         name = _names(type(self), params)
         self.fused = torch.cat([weights[name[role]] for role in ("q", "k", "v", "g")], dim=0).contiguous()
@@ -147,7 +147,7 @@ class StateSpaceDuality(Mixer):
         super().__init__(params, weights, runtime)
         self.heads, self.value_dim, self.state, self.groups, self.inner, self.channels = self.sizes(params)
         self.norm_groups, self.eps = int(params["norm_groups"]), float(params["eps"])
-        if not ops.matrix_recurrence_supported(self.state, self.value_dim):
+        if not ops.decay_recurrence_supported(self.state, self.value_dim):
             raise ValueError(f"state_space_duality: no kernel for a state of {self.state} by {self.value_dim} channels")
         name = _names(type(self), params)
         into = weights[name["in"]]
