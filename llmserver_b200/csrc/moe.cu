@@ -20,7 +20,7 @@
 //   combine    out[t] = sum_j weight[t, j] * down[t * top + j] (+ gate[t] * shared[t]) in 32-bit, slots in order.
 #include "common.cuh"
 
-#define MOE_MAX_TOP 32
+#define MOE_MAX_TOP 1024
 
 struct RouteRule {
     int experts, top;

@@ -2,7 +2,9 @@
 kinds of layers, layers with a dense, a routed and no feed-forward, grouped and ungrouped query heads, value heads smaller
 and larger than key heads, chunks of one position, of a few, of some pages and longer than any prompt, no chunks, few and
 many distance buckets whose last one is reached early, late or never, convolutions of one to six taps, all or a part of a
-retention head rotating or nothing of it, decays of one and far from it, state-space groups of one and of several heads,
+retention head rotating or nothing of it, decays of one and below it (a head that forgets at once
+reads little but its own token, and its sign is all that the division by its root mean square leaves of q . k: rounding
+would decide it), state-space groups of one and of several heads,
 norm parts smaller and larger than a head and ones that cut heads in two, routers whose groups are all kept, half kept or
 absent, as many experts chosen as the kept groups hold, and shared experts beside them or none."""
 
@@ -46,8 +48,8 @@ ATTENTION_ONLY = {
 RETENTION_ONLY = {
     "architecture": "Dozotar", "vocab": 150, "width": 40, "norm": {"eps": 1e-6},
     "layers": [
-        _retention(24, 33, [0.999, 0.6], 8, None),
-        _retention(8, 16, [1.0, 0.98, 0.9, 0.5, 0.0], 8, _dense(72), base=50.0),
+        _retention(24, 33, [0.999, 0.93], 8, None),
+        _retention(8, 16, [1.0, 0.98, 0.9, 0.8, 0.96], 8, _dense(72), base=50.0),
         _retention(72, 20, [0.995], 2, _moe(8, 4, 24, (2, 1), 16)),
         _retention(40, 7, [0.97, 0.99, 0.85], None, None),
     ],

@@ -171,6 +171,24 @@ def route(z, router):
     return chosen, picked / (picked.sum() + 1e-20)
 
 
+def routing_margin(z, router):
+    """How far one token's choice is from another one, in units of the router's logits: the gap between the last expert
+    chosen and the first one left out, and between the last group kept and the first one dropped."""
+    experts, top = int(router["experts"]), int(router["top"])
+    gaps, allowed = [], list(range(experts))
+    if router.get("groups"):
+        count, keep = int(router["groups"]["count"]), int(router["groups"]["keep"])
+        size = experts // count
+        best = sorted(((float(z[g * size:(g + 1) * size].max()), g) for g in range(count)), reverse=True)
+        if keep < count:
+            gaps.append(best[keep - 1][0] - best[keep][0])
+        allowed = [e for e in allowed if e // size in [g for _, g in best[:keep]]]
+    ranked = sorted((float(z[e]) for e in allowed), reverse=True)
+    if top < len(ranked):
+        gaps.append(ranked[top - 1] - ranked[top])
+    return min(gaps) if gaps else math.inf
+
+
 def routed_feed_forward(h, weights, prefix, mlp):
     z = h @ weights[prefix + "router"].T
     y = torch.zeros_like(h)
@@ -206,14 +224,18 @@ def mixer_output(layer, x, weights, prefix, eps, lose_state_at=None):
     return torch.cat([first, ssd(x[lose_state_at:], weights, prefix, m, eps)[0]], dim=0)
 
 
-def forward(config, weights, tokens, lose_state_at=None, streams=None):
-    """float64 logits [T, vocab] of the whole sequence."""
+def forward(config, weights, tokens, lose_state_at=None, streams=None, margins=None):
+    """float64 logits [T, vocab] of the whole sequence.  ``margins``: receives each token's smallest routing margin."""
     eps = float(config["norm"]["eps"])
     x = weights["embed"][torch.tensor(list(tokens))]
     for index, layer in enumerate(config["layers"]):
         prefix = f"l{index}."
         x = x + scalar_norm(mixer_output(layer, x, weights, prefix + "mix.", eps, lose_state_at), weights[prefix + "norm1"], eps)
         if layer.get("mlp"):
+            if margins is not None and layer["mlp"]["kind"] == "moe":
+                z = x @ weights[prefix + "mlp.router"].T
+                found = torch.tensor([routing_margin(row, layer["mlp"]["router"]) for row in z])
+                margins.append(found if not margins else torch.minimum(margins.pop(), found))
             x = x + scalar_norm(feed_forward(x, weights, prefix + "mlp.", layer["mlp"]), weights[prefix + "norm2"], eps)
         if streams is not None:
             streams.append(x.clone())
