@@ -472,6 +472,11 @@ int arrangement(int dim, int vdim, int* partitions, int* threads) {
     return *threads <= kMaxThreads ? rows : 0;
 }
 
+constexpr int kSharedLimit = 200 * 1024;
+int shared_bytes(int rows, int mode, int dim, int vdim, int partitions, int element) {
+    return rows == 16 ? layout_of<16>(mode, dim, vdim, partitions, element).total : layout_of<32>(mode, dim, vdim, partitions, element).total;
+}
+
 int launch(DecayArgs& a, int mode, int n_seqs, int dtype, cudaStream_t stream) {
     if (n_seqs == 0) return LLM_OK;
     const bool segmented = a.segment > 0;
@@ -482,11 +487,11 @@ int launch(DecayArgs& a, int mode, int n_seqs, int dtype, cudaStream_t stream) {
     int threads = 0;
     const int rows = a.heads > 0 && a.dim > 0 && a.vdim > 0 ? arrangement(a.dim, a.vdim, &a.partitions, &threads) : 0;
     const int element = dtype == LLM_BF16 ? 2 : 4;
-    const size_t shared = rows == 0 ? 0 : (size_t)(rows == 16 ? layout_of<16>(mode, a.dim, a.vdim, a.partitions, element) : layout_of<32>(mode, a.dim, a.vdim, a.partitions, element)).total;
+    const size_t shared = rows == 0 ? 0 : (size_t)shared_bytes(rows, mode, a.dim, a.vdim, a.partitions, element);
     const int per = 16 / element;
     a.vec_proj = a.row_width % per == 0 && a.g_offset % per == 0 && a.vdim % per == 0 && aligned16(a.proj) &&
                  (mode == SSD || (a.q_offset % per == 0 && a.k_offset % per == 0 && a.v_offset % per == 0 && a.dim % per == 0));
-    if (!rows || shared > 200 * 1024) {
+    if (!rows || shared > kSharedLimit) {
         llm_set_error("decay recurrence: %d heads of %d key and %d value channels are not supported", a.heads, a.dim, a.vdim);
         return LLM_REFUSED;
     }
@@ -526,10 +531,15 @@ int launch(DecayArgs& a, int mode, int n_seqs, int dtype, cudaStream_t stream) {
 
 }  // namespace
 
-// Threads per block for heads of `dim` x `vdim` (0: not supported); the caller sizes its segments by it.
+// Threads per block for heads of `dim` x `vdim` (0: not supported, in either type or form); the caller sizes its segments
+// by it.
 LLM_EXPORT int llm_decay_recurrence_threads(int dim, int vdim) {
     int partitions, threads;
-    return dim > 0 && vdim > 0 && arrangement(dim, vdim, &partitions, &threads) ? threads : 0;
+    const int rows = dim > 0 && vdim > 0 ? arrangement(dim, vdim, &partitions, &threads) : 0;
+    if (!rows) return 0;
+    for (int mode = RETENTION; mode <= SSD; ++mode)
+        if (shared_bytes(rows, mode, dim, vdim, partitions, 4) > kSharedLimit) return 0;
+    return threads;
 }
 
 LLM_EXPORT int llm_retention_recurrent(const void* proj, int row_width, int q_offset, int k_offset, int v_offset, int g_offset,
