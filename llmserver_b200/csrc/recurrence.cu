@@ -10,7 +10,9 @@
 //     head's query, key or value channels); the first `n_unit_norm` units are then made unit vectors,
 //     y / sqrt(sum(y^2) + norm_eps), and the first `n_scaled` of those multiplied by `scale`.  Results are 32-bit.  A block
 //     takes 64 tokens of one unit; only a sequence's first block touches its stored inputs (a chunk is longer than any
-//     history), reads them for its first tokens and then brings them up to date.
+//     history), reads them for its first tokens and then brings them up to date.  Plain channels may also come without the
+//     SiLU, in the activation type, and with a bias on what goes in (`in_bias`: the bias of the projection in front, which
+//     is then part of the inputs that are kept; in front of a sequence there are zeros, not biases).
 //
 // (3) The recurrences (`llm_wkv_recurrent`, `llm_delta_rule_recurrent`), per head with S in R^(dim x vdim):
 //       wkv     o_t = (S + diag(u) k_t v_t^T)^T r_t;   S <- diag(w_t) S + k_t v_t^T;   w_t = exp(-exp(z_t + w0))
@@ -75,19 +77,22 @@ struct ConvArgs {
     float* state;           // [slots, max(taps - 1, 1), channels]: a sequence's last inputs, oldest first
     const int* state_slots;
     const int* q_start;
-    float* out;             // [N, channels]
+    void* out;              // [N, channels]
     int channels;
     int n_unit_norm, unit_dim, n_scaled;   // units 0 .. n_unit_norm - 1 have unit_dim channels and are made unit vectors
     int n_plain, plain_dim;                // the units behind them (the last may be cut short by `channels`)
     float norm_eps, scale;
     const float* bias;                     // [channels] or null
+    const float* in_bias;                  // [channels] or null: joins every input
+    int silu;                              // 0: no activation
 };
 
 #define CONV_MAX_PER_LANE 16    // a unit has at most 32 * 16 channels
 #define CONV_MAX_TAPS 64
 #define CONV_CHUNK 64           // tokens per block; more than CONV_MAX_TAPS - 1, so only a sequence's first block reads stored inputs
 
-template <typename T>
+// O: the type of the results.
+template <typename T, typename O>
 __global__ void __launch_bounds__(256) short_conv_units_kernel(ConvArgs a) {
     pdl_trigger();
     pdl_wait();
@@ -113,11 +118,11 @@ __global__ void __launch_bounds__(256) short_conv_units_kernel(ConvArgs a) {
                 float sum = a.bias ? a.bias[first + c] : 0.0f;
                 for (int j = 0; j < a.taps; ++j) {
                     const int source = t - history + j;      // on the step's token axis; before `begin`: the stored inputs
-                    const float value = source >= begin ? Num<T>::load(x + (size_t)source * a.row_width + c)
+                    const float value = source >= begin ? Num<T>::load(x + (size_t)source * a.row_width + c) + (a.in_bias ? a.in_bias[first + c] : 0.0f)
                                                         : state[(size_t)(history + source - begin) * a.channels + c];
                     sum = fmaf(a.taps_w[(size_t)(first + c) * a.taps + j], value, sum);
                 }
-                y[u] = sum / (1.0f + expf(-sum));
+                y[u] = a.silu ? sum / (1.0f + expf(-sum)) : sum;
                 squares = fmaf(y[u], y[u], squares);
             }
         }
@@ -129,7 +134,7 @@ __global__ void __launch_bounds__(256) short_conv_units_kernel(ConvArgs a) {
 #pragma unroll
         for (int u = 0; u < CONV_MAX_PER_LANE; ++u) {
             const int c = lane + 32 * u;
-            if (c < size) a.out[(size_t)t * a.channels + first + c] = y[u] * factor;
+            if (c < size) Num<O>::store((O*)a.out + (size_t)t * a.channels + first + c, y[u] * factor);
         }
     }
     if (blockIdx.z != 0) return;
@@ -140,7 +145,7 @@ __global__ void __launch_bounds__(256) short_conv_units_kernel(ConvArgs a) {
     for (int c = threadIdx.x; c < size; c += blockDim.x) {
         for (int r = 0; r < history; ++r) {
             const int source = length - history + r;      // relative to `begin`
-            state[(size_t)r * a.channels + c] = source >= 0 ? Num<T>::load(x + (size_t)(begin + source) * a.row_width + c)
+            state[(size_t)r * a.channels + c] = source >= 0 ? Num<T>::load(x + (size_t)(begin + source) * a.row_width + c) + (a.in_bias ? a.in_bias[first + c] : 0.0f)
                                                              : state[(size_t)(history + source) * a.channels + c];
         }
     }
@@ -150,7 +155,7 @@ __global__ void __launch_bounds__(256) short_conv_units_kernel(ConvArgs a) {
 // a vector's tokens with the inputs in its registers.  The thread that has a sequence's first tokens of a vector is the
 // only one that reads and renews the vector's stored inputs (CONV_ROLL tokens are more than any history it takes).
 #define CONV_ROLL 16
-template <typename T, int TAPS>
+template <typename T, typename O, int TAPS>
 __global__ void __launch_bounds__(128) short_conv_roll_kernel(ConvArgs a) {
     pdl_trigger();
     pdl_wait();
@@ -162,7 +167,7 @@ __global__ void __launch_bounds__(128) short_conv_roll_kernel(ConvArgs a) {
     constexpr int history = TAPS - 1;
     const T* x = (const T*)a.x + a.column + c;
     float* state = a.state + (size_t)a.state_slots[seq] * history * a.channels + c;
-    float w[TAPS][8], v[TAPS][8], bias[8];      // v[j]: the input that tap j meets
+    float w[TAPS][8], v[TAPS][8], bias[8], in_bias[8];      // v[j]: the input that tap j meets
     {
         float rows[8 * TAPS];      // the vector's weights lie one behind the other
 #pragma unroll
@@ -171,15 +176,19 @@ __global__ void __launch_bounds__(128) short_conv_roll_kernel(ConvArgs a) {
         for (int i = 0; i < 8; ++i) {
 #pragma unroll
             for (int j = 0; j < TAPS; ++j) w[j][i] = rows[i * TAPS + j];
-            bias[i] = 0.0f;
+            bias[i] = in_bias[i] = 0.0f;
         }
         if (a.bias) load8<float>(a.bias + c, bias);
+        if (a.in_bias) load8<float>(a.in_bias + c, in_bias);
     }
 #pragma unroll
     for (int j = 0; j < history; ++j) {
         const int source = first - history + j;
-        if (source >= begin) load8<T>(x + (size_t)source * a.row_width, v[j + 1]);
-        else load8<float>(state + (size_t)(history + source - begin) * a.channels, v[j + 1]);
+        if (source >= begin) {
+            load8<T>(x + (size_t)source * a.row_width, v[j + 1]);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) v[j + 1][i] += in_bias[i];
+        } else load8<float>(state + (size_t)(history + source - begin) * a.channels, v[j + 1]);
     }
     constexpr int FETCH = 4;
     for (int t0 = first; t0 < last; t0 += FETCH) {
@@ -197,12 +206,13 @@ __global__ void __launch_bounds__(128) short_conv_roll_kernel(ConvArgs a) {
                 float y[8];
 #pragma unroll
                 for (int i = 0; i < 8; ++i) {
+                    v[TAPS - 1][i] += in_bias[i];
                     float sum = bias[i];
 #pragma unroll
                     for (int j = 0; j < TAPS; ++j) sum = fmaf(w[j][i], v[j][i], sum);
-                    y[i] = sizeof(T) == 2 ? __fdividef(sum, 1.0f + __expf(-sum)) : sum / (1.0f + expf(-sum));
+                    y[i] = !a.silu ? sum : sizeof(T) == 2 ? __fdividef(sum, 1.0f + __expf(-sum)) : sum / (1.0f + expf(-sum));
                 }
-                store8<float>(a.out + (size_t)(t0 + u) * a.channels + c, y);
+                store8<O>((O*)a.out + (size_t)(t0 + u) * a.channels + c, y);
             }
         }
     }
@@ -212,16 +222,22 @@ __global__ void __launch_bounds__(128) short_conv_roll_kernel(ConvArgs a) {
     for (int r = 0; r < history; ++r) {      // oldest first: a row is read before it is overwritten
         const int source = length - history + r;
         float kept[8];
-        if (source >= 0) load8<T>(x + (size_t)(begin + source) * a.row_width, kept);
-        else load8<float>(state + (size_t)(history + source) * a.channels, kept);
+        if (source >= 0) {
+            load8<T>(x + (size_t)(begin + source) * a.row_width, kept);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) kept[i] += in_bias[i];
+        } else load8<float>(state + (size_t)(history + source) * a.channels, kept);
         store8<float>(state + (size_t)r * a.channels, kept);
     }
 }
 
+// `narrow`: the results in the activation type instead of 32-bit; `silu` 0: no activation; `in_bias` (32-bit [channels], may be
+// null) joins every input, also the ones that are kept.
 LLM_EXPORT int llm_short_conv_units(const void* x, int row_width, int column, const float* taps_w, int taps, float* state,
-                                    const int* state_slots, const int* q_start, float* out, int n_seqs, int longest, int n_unit_norm,
+                                    const int* state_slots, const int* q_start, void* out, int n_seqs, int longest, int n_unit_norm,
                                     int unit_dim, int n_scaled, int n_plain, int plain_dim, float norm_eps, float scale,
-                                    const float* bias, int channels, int dtype, cudaStream_t stream) {
+                                    const float* bias, int channels, const float* in_bias, int silu, int narrow, int dtype,
+                                    cudaStream_t stream) {
     if (n_seqs == 0 || longest <= 0) return LLM_OK;
     // the plain units cover the channels behind the normalised ones, only the last of them cut short
     const int plain = channels - n_unit_norm * unit_dim;
@@ -241,18 +257,28 @@ LLM_EXPORT int llm_short_conv_units(const void* x, int row_width, int column, co
     a.state_slots = state_slots; a.q_start = q_start; a.out = out;
     a.channels = channels; a.bias = bias;
     a.n_unit_norm = n_unit_norm; a.unit_dim = unit_dim; a.n_scaled = n_scaled; a.n_plain = n_plain; a.plain_dim = plain_dim;
-    a.norm_eps = norm_eps; a.scale = scale;
+    a.norm_eps = norm_eps; a.scale = scale; a.in_bias = in_bias; a.silu = silu;
     if (n_unit_norm == 0 && taps >= 2 && taps <= 4 && channels % 8 == 0 && column % 8 == 0 && row_width % 8 == 0 && aligned16(x) &&
-        aligned16(state) && aligned16(out) && aligned16(taps_w) && aligned16(bias)) {
+        aligned16(state) && aligned16(out) && aligned16(taps_w) && aligned16(bias) && aligned16(in_bias)) {
         const dim3 grid((longest + CONV_ROLL - 1) / CONV_ROLL, (channels / 8 + 127) / 128, n_seqs);
+#define LLM_CONV_ROLL(O)                                                                               \
+    do {                                                                                               \
+        if (taps == 2) llm_launch(short_conv_roll_kernel<T, O, 2>, grid, 128, 0, stream, a);           \
+        else if (taps == 3) llm_launch(short_conv_roll_kernel<T, O, 3>, grid, 128, 0, stream, a);      \
+        else llm_launch(short_conv_roll_kernel<T, O, 4>, grid, 128, 0, stream, a);                     \
+    } while (0)
         LLM_DISPATCH_DTYPE(dtype, {
-            if (taps == 2) llm_launch(short_conv_roll_kernel<T, 2>, grid, 128, 0, stream, a);
-            else if (taps == 3) llm_launch(short_conv_roll_kernel<T, 3>, grid, 128, 0, stream, a);
-            else llm_launch(short_conv_roll_kernel<T, 4>, grid, 128, 0, stream, a);
+            if (narrow) LLM_CONV_ROLL(T);
+            else LLM_CONV_ROLL(float);
         });
+#undef LLM_CONV_ROLL
         return llm_check_launch("short_conv_units");
     }
-    LLM_DISPATCH_DTYPE(dtype, (llm_launch(short_conv_units_kernel<T>, dim3(n_seqs, n_unit_norm + n_plain, (longest + CONV_CHUNK - 1) / CONV_CHUNK), 256, 0, stream, a)));
+    const dim3 grid(n_seqs, n_unit_norm + n_plain, (longest + CONV_CHUNK - 1) / CONV_CHUNK);
+    LLM_DISPATCH_DTYPE(dtype, {
+        if (narrow) llm_launch(short_conv_units_kernel<T, T>, grid, 256, 0, stream, a);
+        else llm_launch(short_conv_units_kernel<T, float>, grid, 256, 0, stream, a);
+    });
     return llm_check_launch("short_conv_units");
 }
 

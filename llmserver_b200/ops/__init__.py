@@ -26,17 +26,30 @@ __all__ = ["KernelError", "embedding", "add_rmsnorm", "rmsnorm", "silu_mul", "sa
            "gelu_mul", "grouped_rmsnorm", "conv_norm_kv"]
 
 
-def embedding(table: torch.Tensor, ids: torch.Tensor, out: Optional[torch.Tensor] = None, scale: float = 1.0) -> torch.Tensor:
-    """residual[n] = table[ids[n]] * scale, widened to float32.  ids: int32 [N]."""
+def embedding(table: torch.Tensor, ids: torch.Tensor, out: Optional[torch.Tensor] = None, scale: float = 1.0,
+              copies: int = 1, positions: Optional[torch.Tensor] = None, frequencies: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """residual[n] = table[ids[n]] * scale, widened to float32.  ids: int32 [N].
+
+    ``frequencies`` (float32 [ceil(H / 2), 2], a frequency as the sum of two floats) with ``positions`` (int32 [N]): a
+    sinusoidal position vector is added, sin(p f_i) to element 2i and cos(p f_i) to element 2i + 1.  ``copies`` > 1: every row
+    is written that many times, [N, copies, H]."""
     check(table, "embedding table")
     check(ids, "token ids", torch.int32)
     vocab, hidden = table.shape
     tokens = ids.numel()
+    if frequencies is not None:
+        check(frequencies, "position frequencies", torch.float32, 2)
+        check(positions, "positions", torch.int32)
+        if frequencies.shape[0] != (hidden + 1) // 2 or positions.numel() != tokens:
+            raise KernelError(f"{frequencies.shape[0]} frequencies and {positions.numel()} positions for {tokens} rows of {hidden}")
     if out is None:
-        out = torch.empty((tokens, hidden), dtype=torch.float32, device=table.device)
+        out = torch.empty((tokens, hidden) if copies == 1 else (tokens, copies, hidden), dtype=torch.float32, device=table.device)
     check(out, "embedding output", torch.float32, hidden)
+    if out.numel() != tokens * copies * hidden:
+        raise KernelError(f"the embedding's output {tuple(out.shape)} does not hold {copies} copies of {tokens} rows")
     call("llm_embedding_gather", out.data_ptr(), table.data_ptr(), ids.data_ptr(), tokens, hidden, vocab,
-         dtype_code(table.dtype), float(scale), stream_handle())
+         dtype_code(table.dtype), float(scale), int(copies), pointer(positions) if frequencies is not None else 0, pointer(frequencies),
+         stream_handle())
     return out
 
 
@@ -574,7 +587,8 @@ def token_shift_mix(h: torch.Tensor, shift_state: torch.Tensor, batch, mu: torch
 
 def short_conv_units(x: torch.Tensor, column: int, taps_w: torch.Tensor, state: torch.Tensor, batch, n_unit_norm: int,
                      unit_dim: int, n_scaled: int, n_plain: int, plain_dim: int, norm_eps: float, scale: float,
-                     bias: Optional[torch.Tensor] = None, channels: Optional[int] = None) -> torch.Tensor:
+                     bias: Optional[torch.Tensor] = None, channels: Optional[int] = None, in_bias: Optional[torch.Tensor] = None,
+                     silu: bool = True, out_dtype: torch.dtype = torch.float32) -> torch.Tensor:
     """A short causal convolution over time, channel by channel, then SiLU:
 
         y_t[c] = silu(sum_j taps_w[c, j] * x_(t - taps + 1 + j)[c] + bias[c])      zeros before a sequence's start
@@ -583,25 +597,31 @@ def short_conv_units(x: torch.Tensor, column: int, taps_w: torch.Tensor, state: 
     the current token's.  Channels come in units: first ``n_unit_norm`` units of ``unit_dim`` channels, each made a unit
     vector y / sqrt(sum(y^2) + norm_eps), the first ``n_scaled`` of them multiplied by ``scale``; then ``n_plain`` units of
     ``plain_dim`` channels that stay as they are (the last of them cut short where ``channels`` says so).  ``bias`` (float32
-    [channels]) may be absent.  A sequence's last taps - 1 inputs live in its slot of ``state``
-    (float32 [slots, max(taps - 1, 1), channels]) and are brought up to date.  Returns float32 [N, channels]."""
+    [channels]) may be absent, and so may the SiLU (``silu`` False).  ``in_bias`` (float32 [channels]) joins every input, kept
+    ones too: the bias of the projection in front, zeros still standing before a sequence's start.  A sequence's last taps - 1 inputs live in its slot of ``state``
+    (float32 [slots, max(taps - 1, 1), channels]) and are brought up to date.  Returns [N, channels] in float32
+    or, as ``out_dtype``, in x's type."""
     check(x, "x")
     tokens, row_width = x.shape
     channels = n_unit_norm * unit_dim + n_plain * plain_dim if channels is None else int(channels)
     taps = taps_w.shape[1]
     if bias is not None:
         check(bias, "convolution bias", torch.float32, channels)
+    if in_bias is not None:
+        check(in_bias, "input bias", torch.float32, channels)
+    if out_dtype not in (torch.float32, x.dtype):
+        raise KernelError(f"a convolution writes float32 or its input's type, not {out_dtype}")
     check(taps_w, "convolution weights", torch.float32)
     if taps_w.shape[0] != channels or column < 0 or column + channels > row_width:
         raise KernelError(f"{channels} channels from column {column} do not fit rows of {row_width} or weights {tuple(taps_w.shape)}")
     check(state, "convolution state", torch.float32, channels)
     if state.dim() != 3 or state.shape[1] != max(taps - 1, 1):
         raise KernelError(f"the convolution state must be [slots, {max(taps - 1, 1)}, {channels}], got {tuple(state.shape)}")
-    out = torch.empty((tokens, channels), dtype=torch.float32, device=x.device)
+    out = torch.empty((tokens, channels), dtype=out_dtype, device=x.device)
     call("llm_short_conv_units", x.data_ptr(), row_width, int(column), taps_w.data_ptr(), int(taps), state.data_ptr(),
          batch.state_slots.data_ptr(), batch.q_start.data_ptr(), out.data_ptr(), batch.n_seqs, int(batch.max_q_len), int(n_unit_norm),
-         int(unit_dim), int(n_scaled), int(n_plain), int(plain_dim), float(norm_eps), float(scale), pointer(bias), channels, dtype_code(x.dtype),
-         stream_handle())
+         int(unit_dim), int(n_scaled), int(n_plain), int(plain_dim), float(norm_eps), float(scale), pointer(bias), channels, pointer(in_bias),
+         int(bool(silu)), int(out_dtype != torch.float32), dtype_code(x.dtype), stream_handle())
     return out
 
 

@@ -16,7 +16,7 @@ _P, _I, _F, _S = ctypes.c_void_p, ctypes.c_int, ctypes.c_float, ctypes.c_void_p
 
 # name -> argument types (every launcher returns an int status; the stream comes last)
 SIGNATURES = {
-    "llm_embedding_gather": [_P, _P, _P, _I, _I, _I, _I, _F, _S],
+    "llm_embedding_gather": [_P, _P, _P, _I, _I, _I, _I, _F, _I, _P, _P, _S],
     "llm_add_rmsnorm": [_P, _P, _P, _P, _P, _I, _I, _F, _I, _I, _I, _P, _S],
     "llm_rmsnorm": [_P, _P, _P, _I, _I, _F, _I, _I, _S],
     "llm_silu_mul": [_P, _P, _I, _I, _I, _I, _S],
@@ -41,7 +41,9 @@ SIGNATURES = {
     "llm_gla_recurrent": [_P, _I, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _F, _F, _F, _I, _I, _I, _I, _P, _P, _S],
     "llm_pointwise": [_I, _P, _P, _P, ctypes.c_longlong, _F, _F, _I, _I, _S],
     "llm_token_shift_mix": [_P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _S],
-    "llm_short_conv_units": [_P, _I, _I, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _F, _P, _I, _I, _S],
+    "llm_short_conv_units": [_P, _I, _I, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _F, _P, _I, _P, _I, _I, _I, _S],
+    "llm_gated_scan": [_P, _P, _P, _P, _P, _I, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P, _I, _S],
+    "llm_streams_norm": [_P, _I, _I, _P, _P, _P, _F, _F, _P, _P, _P, _F, _F, _P, _P, _P, _P, _F, _I, _P, _P, _I, _I, _I, _S],
     "llm_matrix_recurrence_supports": [_I, _I],
     "llm_wkv_recurrent": [_P, _I, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _F, _P, _P, _I, _I, _I, _I, _I, _P, _P, _S],
     "llm_delta_rule_recurrent": [_P, _I, _I, _P, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _I, _P, _P, _S],
