@@ -32,15 +32,21 @@ class KVPagesNeed:
     else only the last ``window`` tokens are ever read.  ``value_dim``: the size of a value head where it differs
     from a key head's (None: the same).  ``keys_only``: what is cached serves as key and as value (a latent from which
     both are made): one tensor is kept and handed out as both.  ``chunk``: positions are cut into chunks of that many from
-    0 on and a query only ever reads keys of its own chunk, so everything in front of the chunk is done with."""
+    0 on and a query only ever reads keys of its own chunk, so everything in front of the chunk is done with.  ``keep_first``:
+    besides its window a query reads the sequence's first ``keep_first`` tokens, whose pages therefore stay."""
     kv_heads: int
     head_dim: int
     window: Optional[int] = None
     value_dim: Optional[int] = None
     keys_only: bool = False
     chunk: Optional[int] = None
+    keep_first: int = 0
 
     def __post_init__(self):
+        if int(self.keep_first) < 0:
+            raise ValueError(f"a cache cannot keep {self.keep_first} first tokens")
+        if self.window is None:
+            object.__setattr__(self, "keep_first", 0)       # without a window every token is kept
         if self.chunk is not None and (self.window is not None or int(self.chunk) <= 0):
             raise ValueError("a cache is bounded by a window or by chunks of a positive size, not by both")
         if self.keys_only and self.value_dim is not None:
@@ -85,8 +91,13 @@ class CacheGroup:
         table = self.tables[request_id]
         return max(0, -(-total_tokens // self.page_size) - len(table))
 
+    @property
+    def kept_pages(self) -> int:
+        """Leading pages that hold first tokens which every later query reads; they stay until their request ends."""
+        return -(-int(self.need.keep_first) // self.page_size)
+
     def passed_pages(self, num_computed: int) -> int:
-        """Number of leading pages no later query can read when ``num_computed`` tokens are done."""
+        """Number of leading pages (the kept ones aside) no later query can read when ``num_computed`` tokens are done."""
         if self.need.chunk is not None:      # the query at position num_computed sees its own chunk
             return num_computed // self.need.chunk * self.need.chunk // self.page_size
         if self.window is None:
@@ -290,7 +301,7 @@ class CacheManager:
         for group in self.groups:
             upto = min(group.passed_pages(num_computed), len(group.tables[request_id]))
             table = group.tables[request_id]
-            for index in range(group.released_upto[request_id], upto):
+            for index in range(max(group.released_upto[request_id], group.kept_pages), upto):
                 if table[index] != RELEASED:
                     group.pool.release(table[index])
                     table[index] = RELEASED

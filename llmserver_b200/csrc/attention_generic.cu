@@ -20,6 +20,10 @@
 // With `chunk` > 0 the sequence is cut into chunks of that many positions and a query sees the keys of its own chunk
 // only (from (p / chunk) * chunk on).  With `bias` (32-bit [Hq, bias_len]) the score of the key n positions back gets
 // bias[h][min(n, bias_len - 1)] added, which the scale does not multiply.
+//
+// With `keep` > 0 a windowed query also sees the sequence's first `keep` positions, at their true distances; they are
+// visited in front of the window's keys.  With `gate` the results are multiplied by sigmoid(gate[token * gate_stride + h *
+// value_dim + d]), formed in 32-bit, before their one rounding.
 #include "common.cuh"
 
 #define ATTN_MAX_D 512
@@ -31,8 +35,8 @@ __global__ void attention_generic_kernel(const T* __restrict__ q, int q_stride, 
                                          const int* __restrict__ positions, T* __restrict__ out, int n_q_heads,
                                          int n_kv_heads, int head_dim, int value_dim, int page_size, int num_pages,
                                          float scale, int window, const float* __restrict__ sinks,
-                                         int chunk, const float* __restrict__ bias, int bias_len,
-                                         int* __restrict__ error_flag) {
+                                         int chunk, const float* __restrict__ bias, int bias_len, int keep,
+                                         const T* __restrict__ gate, int gate_stride, int* __restrict__ error_flag) {
     pdl_trigger();   // let the next kernel start launching
     pdl_wait();      // everything before this kernel in the stream is complete and visible
     extern __shared__ float q_shared[];  // [warps][head_dim]
@@ -57,9 +61,12 @@ __global__ void attention_generic_kernel(const T* __restrict__ q, int q_stride, 
 
     int first = (window > 0 && position - window + 1 > 0) ? position - window + 1 : 0;
     if (chunk > 0) first = max(first, position / chunk * chunk);
-    for (int base = first; base <= position; base += 32) {
-        const int key = base + lane;
-        const bool valid = key <= position;
+    const int kept = min(keep, first);      // keys 0 .. kept - 1, then first .. position
+    const int count = kept + position - first + 1;
+    for (int base = 0; base < count; base += 32) {
+        const int index = base + lane;
+        const int key = index < kept ? index : first + index - kept;
+        const bool valid = index < count;
         long long offset = 0;  // this lane's key's slot in the pages: its key row lies at offset * head_dim, its value row at offset * value_dim
         float score = -INFINITY;
         if (valid) {
@@ -82,7 +89,7 @@ __global__ void attention_generic_kernel(const T* __restrict__ q, int q_stride, 
         normaliser = normaliser * correction + warp_sum(weight);
 #pragma unroll
         for (int i = 0; i < ATTN_MAX_D / 32; ++i) accumulator[i] *= correction;
-        const int in_chunk = min(32, position - base + 1);
+        const int in_chunk = min(32, count - base);
         for (int j = 0; j < in_chunk; ++j) {
             const float w = __shfl_sync(0xffffffffu, weight, j);
             const long long row = __shfl_sync(0xffffffffu, offset, j);
@@ -108,7 +115,11 @@ __global__ void attention_generic_kernel(const T* __restrict__ q, int q_stride, 
 #pragma unroll
     for (int i = 0; i < ATTN_MAX_D / 32; ++i) {
         const int d = lane + 32 * i;
-        if (d < value_dim) Num<T>::store(dst + d, accumulator[i] * inverse);
+        if (d < value_dim) {
+            float value = accumulator[i] * inverse;
+            if (gate) value /= 1.0f + expf(-Num<T>::load(gate + (size_t)token * gate_stride + (size_t)head * value_dim + d));
+            Num<T>::store(dst + d, value);
+        }
     }
 }
 
@@ -116,7 +127,8 @@ LLM_EXPORT int llm_attention_generic(const void* q, int q_stride, const void* k_
                                      const int* block_tables, int max_blocks, const int* seq_of_token,
                                      const int* positions, void* out, int n_tokens, int n_q_heads, int n_kv_heads,
                                      int head_dim, int value_dim, int page_size, int num_pages, float scale, int window,
-                                     const float* sinks, int chunk, const float* bias, int bias_len, int* error_flag, int dtype, cudaStream_t stream) {
+                                     const float* sinks, int chunk, const float* bias, int bias_len, int keep, const void* gate, int gate_stride,
+                                     int* error_flag, int dtype, cudaStream_t stream) {
     if (n_tokens == 0) return LLM_OK;
     if (head_dim > ATTN_MAX_D || head_dim <= 0) {
         llm_set_error("attention_generic: head_dim %d is outside 1..%d", head_dim, ATTN_MAX_D);
@@ -134,8 +146,8 @@ LLM_EXPORT int llm_attention_generic(const void* q, int q_stride, const void* k_
         llm_set_error("attention_generic: %d query heads are no multiple of %d kv heads", n_q_heads, n_kv_heads);
         return LLM_REFUSED;
     }
-    if (chunk < 0 || (bias && bias_len <= 0)) {
-        llm_set_error("attention_generic: a chunk of %d positions or a bias of %d distances", chunk, bias_len);
+    if (chunk < 0 || (bias && bias_len <= 0) || keep < 0 || (keep > 0 && chunk > 0)) {
+        llm_set_error("attention_generic: a chunk of %d positions, a bias of %d distances or %d kept positions", chunk, bias_len, keep);
         return LLM_REFUSED;
     }
     const int warps = 4;
@@ -144,6 +156,6 @@ LLM_EXPORT int llm_attention_generic(const void* q, int q_stride, const void* k_
     LLM_DISPATCH_DTYPE(dtype, (llm_launch(attention_generic_kernel<T>, grid, warps * 32, shared, stream, 
                                   (const T*)q, q_stride, (const T*)k_pages, (const T*)v_pages, block_tables,
                                   max_blocks, seq_of_token, positions, (T*)out, n_q_heads, n_kv_heads, head_dim,
-                                  value_dim, page_size, num_pages, scale, window, sinks, chunk, bias, bias_len, error_flag)));
+                                  value_dim, page_size, num_pages, scale, window, sinks, chunk, bias, bias_len, keep, (const T*)gate, gate_stride, error_flag)));
     return llm_check_launch("attention_generic");
 }

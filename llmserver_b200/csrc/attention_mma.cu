@@ -28,7 +28,9 @@
 // 16 significant bits, two MMAs instead of one), and exp(sink) joins the denominator once per row.  That form also
 // takes attention in chunks (a query sees the keys of its own chunk of positions only) and a learned bias per head and
 // distance between query and key, added to the scaled score (BIAS): the group's rows of the bias are staged in shared
-// memory, or read where they lie when they are too long for it.
+// memory, or read where they lie when they are too long for it.  With a window it can also keep a sequence's first `keep`
+// positions visible: the tiles that hold them are walked in front of the window's (walk_of), and tiles between the two are
+// skipped.  `gate` multiplies the results by the sigmoid of a number per element before their one rounding.
 #include "common.cuh"
 #include "tma.cuh"
 #include "tcgen05.cuh"
@@ -75,6 +77,9 @@ struct AttnParams {
     int bias_len = 0;               // at most bias_len - 1 (farther keys: the last entry); BIAS kernels only
     int bias_stride = 0;            // floats between two heads' staged rows; 0: the bias is not staged
     int bias_offset = 0;            // where the staged rows lie in the kernel's shared memory (bytes)
+    int keep = 0;                   // with a window: keys 0 .. keep - 1 stay visible; cp.async kernels only
+    const __nv_bfloat16* gate = nullptr;    // row of token n from gate + n * gate_stride on, [Hq * DV]: results are multiplied
+    int gate_stride = 0;                    // by its sigmoid; cp.async kernels and their merge only
 };
 
 // The first key that the query at `position` may see.
@@ -82,6 +87,27 @@ __device__ __forceinline__ int first_visible(const AttnParams& p, int position) 
     int low = p.window > 0 ? max(0, position - p.window + 1) : 0;
     if (p.chunk > 0 && position >= 0) low = max(low, position / p.chunk * p.chunk);
     return low;
+}
+
+// The tiles a row tile walks whose first row sees nothing in front of key `low` but the kept positions: tiles that hold kept
+// keys and end in front of the window's first tile, then the window's.  Tile i of the walk begins at key walk_key(i).
+struct Walk {
+    int kept_tiles, first_key;      // first_key: where the window's first tile begins
+};
+__device__ __forceinline__ Walk walk_of(const AttnParams& p, int low) {
+    Walk walk;
+    walk.first_key = low / kTileKeys * kTileKeys;
+    walk.kept_tiles = min((p.keep + kTileKeys - 1) / kTileKeys, low / kTileKeys);
+    return walk;
+}
+__device__ __forceinline__ int walk_key(const Walk& walk, int tile) {
+    return tile < walk.kept_tiles ? tile * kTileKeys : walk.first_key + (tile - walk.kept_tiles) * kTileKeys;
+}
+// Keys from the walk's start to the end of the context, whole tiles of kept keys included.
+__device__ __forceinline__ int walk_span(const Walk& walk, int context) { return walk.kept_tiles * kTileKeys + context - walk.first_key; }
+
+__device__ __forceinline__ float gated(const AttnParams& p, float value, int token, int column) {
+    return value * __fdividef(1.0f, 1.0f + __expf(-__bfloat162float(p.gate[(size_t)token * p.gate_stride + column])));
 }
 
 // Stages the group's rows of the bias behind the tiles (the caller's next block barrier makes them visible) and returns
@@ -267,7 +293,7 @@ __device__ __forceinline__ void warp_tile(const uint32_t (&q_frag)[D / 16][4], c
                                           const __nv_bfloat16* v_tile, int key_row, int key_index,
                                           const int (&row_low)[2], const int (&row_high)[2], float scale_log2,
                                           float (&o_acc)[DV / 8][4], float (&row_max)[2], float (&row_sum)[2],
-                                          const float* const* bias_row = nullptr, int bias_last = 0) {
+                                          const float* const* bias_row = nullptr, int bias_last = 0, int keep = 0) {
     const int lane = threadIdx.x & 31;
     const int matrix = lane >> 3, matrix_row = lane & 7;
     float s_acc[NT][4];
@@ -298,7 +324,7 @@ __device__ __forceinline__ void warp_tile(const uint32_t (&q_frag)[D / 16][4], c
         for (int i = 0; i < 4; ++i) {
             const int h = i >> 1;
             const int key = key_index + n * 8 + 2 * t + (i & 1);
-            const bool seen = key >= row_low[h] && key <= row_high[h];
+            const bool seen = (key >= row_low[h] || key < keep) && key <= row_high[h];
             if (BIAS) s_acc[n][i] = seen ? fmaf(s_acc[n][i], scale_log2, bias_row[h][min(row_high[h] - key, bias_last)]) : -INFINITY;
             else s_acc[n][i] = seen ? s_acc[n][i] * scale_log2 : -INFINITY;
             tile_max[h] = fmaxf(tile_max[h], s_acc[n][i]);
@@ -415,10 +441,10 @@ __global__ void __launch_bounds__(kThreads) attention_portions_kernel(const Attn
     const int base_position = context - q_len;
     const int high_key = base_position + last_token;
     const int low_key = first_visible(p, base_position + first_token);
-    const int first_tile_key = (low_key / kTileKeys) * kTileKeys;
-    const int n_tiles = (high_key - first_tile_key) / kTileKeys + 1;
+    const Walk walk = walk_of(p, low_key);
+    const int n_tiles = walk.kept_tiles + (high_key - walk.first_key) / kTileKeys + 1;
 
-    load_kv_tile<D, DV>(kv_tiles, kv_tiles + kTileKeys * D, p, table, kv_head, first_tile_key, context);
+    load_kv_tile<D, DV>(kv_tiles, kv_tiles + kTileKeys * D, p, table, kv_head, walk_key(walk, 0), context);
     cp_async_commit();
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -458,7 +484,7 @@ __global__ void __launch_bounds__(kThreads) attention_portions_kernel(const Attn
         __nv_bfloat16* v_tile = (DV == D && p.v_pages == p.k_pages) ? k_tile : k_tile + kTileKeys * D;
         if (it + 1 < n_tiles) {
             __nv_bfloat16* next_k = kv_tiles + (stage ^ 1) * kStage;
-            load_kv_tile<D, DV>(next_k, next_k + kTileKeys * D, p, table, kv_head, first_tile_key + (it + 1) * kTileKeys, context);
+            load_kv_tile<D, DV>(next_k, next_k + kTileKeys * D, p, table, kv_head, walk_key(walk, it + 1), context);
             cp_async_commit();
             cp_async_wait<1>();
         } else {
@@ -473,10 +499,10 @@ __global__ void __launch_bounds__(kThreads) attention_portions_kernel(const Attn
                 ldmatrix_x4(q_frag[ks], smem_address(q_tile + swizzled<D>(row, 2 * ks + (matrix >> 1))));
             }
         }
-        const int tile_key = first_tile_key + it * kTileKeys;
+        const int tile_key = walk_key(walk, it);
         // a warp whose rows all end before this tile has nothing to add (the causal upper triangle)
         if (tile_key <= warp_high)
-            warp_tile<D, 8, XorLayout<D>, DV, PRECISE, XorLayout<DV>, BIAS>(q_frag, k_tile, v_tile, 0, tile_key, row_low, row_high, p.scale_log2, o_acc, row_max, row_sum, bias_row, p.bias_len - 1);
+            warp_tile<D, 8, XorLayout<D>, DV, PRECISE, XorLayout<DV>, BIAS>(q_frag, k_tile, v_tile, 0, tile_key, row_low, row_high, p.scale_log2, o_acc, row_max, row_sum, bias_row, p.bias_len - 1, p.keep);
         __syncthreads();   // the stage is overwritten by the load issued in the next iteration
     }
 
@@ -500,8 +526,13 @@ __global__ void __launch_bounds__(kThreads) attention_portions_kernel(const Attn
         __nv_bfloat16* dst = p.out + (size_t)(token0 + r / group) * p.n_q_heads * DV + (size_t)(kv_head * group + r % group) * DV;
 #pragma unroll
         for (int n = 0; n < DV / 8; ++n) {
-            const uint32_t packed = pack_bf16(o_acc[n][2 * h] * inverse, o_acc[n][2 * h + 1] * inverse);
-            *reinterpret_cast<uint32_t*>(dst + n * 8 + 2 * t) = packed;
+            float low = o_acc[n][2 * h] * inverse, high = o_acc[n][2 * h + 1] * inverse;
+            if (p.gate) {
+                const int column = (kv_head * group + r % group) * DV + n * 8 + 2 * t;
+                low = gated(p, low, token0 + r / group, column);
+                high = gated(p, high, token0 + r / group, column + 1);
+            }
+            *reinterpret_cast<uint32_t*>(dst + n * 8 + 2 * t) = pack_bf16(low, high);
         }
     }
 }
@@ -532,15 +563,15 @@ __global__ void __launch_bounds__(kThreads) attention_decode_kernel(const AttnPa
     const int context = p.context_len[seq];
     const int position = context - 1;
     const int low_key = first_visible(p, position);
-    const int first_key = (low_key / kTileKeys) * kTileKeys;
-    const int split_len = split_length(p, context - first_key);
-    const int n_splits = (context - first_key + split_len - 1) / split_len;
+    const Walk walk = walk_of(p, low_key);
+    const int span = walk_span(walk, context);      // splits divide the walk, kept tiles first
+    const int split_len = split_length(p, span);
+    const int n_splits = (span + split_len - 1) / split_len;
     if (n_splits > p.max_splits && split == 0 && kv_head == 0 && threadIdx.x == 0 && p.error_flag) atomicExch(p.error_flag, 6);
     if (context <= 0 && split == 0) zero_output<DV>(p, token, kv_head, group);     // nothing to attend to
     if (split >= n_splits) return;
-    const int split_begin = first_key + split * split_len;
-    const int split_end = min(split_begin + split_len, context);
-    const int n_tiles = (split_end - split_begin + kTileKeys - 1) / kTileKeys;
+    const int first_tile = split * split_len / kTileKeys;      // of the walk; splits are whole tiles
+    const int n_tiles = (min(split_len, span - split * split_len) + kTileKeys - 1) / kTileKeys;
     const int* table = p.block_tables + (size_t)seq * p.max_blocks;
 
     {
@@ -553,7 +584,7 @@ __global__ void __launch_bounds__(kThreads) attention_decode_kernel(const AttnPa
             cp_async_16(smem_address(q_tile + swizzled<D>(row, chunk)), src, valid ? 16 : 0);
         }
     }
-    load_kv_tile<D, DV>(kv_tiles, kv_tiles + kTileKeys * D, p, table, kv_head, split_begin, split_end);
+    load_kv_tile<D, DV>(kv_tiles, kv_tiles + kTileKeys * D, p, table, kv_head, walk_key(walk, first_tile), context);
     cp_async_commit();
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -586,7 +617,7 @@ __global__ void __launch_bounds__(kThreads) attention_decode_kernel(const AttnPa
         __nv_bfloat16* v_tile = (DV == D && p.v_pages == p.k_pages) ? k_tile : k_tile + kTileKeys * D;
         if (it + 1 < n_tiles) {
             __nv_bfloat16* next_k = kv_tiles + (stage ^ 1) * kStage;
-            load_kv_tile<D, DV>(next_k, next_k + kTileKeys * D, p, table, kv_head, split_begin + (it + 1) * kTileKeys, split_end);
+            load_kv_tile<D, DV>(next_k, next_k + kTileKeys * D, p, table, kv_head, walk_key(walk, first_tile + it + 1), context);
             cp_async_commit();
             cp_async_wait<1>();
         } else {
@@ -602,9 +633,9 @@ __global__ void __launch_bounds__(kThreads) attention_decode_kernel(const AttnPa
             }
         }
         // each warp takes 16 of the tile's 64 keys
-        const int key_index = split_begin + it * kTileKeys + warp * 16;
-        if (key_index < split_end)
-            warp_tile<D, 2, XorLayout<D>, DV, PRECISE, XorLayout<DV>, BIAS>(q_frag, k_tile, v_tile, warp * 16, key_index, row_low, row_high, p.scale_log2, o_acc, row_max, row_sum, bias_row, p.bias_len - 1);
+        const int key_index = walk_key(walk, first_tile + it) + warp * 16;
+        if (key_index < context)
+            warp_tile<D, 2, XorLayout<D>, DV, PRECISE, XorLayout<DV>, BIAS>(q_frag, k_tile, v_tile, warp * 16, key_index, row_low, row_high, p.scale_log2, o_acc, row_max, row_sum, bias_row, p.bias_len - 1, p.keep);
         __syncthreads();
     }
 
@@ -647,7 +678,9 @@ __global__ void __launch_bounds__(kThreads) attention_decode_kernel(const AttnPa
             denominator += row[DV + 1] * weight;
         }
         if (n_splits == 1) {
-            p.out[(size_t)token * p.n_q_heads * DV + (size_t)head * DV + d] = __float2bfloat16_rn(numerator / denominator);
+            float value = numerator / denominator;
+            if (p.gate) value = gated(p, value, token, head * DV + d);
+            p.out[(size_t)token * p.n_q_heads * DV + (size_t)head * DV + d] = __float2bfloat16_rn(value);
         } else {
             const size_t slot = ((size_t)(p.slot_by_seq ? seq : token) * p.n_q_heads + head) * p.max_splits + split;
             p.partial_out[slot * DV + d] = numerator / denominator;
@@ -966,9 +999,9 @@ __global__ void attention_decode_merge_kernel(const AttnParams p) {
     if (p.q_start[seq + 1] - token != 1) return;
     const int context = p.context_len[seq];
     const int low_key = first_visible(p, context - 1);
-    const int first_key = (low_key / kTileKeys) * kTileKeys;
-    const int split_len = split_length(p, context - first_key);
-    const int n_splits = min((context - first_key + split_len - 1) / split_len, p.max_splits);
+    const int span = walk_span(walk_of(p, low_key), context);
+    const int split_len = split_length(p, span);
+    const int n_splits = min((span + split_len - 1) / split_len, p.max_splits);
     if (n_splits <= 1) return;
     const size_t slot0 = ((size_t)(p.slot_by_seq ? seq : token) * p.n_q_heads + head) * p.max_splits;
     float best = -INFINITY;
@@ -980,7 +1013,9 @@ __global__ void attention_decode_merge_kernel(const AttnParams p) {
             numerator += p.partial_out[(slot0 + s) * D + d] * weight;
             denominator += weight;
         }
-        p.out[(size_t)token * p.n_q_heads * D + (size_t)head * D + d] = __float2bfloat16_rn(numerator / denominator);
+        float value = numerator / denominator;
+        if (p.gate) value = gated(p, value, token, head * D + d);
+        p.out[(size_t)token * p.n_q_heads * D + (size_t)head * D + d] = __float2bfloat16_rn(value);
     }
 }
 
@@ -1342,12 +1377,15 @@ LLM_EXPORT int llm_attention_mma_sinks_supports(int head_dim, int value_dim, int
 //
 // Attention whose weights keep 16 significant bits in the P V product (see PRECISE above), with value heads of
 // `value_dim` elements and, with `sinks` (float32 [Hq], may be null), one more term exp(sinks[h]) in every row's
-// denominator.  The other arguments as for llm_attention_mma; out is [N, Hq * value_dim].
+// denominator.  `keep`: with a window, the first `keep` positions of a sequence stay visible.  `gate` (bfloat16, may be null):
+// token n's row gate + n * gate_stride holds a number per element of its output, whose sigmoid multiplies the result.  The
+// other arguments as for llm_attention_mma; out is [N, Hq * value_dim].
 LLM_EXPORT int llm_attention_mma_sinks(const void* q, int q_stride, const void* k_pages, const void* v_pages,
                                        const int* block_tables, int max_blocks, const int* q_start, const int* context_len,
                                        void* out, int n_seqs, int n_q_heads, int n_kv_heads, int head_dim, int value_dim,
                                        int page_size, int num_pages, float scale, int window, const float* sinks,
-                                       int chunk, const float* bias, int bias_len, int run_portions, int total_tiles, int run_decode, int split_len, int max_splits,
+                                       int chunk, const float* bias, int bias_len, int keep, const void* gate, int gate_stride,
+                                       int run_portions, int total_tiles, int run_decode, int split_len, int max_splits,
                                        float* partial_out, float* partial_ml, int* error_flag, cudaStream_t stream) {
     if (!llm_attention_mma_sinks_supports(head_dim, value_dim, n_q_heads, n_kv_heads)) {
         llm_set_error("attention_mma_sinks: keys of %d and values of %d with %d/%d heads are not supported (64 or 128 each, "
@@ -1389,13 +1427,16 @@ LLM_EXPORT int llm_attention_mma_sinks(const void* q, int q_stride, const void* 
     p.partial_ml = partial_ml;
     p.error_flag = error_flag;
     p.sinks = sinks;
-    if (chunk < 0 || (bias && bias_len <= 0)) {
-        llm_set_error("attention_mma_sinks: a chunk of %d positions or a bias of %d distances", chunk, bias_len);
+    if (chunk < 0 || (bias && bias_len <= 0) || keep < 0 || (keep > 0 && chunk > 0)) {
+        llm_set_error("attention_mma_sinks: a chunk of %d positions, a bias of %d distances or %d kept positions", chunk, bias_len, keep);
         return LLM_REFUSED;
     }
     p.chunk = chunk;
     p.bias = bias;
     p.bias_len = bias_len;
+    p.keep = window > 0 ? keep : 0;
+    p.gate = (const __nv_bfloat16*)gate;
+    p.gate_stride = gate_stride;
 #define LLM_PRECISE(BIAS)                                                                                                  \
     do {                                                                                                                   \
         if (head_dim == 64)                                                                                                \

@@ -75,7 +75,15 @@ struct PrefillParams {
     const float* bias = nullptr;    // BIAS: [Hq, bias_len], times log2(e): added to the score of the key n positions back, n at
     int bias_len = 0;               // most bias_len - 1 (farther keys: the last entry)
     int bias_stride = 0;            // floats between two heads' staged rows
+    int keep = 0;                   // with a window: keys 0 .. keep - 1 stay visible
+    const __nv_bfloat16* gate = nullptr;    // row of token n from gate + n * gate_stride on, [Hq * kDim]: results are
+    int gate_stride = 0;                    // multiplied by its sigmoid
 };
+
+// Where tile t of a row tile's walk begins: tiles of kept keys in front of the window's first tile, then the window's.
+__device__ __forceinline__ int walk_key(int kept_tiles, int first_tile_key, int t) {
+    return t < kept_tiles ? t * kKeys : first_tile_key + (t - kept_tiles) * kKeys;
+}
 
 // The first key that the query at `position` may see.
 __device__ __forceinline__ int first_visible(const PrefillParams& p, int position) {
@@ -187,7 +195,8 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_tcgen05_kernel(
     const int high_key = base_position + min(first_token + tokens_per_tile, q_len) - 1;
     const int low_key = first_visible(p, base_position + first_token);
     const int first_tile_key = (low_key / kKeys) * kKeys;
-    const int n_tiles = (high_key - first_tile_key) / kKeys + 1;
+    const int kept_tiles = min((p.keep + kKeys - 1) / kKeys, low_key / kKeys);
+    const int n_tiles = kept_tiles + (high_key - first_tile_key) / kKeys + 1;
 
     // fresh barriers for every pass: at the end of a pass every copy has landed and every MMA has retired
     if (threadIdx.x == 0) {
@@ -233,7 +242,7 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_tcgen05_kernel(
                     if (lane < copies) {
                         // whole tiles always: pages past the sequence's end come from whatever the zero-padded
                         // table names (an existing page with finite contents, masked out below)
-                        const int key = first_tile_key + t * kKeys + my_page * p.page_size;
+                        const int key = walk_key(kept_tiles, first_tile_key, t) + my_page * p.page_size;
                         const int page = table[min(key / p.page_size, p.max_blocks - 1)];
                         if ((unsigned)page >= (unsigned)p.num_pages && p.error_flag) atomicExch(p.error_flag, 5);
                         const uint32_t offset = s * kKVBytes + (uint32_t)(my_page * p.page_size) * 256u;
@@ -248,7 +257,7 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_tcgen05_kernel(
                     if (lane == 0) mbar_expect_tx(smem_u32(&v_full[s]), kKVBytes);
                     __syncwarp();
                     if (lane < copies) {
-                        const int key = first_tile_key + t * kKeys + my_page * p.page_size;
+                        const int key = walk_key(kept_tiles, first_tile_key, t) + my_page * p.page_size;
                         const int page = table[min(key / p.page_size, p.max_blocks - 1)];
                         const uint32_t offset = s * kKVBytes + (uint32_t)(my_page * p.page_size) * 256u;
                         tma_load_5d(v_smem + offset, &map_v, smem_u32(&v_full[s]), 0, 0, 0, 0, page * p.n_kv_heads + kv_head);
@@ -322,7 +331,7 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_tcgen05_kernel(
             const uint32_t s_address = lane_base + (b ? kColS1 : kColS0);
             uint32_t raw[64];
             tmem_load_64(s_address, raw);
-            const int tile_key = first_tile_key + j * kKeys;
+            const int tile_key = walk_key(kept_tiles, first_tile_key, j);
             if (BIAS) {      // scores leave here as they enter the exponent: scaled, with their bias, times log2(e)
                 const int back = position - tile_key;      // distance of the tile's first key; its last one is kKeys - 1 nearer
                 if (back - (kKeys - 1) >= p.bias_len - 1) {      // the whole tile lies beyond the last distance
@@ -340,7 +349,7 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_tcgen05_kernel(
             if (tile_key + kKeys - 1 > position || tile_key < low) {
 #pragma unroll
                 for (int c = 0; c < 64; ++c)
-                    if (!(tile_key + c >= low && tile_key + c <= position)) raw[c] = 0xff800000u;      // -inf
+                    if (!((tile_key + c >= low || tile_key + c < p.keep) && tile_key + c <= position)) raw[c] = 0xff800000u;      // -inf
             }
             // The maximum is taken over the raw scores (the scale is positive); the scale and the reference enter
             // the exponent in one fused multiply-add.  Eight running maxima and four running sums keep the
@@ -424,6 +433,17 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_tcgen05_kernel(
             uint32_t o_raw[32];
             tmem_load_32(lane_base + kColO + chunk * 32, o_raw);
             if (exists) {
+                if (p.gate) {
+                    const __nv_bfloat16* gate = p.gate + (size_t)(token0 + token) * p.gate_stride + (size_t)head * kDim + chunk * 32;
+#pragma unroll
+                    for (int v = 0; v < 4; ++v) {
+                        float g[8];
+                        load8<__nv_bfloat16>(gate + v * 8, g);
+#pragma unroll
+                        for (int e = 0; e < 8; ++e)
+                            o_raw[8 * v + e] = __float_as_uint(__fdividef(__uint_as_float(o_raw[8 * v + e]), 1.0f + __expf(-g[e])));
+                    }
+                }
 #pragma unroll
                 for (int v = 0; v < 4; ++v) {
                     uint4 words;
@@ -483,7 +503,7 @@ static int launch_prefill_tcgen05(const void* q, int q_stride, int n_tokens, con
                                   const int* context_len, void* out, int n_seqs, int n_q_heads, int n_kv_heads,
                                   int head_dim, int page_size, int num_pages, float scale, int window, int skip_single, int pairing,
                                   int total_pairs, int* error_flag, const float* sinks, bool precise, int chunk, const float* bias,
-                                  int bias_len, cudaStream_t stream) {
+                                  int bias_len, int keep, const void* gate, int gate_stride, cudaStream_t stream) {
     if (total_pairs <= 0) return LLM_OK;
     if (num_pages <= 0) {
         llm_set_error("attention_prefill_tcgen05: the page pool has %d pages", num_pages);
@@ -538,6 +558,13 @@ static int launch_prefill_tcgen05(const void* q, int q_stride, int n_tokens, con
         return LLM_REFUSED;
     }
     p.bias_stride = bias ? bias_row_stride(bias_len, group) : 0;
+    if (keep < 0 || (keep > 0 && chunk > 0) || (gate && (!aligned16(gate) || gate_stride % 8))) {
+        llm_set_error("attention_prefill_tcgen05: %d kept positions, or a gate whose rows are not 16-byte aligned", keep);
+        return LLM_REFUSED;
+    }
+    p.keep = window > 0 ? keep : 0;
+    p.gate = (const __nv_bfloat16*)gate;
+    p.gate_stride = gate_stride;
     const size_t shared = kSharedBytes;
     dim3 grid(total_pairs, n_kv_heads);
     if (bias) {
@@ -560,21 +587,22 @@ LLM_EXPORT int llm_attention_prefill_tcgen05(const void* q, int q_stride, int n_
                                              int total_pairs, int* error_flag, cudaStream_t stream) {
     return launch_prefill_tcgen05(q, q_stride, n_tokens, k_pages, v_pages, block_tables, max_blocks, q_start, context_len, out, n_seqs,
                                   n_q_heads, n_kv_heads, head_dim, page_size, num_pages, scale, window, skip_single, pairing,
-                                  total_pairs, error_flag, nullptr, false, 0, nullptr, 0, stream);
+                                  total_pairs, error_flag, nullptr, false, 0, nullptr, 0, 0, nullptr, 0, stream);
 }
 
 // The same with attention weights of 16 significant bits in the P V product and, with `sinks` (float32 [Hq], may be
 // null), one more term exp(sinks[h]) in every row's softmax denominator.  `chunk` > 0: a query sees the keys of its own
 // chunk of positions only.  `bias` (float32 [Hq, bias_len], given times log2(e); may be null): what is added to the score
-// of the key n positions back, at min(n, bias_len - 1).
+// of the key n positions back, at min(n, bias_len - 1).  `keep`: with a window, the first `keep` positions of a sequence stay
+// visible.  `gate` (bfloat16, 16-byte aligned rows gate + n * gate_stride, may be null): results are multiplied by its sigmoid.
 LLM_EXPORT int llm_attention_prefill_tcgen05_precise(const void* q, int q_stride, int n_tokens, const void* k_pages, const void* v_pages,
                                                      const int* block_tables, int max_blocks, const int* q_start,
                                                      const int* context_len, void* out, int n_seqs, int n_q_heads, int n_kv_heads,
                                                      int head_dim, int page_size, int num_pages, float scale, int window,
                                                      int skip_single, int pairing, int total_pairs, int* error_flag,
-                                                     const float* sinks, int chunk, const float* bias, int bias_len,
-                                                     cudaStream_t stream) {
+                                                     const float* sinks, int chunk, const float* bias, int bias_len, int keep,
+                                                     const void* gate, int gate_stride, cudaStream_t stream) {
     return launch_prefill_tcgen05(q, q_stride, n_tokens, k_pages, v_pages, block_tables, max_blocks, q_start, context_len, out, n_seqs,
                                   n_q_heads, n_kv_heads, head_dim, page_size, num_pages, scale, window, skip_single, pairing,
-                                  total_pairs, error_flag, sinks, true, chunk, bias, bias_len, stream);
+                                  total_pairs, error_flag, sinks, true, chunk, bias, bias_len, keep, gate, gate_stride, stream);
 }

@@ -219,13 +219,15 @@ def attention_generic(q: torch.Tensor, q_stride: int, k_pages: torch.Tensor, v_p
                       n_q_heads: int, n_kv_heads: int, head_dim: int, scale: float, window: int = 0,
                       out: Optional[torch.Tensor] = None, error_flag: Optional[torch.Tensor] = None,
                       value_dim: Optional[int] = None, sinks: Optional[torch.Tensor] = None, chunk: int = 0,
-                      bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+                      bias: Optional[torch.Tensor] = None, keep: int = 0, gate: Optional[torch.Tensor] = None,
+                      gate_column: int = 0) -> torch.Tensor:
     """Causal (optionally windowed) attention of every token over its sequence's pages, 32-bit
     arithmetic.  ``q`` holds head h of token n at q[n * q_stride + h * D]; returns [N, Hq * Dv], Dv = ``value_dim``
     (default D).  ``sinks`` (float32 [Hq]): one more term exp(sinks[h]) in each head's softmax denominator.  ``chunk`` > 0:
     a query sees the keys of its own chunk of that many positions only.  ``bias`` (float32 [Hq, L]): bias[h, min(n, L - 1)]
-    is added to the scaled score of the key n positions back.  A
-    block-table entry that names no page of the pool is not followed: page 0 is read instead and ``error_flag``
+    is added to the scaled score of the key n positions back.  ``keep`` > 0: a windowed query also sees the sequence's first
+    ``keep`` positions.  ``gate`` ([N, row], q's type): the result's element c of token n is multiplied by
+    sigmoid(gate[n, gate_column + c]).  A block-table entry that names no page of the pool is not followed: page 0 is read instead and ``error_flag``
     (default: the device's shared flag) is set to 5."""
     check(q, "q")
     tokens = positions.numel()
@@ -242,6 +244,7 @@ def attention_generic(q: torch.Tensor, q_stride: int, k_pages: torch.Tensor, v_p
         if sinks.numel() != n_q_heads:
             raise KernelError(f"sinks must hold one number per query head ({n_q_heads}), got {sinks.numel()}")
     _check_bias(bias, n_q_heads)
+    gate_pointer, gate_stride = _gate_rows(gate, gate_column, tokens, n_q_heads * value_dim, q.dtype)
     if out is None:
         out = torch.empty((tokens, n_q_heads * value_dim), dtype=q.dtype, device=q.device)
     check(out, "attention output", q.dtype, n_q_heads * value_dim)
@@ -249,9 +252,19 @@ def attention_generic(q: torch.Tensor, q_stride: int, k_pages: torch.Tensor, v_p
          block_tables.data_ptr(), block_tables.shape[-1], seq_of_token.data_ptr(), positions.data_ptr(),
          out.data_ptr(), tokens, n_q_heads, n_kv_heads, head_dim, value_dim, k_pages.shape[2], k_pages.shape[0],
          float(scale), int(window), pointer(sinks), int(chunk), pointer(bias), 0 if bias is None else bias.shape[1],
-         (error_flag if error_flag is not None else wait_error_flag(q.device)).data_ptr(), dtype_code(q.dtype),
+         int(keep) if window else 0, gate_pointer, gate_stride, (error_flag if error_flag is not None else wait_error_flag(q.device)).data_ptr(), dtype_code(q.dtype),
          stream_handle())
     return out
+
+
+def _gate_rows(gate: Optional[torch.Tensor], column: int, tokens: int, width: int, dtype: torch.dtype):
+    """(address of the first token's gate, elements from one token's to the next's) of an output gate, or (0, 0)."""
+    if gate is None:
+        return 0, 0
+    check(gate, "output gate", dtype)
+    if gate.dim() != 2 or gate.shape[0] != tokens or column < 0 or column + width > gate.shape[1]:
+        raise KernelError(f"an output gate of {width} columns from column {column} does not lie in {tuple(gate.shape)} for {tokens} tokens")
+    return gate.data_ptr() + int(column) * gate.element_size(), int(gate.shape[1])
 
 
 def _check_bias(bias: Optional[torch.Tensor], n_q_heads: int) -> None:
@@ -1240,12 +1253,13 @@ def attention(qkv: torch.Tensor, batch, block_tables: torch.Tensor, k_pages: tor
               n_q_heads: int, n_kv_heads: int, head_dim: int, scale: float, window: int = 0,
               value_dim: Optional[int] = None, sinks: Optional[torch.Tensor] = None, precise: bool = False,
               q_stride: Optional[int] = None, chunk: int = 0, bias: Optional[torch.Tensor] = None,
-              bias_log2: Optional[torch.Tensor] = None) -> torch.Tensor:
+              bias_log2: Optional[torch.Tensor] = None, keep: int = 0, gate: Optional[torch.Tensor] = None,
+              gate_column: int = 0) -> torch.Tensor:
     """Attention of a step's tokens over the paged cache; ``qkv`` is the packed projection whose Q
     heads have been normalised and rotated in place (``q_stride``: elements from one token's queries to the next's,
     where they are not such a packed row).  Chooses the kernel by dtype, head size and the
     shape of the batch; every choice computes the same function.  ``value_dim`` (default: head_dim) and ``sinks``,
-    ``chunk`` and ``bias`` as in ``attention_generic``; ``bias_log2``: the bias times log2(e), which the tensor-core kernels
+    ``chunk``, ``bias``, ``keep`` and ``gate`` as in ``attention_generic``; ``bias_log2``: the bias times log2(e), which the tensor-core kernels
     take (made here when it is not given).  ``precise``: the attention weights may not be rounded to bfloat16 on their way into the
     P V product (the tensor-core kernels then carry each as two bfloat16 numbers)."""
     value_dim = head_dim if value_dim is None else int(value_dim)
@@ -1253,17 +1267,19 @@ def attention(qkv: torch.Tensor, batch, block_tables: torch.Tensor, k_pages: tor
         q_stride = (n_q_heads + n_kv_heads) * head_dim + n_kv_heads * value_dim
     if qkv.dtype == torch.bfloat16:
         from . import attention_bf16
-        if value_dim == head_dim and sinks is None and not precise and not chunk and bias is None:
+        if value_dim == head_dim and sinks is None and not precise and not chunk and bias is None and not keep and gate is None:
             result = attention_bf16.try_attention(qkv, q_stride, batch, block_tables, k_pages, v_pages, n_q_heads,
                                                   n_kv_heads, head_dim, scale, window)
         else:
             result = attention_bf16.try_attention_precise(qkv, q_stride, batch, block_tables, k_pages, v_pages, n_q_heads,
                                                           n_kv_heads, head_dim, value_dim, scale, window, sinks, chunk,
-                                                          bias_log2 if bias_log2 is not None or bias is None else bias * LOG2E)
+                                                          bias_log2 if bias_log2 is not None or bias is None else bias * LOG2E,
+                                                          keep, gate, gate_column)
         if result is not None:
             return result
     return attention_generic(qkv, q_stride, k_pages, v_pages, block_tables, batch.seq_of_token, batch.positions,
-                             n_q_heads, n_kv_heads, head_dim, scale, window, value_dim=value_dim, sinks=sinks, chunk=chunk, bias=bias)
+                             n_q_heads, n_kv_heads, head_dim, scale, window, value_dim=value_dim, sinks=sinks, chunk=chunk, bias=bias,
+                             keep=keep, gate=gate, gate_column=gate_column)
 
 
 LOG2E = 1.4426950408889634

@@ -194,12 +194,20 @@ PRECISE_PREFILL_KERNEL = os.environ.get("LLMSERVER_B200_PRECISE_PREFILL", "tcgen
 PRECISE_DECODE_BLOCKS_PER_SM = int(os.environ.get("LLMSERVER_B200_PRECISE_DECODE_BLOCKS", "3"))
 
 
+def key_span(window, chunk, keep=0):
+    """The most keys a query walks where a window or a chunk bounds them (kept keys in whole tiles), else None."""
+    if chunk:
+        return int(chunk)
+    return int(window) + -(-int(keep) // TILE) * TILE if window else None
+
+
 def try_attention_precise(qkv, q_stride, batch, block_tables, k_pages, v_pages, n_q_heads, n_kv_heads, head_dim, value_dim,
-                          scale, window, sinks, chunk=0, bias_log2=None):
+                          scale, window, sinks, chunk=0, bias_log2=None, keep=0, gate=None, gate_column=0):
     """The tensor-core kernels in the form that keeps attention weights at 16 significant bits through the P V product,
     takes value heads of another size than key heads and adds exp(sinks[h]) to each softmax denominator; with ``chunk`` a
     query sees the keys of its own chunk of positions, with ``bias_log2`` (float32 [Hq, distances], times log2(e)) scores get
-    a bias by distance.  None when the sizes are not ones it takes (64 or 128 each)."""
+    a bias by distance; with ``keep`` a windowed query also sees the first ``keep`` positions; ``gate`` ([N, row], from
+    ``gate_column`` on): its sigmoid multiplies the results.  None when the sizes are not ones it takes (64 or 128 each)."""
     if not library().llm_attention_mma_sinks_supports(head_dim, value_dim, n_q_heads, n_kv_heads):
         return None
     check(qkv, "qkv", torch.bfloat16)
@@ -216,7 +224,10 @@ def try_attention_precise(qkv, q_stride, batch, block_tables, k_pages, v_pages, 
     # and splits without the cluster's bound keep more bytes in flight
     run_portions, tiles, run_decode, split_len, max_splits = plan(batch, n_q_heads // n_kv_heads, n_kv_heads, qkv.device,
                                                                   blocks_per_sm=PRECISE_DECODE_BLOCKS_PER_SM, cluster=False,
-                                                                  span=int(chunk) or None)
+                                                                  span=key_span(window, chunk, keep))
+    from . import _gate_rows
+    gate_pointer, gate_stride = _gate_rows(gate, gate_column, batch.n_tokens, n_q_heads * value_dim, torch.bfloat16)
+    keep = int(keep) if window else 0
     out = torch.empty((batch.n_tokens, n_q_heads * value_dim), dtype=torch.bfloat16, device=qkv.device)
     partial_out = partial_ml = None
     if run_decode and max_splits > 1:
@@ -228,7 +239,7 @@ def try_attention_precise(qkv, q_stride, batch, block_tables, k_pages, v_pages, 
             batch.scratch[key] = scratch
         partial_out, partial_ml = scratch
     page_size = k_pages.shape[2]
-    if run_portions and value_dim == head_dim and PRECISE_PREFILL_KERNEL == "tcgen05" and \
+    if run_portions and value_dim == head_dim and PRECISE_PREFILL_KERNEL == "tcgen05" and gate_pointer % 16 == 0 and gate_stride % 8 == 0 and \
             (bias_log2 is None or library().llm_attention_prefill_tcgen05_bias_fits(bias_log2.shape[1], n_q_heads // n_kv_heads)) and \
             prefill_tcgen05_supported(head_dim, n_q_heads, n_kv_heads, page_size):
         # prompt portions on the 128-row tcgen05 kernel in its form with two-part weights; single tokens, if any, below
@@ -245,7 +256,7 @@ def try_attention_precise(qkv, q_stride, batch, block_tables, k_pages, v_pages, 
              out.data_ptr(), batch.n_seqs, n_q_heads, n_kv_heads, head_dim, page_size, k_pages.shape[0], float(scale), int(window),
              int(run_decode), int(pairing), paired if pairing else sum(tile_counts), wait_error_flag(qkv.device).data_ptr(),
              0 if sinks is None else sinks.data_ptr(), int(chunk), 0 if bias_log2 is None else bias_log2.data_ptr(),
-             0 if bias_log2 is None else bias_log2.shape[1], stream_handle())
+             0 if bias_log2 is None else bias_log2.shape[1], keep, gate_pointer, gate_stride, stream_handle())
         run_portions = False
         if not run_decode:
             return out
@@ -253,7 +264,7 @@ def try_attention_precise(qkv, q_stride, batch, block_tables, k_pages, v_pages, 
          block_tables.shape[-1], batch.q_start.data_ptr(), batch.context_len.data_ptr(), out.data_ptr(), batch.n_seqs,
          n_q_heads, n_kv_heads, head_dim, value_dim, k_pages.shape[2], k_pages.shape[0], float(scale), int(window),
          0 if sinks is None else sinks.data_ptr(), int(chunk), 0 if bias_log2 is None else bias_log2.data_ptr(),
-         0 if bias_log2 is None else bias_log2.shape[1], int(run_portions), tiles, int(run_decode), split_len, max_splits,
+         0 if bias_log2 is None else bias_log2.shape[1], keep, gate_pointer, gate_stride, int(run_portions), tiles, int(run_decode), split_len, max_splits,
          0 if partial_out is None else partial_out.data_ptr(), 0 if partial_ml is None else partial_ml.data_ptr(),
          wait_error_flag(qkv.device).data_ptr(), stream_handle())
     return out

@@ -29,7 +29,7 @@ SIGNATURES = {
     "llm_sample": [_P, _P, _P, _P, _P, _I, _I, _P, _P, _S],
     "llm_sample_slices": [_I, _I],
     "llm_qk_norm_rope_kv_write": [_P, _P, _P, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _P, _I, _I, _I, _I, _S],
-    "llm_attention_generic": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _I, _P, _I, _P, _I, _S],
+    "llm_attention_generic": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _I, _P, _I, _I, _P, _I, _P, _I, _S],
     "llm_rope_kv_write_split": [_P, _P, _F, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _I, _I, _S],
     "llm_normed_add_rmsnorm": [_P, _P, _P, _F, _P, _P, _P, _P, _I, _I, _F, _I, _I, _I, _P, _S],
     "llm_norm_rope_units": [_P, _I, _P, _P, _P, _F, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _S],
@@ -62,11 +62,11 @@ SIGNATURES = {
     "llm_gemm_f32": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _S],
     "llm_attention_mma_supports": [_I, _I, _I],
     "llm_attention_mma_sinks_supports": [_I, _I, _I, _I],
-    "llm_attention_mma_sinks": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _P, _P, _P, _S],
+    "llm_attention_mma_sinks": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _I, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _P, _P, _P, _S],
     "llm_attention_prefill_tcgen05_supports": [_I, _I, _I, _I],
     "llm_attention_prefill_tcgen05": [_P, _I, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _I, _P, _S],
     "llm_attention_prefill_tcgen05_bias_fits": [_I, _I],
-    "llm_attention_prefill_tcgen05_precise": [_P, _I, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _I, _P, _P, _I, _P, _I, _S],
+    "llm_attention_prefill_tcgen05_precise": [_P, _I, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _I, _P, _P, _I, _P, _I, _I, _P, _I, _S],
     "llm_attention_prefill_wide_supports": [_I, _I, _I, _I],
     "llm_attention_prefill_wide": [_P, _I, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _I, _P, _S],
     "llm_gemm_small_m_supports": [_I, _I, _I],
