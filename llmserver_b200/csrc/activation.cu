@@ -6,6 +6,8 @@
 // With `group` > 0 the gate and up columns are interleaved in groups: columns [2 b group, 2 b group + group) hold the
 // gate values of outputs [b group, (b + 1) group) and the next `group` columns their up values (the layout in which a
 // 128-row tile of the fused gate/up weight holds 64 gate rows and their 64 up rows).
+//
+// `bias` (32-bit, one number per column of gate_up, in the same layout; may be null) joins gate and up before the activation.
 #include "common.cuh"
 
 // silu(x) * y in 32-bit.  For 16-bit activations the exponential and the reciprocal are the hardware
@@ -37,7 +39,7 @@ __device__ __forceinline__ int gate_column(int column, int group) {
 
 template <typename T, int ACT>
 __global__ void silu_mul_vec_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int intermediate,
-                                    size_t total_vectors, int group) {
+                                    size_t total_vectors, int group, const float* __restrict__ bias) {
     pdl_trigger();   // let the next kernel start launching
     pdl_wait();      // everything before this kernel in the stream is complete and visible
     constexpr int kCount = Vec16<T>::kCount;
@@ -58,6 +60,17 @@ __global__ void silu_mul_vec_kernel(const T* __restrict__ gate_up, T* __restrict
         Vec16<T>::load(src_v + to_up, up_v);
         Vec16<T>::load(src_w, gate_w);
         Vec16<T>::load(src_w + to_up, up_w);
+        if (bias) {
+            const float* bias_v = bias + gate_column(column_v, group);
+            const float* bias_w = bias + gate_column(column_w, group);
+#pragma unroll
+            for (int i = 0; i < kCount; ++i) {
+                gate_v[i] += bias_v[i];
+                up_v[i] += bias_v[to_up + i];
+                gate_w[i] += bias_w[i];
+                up_w[i] += bias_w[to_up + i];
+            }
+        }
 #pragma unroll
         for (int i = 0; i < kCount; ++i) result[i] = gate_times<T, ACT>(gate_v[i], up_v[i]);
         Vec16<T>::store(out + row_v * (size_t)intermediate + column_v, result);
@@ -70,21 +83,23 @@ __global__ void silu_mul_vec_kernel(const T* __restrict__ gate_up, T* __restrict
 }
 
 template <typename T, int ACT>
-__global__ void silu_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int intermediate, size_t total, int group) {
+__global__ void silu_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int intermediate, size_t total, int group,
+                                const float* __restrict__ bias) {
     pdl_trigger();   // let the next kernel start launching
     pdl_wait();      // everything before this kernel in the stream is complete and visible
     for (size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x; e < total; e += (size_t)gridDim.x * blockDim.x) {
         const size_t row = e / intermediate;
         const int column = (int)(e % intermediate);
-        const T* src = gate_up + row * 2 * (size_t)intermediate + gate_column(column, group);
-        const float gate = Num<T>::load(src);
-        const float up = Num<T>::load(src + (group > 0 ? group : intermediate));
+        const int from = gate_column(column, group), to_up = group > 0 ? group : intermediate;
+        const T* src = gate_up + row * 2 * (size_t)intermediate + from;
+        const float gate = Num<T>::load(src) + (bias ? bias[from] : 0.0f);
+        const float up = Num<T>::load(src + to_up) + (bias ? bias[from + to_up] : 0.0f);
         Num<T>::store(out + e, ACT == GLU_GELU ? gelu_times<float>(gate, up) : gate / (1.0f + expf(-gate)) * up);
     }
 }
 
 template <int ACT>
-static int glu_launch(const void* gate_up, void* out, int n_rows, int intermediate, int group, int dtype, cudaStream_t stream) {
+static int glu_launch(const void* gate_up, void* out, int n_rows, int intermediate, int group, const float* bias, int dtype, cudaStream_t stream) {
     if (n_rows == 0 || intermediate == 0) return LLM_OK;
     if (group < 0 || (group > 0 && intermediate % group)) {
         llm_set_error("silu_mul / gelu_mul: the intermediate size %d is no multiple of the group %d", intermediate, group);
@@ -99,21 +114,23 @@ static int glu_launch(const void* gate_up, void* out, int n_rows, int intermedia
     if (blocks > 148 * 16) blocks = 148 * 16;
     if (vector_form) {
         LLM_DISPATCH_DTYPE(dtype, (llm_launch(silu_mul_vec_kernel<T, ACT>, (unsigned)blocks, threads, 0, stream,
-                                      (const T*)gate_up, (T*)out, intermediate, work, group)));
+                                      (const T*)gate_up, (T*)out, intermediate, work, group, bias)));
     } else {
         LLM_DISPATCH_DTYPE(dtype, (llm_launch(silu_mul_kernel<T, ACT>, (unsigned)blocks, threads, 0, stream,
-                                      (const T*)gate_up, (T*)out, intermediate, work, group)));
+                                      (const T*)gate_up, (T*)out, intermediate, work, group, bias)));
     }
     return llm_check_launch(ACT == GLU_GELU ? "gelu_mul" : "silu_mul");
 }
 
-LLM_EXPORT int llm_silu_mul(const void* gate_up, void* out, int n_rows, int intermediate, int group, int dtype, cudaStream_t stream) {
-    return glu_launch<GLU_SILU>(gate_up, out, n_rows, intermediate, group, dtype, stream);
+LLM_EXPORT int llm_silu_mul(const void* gate_up, void* out, int n_rows, int intermediate, int group, const float* bias, int dtype,
+                            cudaStream_t stream) {
+    return glu_launch<GLU_SILU>(gate_up, out, n_rows, intermediate, group, bias, dtype, stream);
 }
 
 // The same layouts with gelu (tanh form) in silu's place.
-LLM_EXPORT int llm_gelu_mul(const void* gate_up, void* out, int n_rows, int intermediate, int group, int dtype, cudaStream_t stream) {
-    return glu_launch<GLU_GELU>(gate_up, out, n_rows, intermediate, group, dtype, stream);
+LLM_EXPORT int llm_gelu_mul(const void* gate_up, void* out, int n_rows, int intermediate, int group, const float* bias, int dtype,
+                            cudaStream_t stream) {
+    return glu_launch<GLU_GELU>(gate_up, out, n_rows, intermediate, group, bias, dtype, stream);
 }
 
 // Point-wise steps that stand alone (32-bit arithmetic, one rounding on the store):

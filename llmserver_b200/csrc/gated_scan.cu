@@ -23,9 +23,10 @@ constexpr int kScanThreads = 64;
 constexpr int kAhead = 4;      // tokens fetched at a time
 
 struct ScanArgs {
-    float* z;                  // [N, 2 * width]; the local pass overwrites it
+    float* z;                  // unit u of token t: 2 * unit numbers from t * z_token + u * z_unit on; the local pass overwrites it
+    long long z_token, z_unit;
     const void* u;             // [N, width]
-    const float* gate_bias;    // [2 * width], laid out as a row of z
+    const float* gate_bias;    // [2 * width]: per unit the biases of its recurrence gates, then of its input gates
     const float* rate;         // [width]
     const void* y;             // rows of y_row elements, the width channels from y_column on
     int y_row, y_column;
@@ -115,8 +116,9 @@ __global__ void __launch_bounds__(kScanThreads) gated_scan_kernel(ScanArgs a) {
         begin += segment * a.segment;
         end = min(end, begin + a.segment);
     }
-    const int z_column = c / a.unit * 2 * a.unit + c % a.unit;      // the channel's recurrence gate; its input gate lies `unit` further
-    float* z = a.z + z_column;
+    // the channel's recurrence gate; its input gate lies `unit` further
+    const int bias_column = c / a.unit * 2 * a.unit + c % a.unit;
+    float* z = a.z + c / a.unit * a.z_unit + c % a.unit;
     const T* u = (const T*)a.u + c;
     const T* y = (const T*)a.y + a.y_column + c;
     T* out = (T*)a.out + c;
@@ -126,8 +128,8 @@ __global__ void __launch_bounds__(kScanThreads) gated_scan_kernel(ScanArgs a) {
     float S[V], product[V], rate[V], bias_r[V], bias_i[V], y_bias[V];
     if (MODE != SCAN_OUTPUT) {
         load_values<float, V>(a.rate + c, rate);
-        load_values<float, V>(a.gate_bias + z_column, bias_r);
-        load_values<float, V>(a.gate_bias + z_column + a.unit, bias_i);
+        load_values<float, V>(a.gate_bias + bias_column, bias_r);
+        load_values<float, V>(a.gate_bias + bias_column + a.unit, bias_i);
     }
     if (MODE != SCAN_LOCAL) load_values<float, V>(a.y_bias + c, y_bias);
 #pragma unroll
@@ -164,8 +166,8 @@ __global__ void __launch_bounds__(kScanThreads) gated_scan_kernel(ScanArgs a) {
 #pragma unroll
         for (int k = 0; k < kAhead; ++k) {
             const size_t t = (size_t)min(t0 + k, end - 1);
-            load_values<float, V>(z + t * 2 * a.width, zr[k]);
-            load_values<float, V>(z + t * 2 * a.width + a.unit, zi[k]);
+            load_values<float, V>(z + t * a.z_token, zr[k]);
+            load_values<float, V>(z + t * a.z_token + a.unit, zi[k]);
             if (MODE != SCAN_OUTPUT) load_values<T, V>(u + t * a.width, us[k]);
             if (MODE != SCAN_LOCAL) load_values<T, V>(y + t * a.y_row, ys[k]);
         }
@@ -189,8 +191,8 @@ __global__ void __launch_bounds__(kScanThreads) gated_scan_kernel(ScanArgs a) {
                 else result[v] = S[v] * gelu_tanh<FAST>(ys[k][v] + y_bias[v]);
             }
             if (MODE == SCAN_LOCAL) {
-                store_values<float, V>(z + t * 2 * a.width, zr[k]);
-                store_values<float, V>(z + t * 2 * a.width + a.unit, zi[k]);
+                store_values<float, V>(z + t * a.z_token, zr[k]);
+                store_values<float, V>(z + t * a.z_token + a.unit, zi[k]);
             } else {
                 store_values<T, V>(out + t * a.width, result);
             }
@@ -208,7 +210,7 @@ __global__ void __launch_bounds__(kScanThreads) gated_scan_kernel(ScanArgs a) {
 
 // segment 0: one pass.  Otherwise `segments` = ceil(longest / segment), summary: float [n_seqs, segments, width, 2], start: float
 // [n_seqs, width], and z is overwritten.
-LLM_EXPORT int llm_gated_scan(float* z, const void* u, const float* gate_bias, const float* rate, const void* y, int y_row, int y_column,
+LLM_EXPORT int llm_gated_scan(float* z, long long z_token, long long z_unit, const void* u, const float* gate_bias, const float* rate, const void* y, int y_row, int y_column,
                               const float* y_bias, float* state, const int* state_slots, const int* q_start, void* out, int n_seqs, int width,
                               int unit, int longest, int segment, int segments, void* summary, float* start, int dtype, cudaStream_t stream) {
     if (n_seqs == 0 || longest <= 0) return LLM_OK;
@@ -221,10 +223,10 @@ LLM_EXPORT int llm_gated_scan(float* z, const void* u, const float* gate_bias, c
         return LLM_REFUSED;
     }
     ScanArgs a;
-    a.z = z; a.u = u; a.gate_bias = gate_bias; a.rate = rate; a.y = y; a.y_row = y_row; a.y_column = y_column; a.y_bias = y_bias;
+    a.z = z; a.z_token = z_token; a.z_unit = z_unit; a.u = u; a.gate_bias = gate_bias; a.rate = rate; a.y = y; a.y_row = y_row; a.y_column = y_column; a.y_bias = y_bias;
     a.state = state; a.state_slots = state_slots; a.q_start = q_start; a.out = out; a.width = width; a.unit = unit;
     a.segment = segment; a.max_segments = segments; a.summary = (float2*)summary; a.start = start;
-    const bool by_four = unit % 4 == 0 && y_row % 4 == 0 && y_column % 4 == 0 && aligned16(z) && aligned16(u) && aligned16(gate_bias) &&
+    const bool by_four = unit % 4 == 0 && z_token % 4 == 0 && z_unit % 4 == 0 && y_row % 4 == 0 && y_column % 4 == 0 && aligned16(z) && aligned16(u) && aligned16(gate_bias) &&
                          aligned16(rate) && aligned16(y) && aligned16(y_bias) && aligned16(state) && aligned16(out) && aligned16(start);
     const int per_block = kScanThreads * (by_four ? 4 : 1);
     const dim3 grid((width + per_block - 1) / per_block, segment > 0 ? segments : 1, n_seqs);

@@ -15,9 +15,11 @@
 //                  g = min(gate, limit), u = clamp(up, -limit, limit), y = g * sigmoid(alpha * g) * (u + up_shift)
 //              computed in 32-bit and rounded once (an infinite limit, alpha 1 and up_shift 0 give silu(gate) * up).
 //              With `in_scale` pair p's input row is multiplied by in_scale[p] as it is read (32-bit): a routing
-//              weight that acts on what goes into an expert.  Read-once for steps of few tokens; prompts take the tiled
+//              weight that acts on what goes into an expert.  An expert without a gate has the output max(sum, 0)^2 instead
+//              (squared_relu).  A pair whose index names no matrix (an identity output of the router) is left out.  Read-once for steps of few tokens; prompts take the tiled
 //              kernels of moe_grouped.cu.
-//   combine    out[t] = sum_j weight[t, j] * down[t * top + j] (+ gate[t] * shared[t]) in 32-bit, slots in order.
+//   combine    out[t] = sum_j weight[t, j] * down[t * top + j] (+ gate[t] * shared[t]) in 32-bit, slots in order.  A router may
+//              have identity outputs behind its experts: a pair that chose one contributes the token's own row x[t].
 #include "common.cuh"
 
 #define MOE_MAX_TOP 1024
@@ -170,10 +172,11 @@ __device__ __forceinline__ float gated_activation(float gate, float up, float li
 template <typename T, typename O, bool GATED>
 __global__ void indexed_linear_kernel(const T* __restrict__ in, const T* __restrict__ weight, const int* __restrict__ index,
                                       O* __restrict__ out, int rows, int inner, int in_div, float limit, float alpha, int index_mod,
-                                      const float* __restrict__ in_scale, float up_shift) {
+                                      const float* __restrict__ in_scale, float up_shift, int squared_relu, int n_matrices) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float in_row[];       // [inner]
+    if (index && (unsigned)index[blockIdx.x] >= (unsigned)n_matrices) return;
     const int pair = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
     const T* src = in + (size_t)(pair / in_div) * inner;
     const float row_scale = in_scale ? in_scale[pair] : 1.0f;
@@ -221,7 +224,8 @@ __global__ void indexed_linear_kernel(const T* __restrict__ in, const T* __restr
         const float total = warp_sum(sum[q]);
         const float total_up = GATED ? warp_sum(sum_up[q]) : 0.0f;
         if (lane == 0 && r0 + q < rows) {
-            const float value = GATED ? gated_activation(total, total_up, limit, alpha, up_shift) : total;
+            float value = GATED ? gated_activation(total, total_up, limit, alpha, up_shift) : total;
+            if (!GATED && squared_relu) value = fmaxf(value, 0.0f) * fmaxf(value, 0.0f);
             Num<O>::store(out + (size_t)pair * rows + r0 + q, value);
         }
     }
@@ -229,7 +233,8 @@ __global__ void indexed_linear_kernel(const T* __restrict__ in, const T* __restr
 
 template <typename T>
 __global__ void moe_combine_kernel(const float* __restrict__ down, const float* __restrict__ weights, const T* __restrict__ shared_out,
-                                   const float* __restrict__ shared_gate, T* __restrict__ out, int width, int top, size_t total) {
+                                   const float* __restrict__ shared_gate, T* __restrict__ out, int width, int top, size_t total,
+                                   const int* __restrict__ chosen, int experts, const T* __restrict__ x) {
     pdl_trigger();
     pdl_wait();
     for (size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x; e < total; e += (size_t)gridDim.x * blockDim.x) {
@@ -237,7 +242,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ down, const float* 
         const int column = (int)(e % width);
         float sum = 0.0f;
         for (int j = 0; j < top; ++j)
-            sum = fmaf(weights[token * top + j], down[(token * top + j) * width + column], sum);
+            sum = fmaf(weights[token * top + j], x && chosen[token * top + j] >= experts ? Num<T>::load(x + e) : down[(token * top + j) * width + column], sum);
         if (shared_out) sum = fmaf(shared_gate ? shared_gate[token] : 1.0f, Num<T>::load(shared_out + e), sum);
         Num<T>::store(out + e, sum);
     }
@@ -344,8 +349,13 @@ LLM_EXPORT int llm_moe_select(const float* logits, const float* correction, int*
 
 LLM_EXPORT int llm_indexed_linear(const void* in, const void* weight, const int* index, void* out, int n_pairs, int rows,
                                   int inner, int in_div, int gated, float limit, float alpha, int dtype, int out_f32,
-                                  int index_mod, const float* in_scale, float up_shift, cudaStream_t stream) {
+                                  int index_mod, const float* in_scale, float up_shift, int squared_relu, int n_matrices,
+                                  cudaStream_t stream) {
     if (n_pairs == 0 || rows == 0) return LLM_OK;
+    if (index && n_matrices <= 0) {
+        llm_set_error("indexed_linear: an index over %d matrices", n_matrices);
+        return LLM_REFUSED;
+    }
     if (in_div <= 0 || inner <= 0) {
         llm_set_error("indexed_linear: in_div %d and inner %d must be positive", in_div, inner);
         return LLM_REFUSED;
@@ -368,7 +378,7 @@ LLM_EXPORT int llm_indexed_linear(const void* in, const void* weight, const int*
             if (status != LLM_OK) return status;                                                                        \
         }                                                                                                               \
         llm_launch(indexed_linear_kernel<T, O, GATED>, grid, warps * 32, shared, stream, (const T*)in, (const T*)weight, index, \
-                   (O*)out, rows, inner, in_div, limit, alpha, index_mod, in_scale, up_shift);                                  \
+                   (O*)out, rows, inner, in_div, limit, alpha, index_mod, in_scale, up_shift, squared_relu, n_matrices);        \
     } while (0)
     LLM_DISPATCH_DTYPE(dtype, {
         if (gated && out_f32) {
@@ -384,13 +394,17 @@ LLM_EXPORT int llm_indexed_linear(const void* in, const void* weight, const int*
 }
 
 LLM_EXPORT int llm_moe_combine(const float* down, const float* weights, const void* shared_out, const float* shared_gate, void* out, int n_tokens,
-                               int width, int top, int dtype, cudaStream_t stream) {
+                               int width, int top, const int* chosen, int experts, const void* x, int dtype, cudaStream_t stream) {
     if (n_tokens == 0) return LLM_OK;
+    if (x && !chosen) {
+        llm_set_error("moe_combine: identity outputs need the choices");
+        return LLM_REFUSED;
+    }
     const size_t total = (size_t)n_tokens * width;
     size_t blocks = (total + 255) / 256;
     if (blocks > 148 * 16) blocks = 148 * 16;
     LLM_DISPATCH_DTYPE(dtype, (llm_launch(moe_combine_kernel<T>, (unsigned)blocks, 256, 0, stream, down, weights,
-                                  (const T*)shared_out, shared_gate, (T*)out, width, top, total)));
+                                  (const T*)shared_out, shared_gate, (T*)out, width, top, total, chosen, experts, (const T*)x)));
     return llm_check_launch("moe_combine");
 }
 

@@ -12,7 +12,11 @@
 //            its up rows and a tile takes 64 features' gate rows and the same features' up rows in alternating
 //            groups of eight, so that a thread holds both halves of an output and writes
 //                min(g, limit) * sigmoid(alpha * min(g, limit)) * (clamp(u, -limit, limit) + 1)
-//            rounded once to bfloat16; and *plain*, which writes the 32-bit sums.
+//            rounded once to bfloat16; and *plain*, which writes the 32-bit sums, or, for experts without a gate, max(sum,
+//            0)^2 rounded once to bfloat16 (*squared relu*).
+//
+// A router may have identity outputs behind its experts: pairs that chose one (an expert number beyond the last) get no row
+// (row_of_pair -1), the rows left over at the end belong to no tile, and the weighted sum takes the token's own row instead.
 #include "common.cuh"
 
 namespace {
@@ -55,7 +59,8 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const int* __restrict__ 
     int* start = plan_shared + experts;
     for (int e = threadIdx.x; e < experts; e += blockDim.x) count[e] = 0;
     __syncthreads();
-    for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) atomicAdd(count + chosen[p], 1);
+    for (int p = threadIdx.x; p < n_pairs; p += blockDim.x)
+        if (chosen[p] < experts) atomicAdd(count + chosen[p], 1);
     __syncthreads();
     if (threadIdx.x == 0) {
         int total = 0, tile = 0;
@@ -78,13 +83,20 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const int* __restrict__ 
     __syncthreads();
     for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
         const int e = chosen[p];
+        if (e >= experts) {
+            row_of_pair[p] = -1;
+            continue;
+        }
         const int row = start[e] + atomicAdd(count + e, 1);
         pair_of_row[row] = p;
         row_of_pair[p] = row;
     }
+    // rows that no pair got: whoever walks all rows finds a pair that exists
+    for (int row = start[experts] + threadIdx.x; row < n_pairs; row += blockDim.x) pair_of_row[row] = 0;
 }
 
-template <bool GATED>
+enum : int { FORM_PLAIN = 0, FORM_GATED = 1, FORM_SQUARED_RELU = 2 };
+template <int FORM>
 __global__ void __launch_bounds__(kGemmThreads) moe_grouped_kernel(const __nv_bfloat16* __restrict__ a, const __nv_bfloat16* __restrict__ w,
                                                                    const int* __restrict__ tiles, const int* __restrict__ pair_of_row,
                                                                    int in_div, void* __restrict__ out, int out_cols, int inner,
@@ -92,6 +104,7 @@ __global__ void __launch_bounds__(kGemmThreads) moe_grouped_kernel(const __nv_bf
     pdl_trigger();
     pdl_wait();
     if ((int)blockIdx.x >= tiles[0]) return;
+    constexpr bool GATED = FORM == FORM_GATED;
     extern __shared__ __align__(128) unsigned char grouped_shared[];
     __nv_bfloat16* a_tiles = reinterpret_cast<__nv_bfloat16*>(grouped_shared);                   // [stages][128][64]
     __nv_bfloat16* w_tiles = a_tiles + kStages * kBlockRows * kBlockInner;                        // [stages][128][64]
@@ -212,6 +225,15 @@ __global__ void __launch_bounds__(kGemmThreads) moe_grouped_kernel(const __nv_bf
                         dst[feature] = __float2bfloat16_rn(y[0]);
                     }
                 }
+            } else if (FORM == FORM_SQUARED_RELU) {
+                __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(out) + out_row * out_cols;
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const int column = col0 + warp_col + j * 8 + 2 * t;      // columns come in eights
+                    if (column + 1 >= out_cols) continue;
+                    const float y0 = fmaxf(acc[i][j][2 * half], 0.0f), y1 = fmaxf(acc[i][j][2 * half + 1], 0.0f);
+                    *reinterpret_cast<__nv_bfloat162*>(dst + column) = __floats2bfloat162_rn(y0 * y0, y1 * y1);
+                }
             } else {
                 float* dst = reinterpret_cast<float*>(out) + out_row * out_cols;
 #pragma unroll
@@ -232,7 +254,8 @@ __global__ void __launch_bounds__(kGemmThreads) moe_grouped_kernel(const __nv_bf
 template <typename T>
 __global__ void moe_combine_rows_kernel(const float* __restrict__ down, const int* __restrict__ row_of_pair,
                                         const float* __restrict__ weights, const T* __restrict__ shared_out,
-                                        const float* __restrict__ shared_gate, T* __restrict__ out, int width, int top) {
+                                        const float* __restrict__ shared_gate, T* __restrict__ out, int width, int top,
+                                        const T* __restrict__ x) {
     pdl_trigger();
     pdl_wait();
     const size_t token = blockIdx.x;
@@ -241,7 +264,14 @@ __global__ void moe_combine_rows_kernel(const float* __restrict__ down, const in
         float sum[4] = {0.0f, 0.0f, 0.0f, 0.0f};
         for (int j = 0; j < top; ++j) {
             const float weight = weights[token * top + j];
-            const float4 value = *reinterpret_cast<const float4*>(down + (size_t)row_of_pair[token * top + j] * width + column);
+            const int row = row_of_pair[token * top + j];
+            float4 value;
+            if (row < 0) {      // an identity output
+                const T* own = x + token * width + column;
+                value = make_float4(Num<T>::load(own), Num<T>::load(own + 1), Num<T>::load(own + 2), Num<T>::load(own + 3));
+            } else {
+                value = *reinterpret_cast<const float4*>(down + (size_t)row * width + column);
+            }
             sum[0] = fmaf(weight, value.x, sum[0]);
             sum[1] = fmaf(weight, value.y, sum[1]);
             sum[2] = fmaf(weight, value.z, sum[2]);
@@ -280,10 +310,12 @@ LLM_EXPORT int llm_moe_grouped_supports(int out_cols, int inner, int gated) {
 
 // One product over all tiles of the plan.  a: bfloat16 [*, inner]; w: bfloat16 [experts, (gated ? 2 : 1) * out_cols,
 // inner]; pair_of_row null: row r of the plan reads row r of a, else row pair_of_row[r] / in_div; out: bfloat16
-// [n_pairs, out_cols] (gated) or float32 [n_pairs, out_cols], rows in the plan's order.
+// [n_pairs, out_cols] (gated, squared relu) or float32 [n_pairs, out_cols], rows in the plan's order.  `form`: 0 plain, 1
+// gated, 2 squared relu.
 LLM_EXPORT int llm_moe_grouped(const void* a, const void* w, const int* tiles, const int* pair_of_row, int in_div, void* out,
-                               int out_cols, int inner, int max_tiles, int gated, float limit, float alpha, float up_shift, cudaStream_t stream) {
+                               int out_cols, int inner, int max_tiles, int form, float limit, float alpha, float up_shift, cudaStream_t stream) {
     if (max_tiles <= 0) return LLM_OK;
+    const bool gated = form == FORM_GATED;
     if (!llm_moe_grouped_supports(out_cols, inner, gated) || in_div <= 0) {
         llm_set_error("moe_grouped: %d output columns over an inner size of %d are not supported (inner a multiple of %d, "
                       "columns a multiple of 8)", out_cols, inner, kBlockInner);
@@ -296,26 +328,28 @@ LLM_EXPORT int llm_moe_grouped(const void* a, const void* w, const int* tiles, c
         llm_set_error("moe_grouped: %d output columns are too many for one launch", out_cols);
         return LLM_REFUSED;
     }
-    if (gated) {
-        if (int status = llm_raise_shared_limit((const void*)moe_grouped_kernel<true>, shared, "moe_grouped")) return status;
-        llm_launch(moe_grouped_kernel<true>, grid, kGemmThreads, shared, stream, (const __nv_bfloat16*)a, (const __nv_bfloat16*)w,
-                   tiles, pair_of_row, in_div, out, out_cols, inner, limit, alpha, up_shift);
-    } else {
-        if (int status = llm_raise_shared_limit((const void*)moe_grouped_kernel<false>, shared, "moe_grouped")) return status;
-        llm_launch(moe_grouped_kernel<false>, grid, kGemmThreads, shared, stream, (const __nv_bfloat16*)a, (const __nv_bfloat16*)w,
-                   tiles, pair_of_row, in_div, out, out_cols, inner, limit, alpha, up_shift);
-    }
+#define LLM_GROUPED(FORM)                                                                                                              \
+    do {                                                                                                                               \
+        if (int status = llm_raise_shared_limit((const void*)moe_grouped_kernel<FORM>, shared, "moe_grouped")) return status;           \
+        llm_launch(moe_grouped_kernel<FORM>, grid, kGemmThreads, shared, stream, (const __nv_bfloat16*)a, (const __nv_bfloat16*)w,       \
+                   tiles, pair_of_row, in_div, out, out_cols, inner, limit, alpha, up_shift);                                          \
+    } while (0)
+    if (gated) LLM_GROUPED(FORM_GATED);
+    else if (form == FORM_SQUARED_RELU) LLM_GROUPED(FORM_SQUARED_RELU);
+    else LLM_GROUPED(FORM_PLAIN);
+#undef LLM_GROUPED
     return llm_check_launch("moe_grouped");
 }
 
 LLM_EXPORT int llm_moe_combine_rows(const float* down, const int* row_of_pair, const float* weights, const void* shared_out,
-                                    const float* shared_gate, void* out, int n_tokens, int width, int top, int dtype, cudaStream_t stream) {
+                                    const float* shared_gate, void* out, int n_tokens, int width, int top, const void* x, int dtype,
+                                    cudaStream_t stream) {
     if (n_tokens == 0) return LLM_OK;
     if (width % 4) {
         llm_set_error("moe_combine_rows: the width %d is no multiple of 4", width);
         return LLM_REFUSED;
     }
     LLM_DISPATCH_DTYPE(dtype, (llm_launch(moe_combine_rows_kernel<T>, n_tokens, 256, 0, stream, down, row_of_pair, weights,
-                                  (const T*)shared_out, shared_gate, (T*)out, width, top)));
+                                  (const T*)shared_out, shared_gate, (T*)out, width, top, (const T*)x)));
     return llm_check_launch("moe_combine_rows");
 }

@@ -12,7 +12,8 @@
 //   gated   B = 128 gate rows and the same features' 128 up rows: a thread finds gate and up of an output in columns
 //           j and 128 + j of its own row and writes  min(g, limit) * sigmoid(alpha * min(g, limit)) * (clamp(u) + 1)
 //           rounded once to bfloat16;
-//   plain   B = 256 rows; the 32-bit sums are written as they are.
+//   plain   B = 256 rows; the 32-bit sums are written as they are;
+//   squared relu    B = 256 rows; max(sum, 0)^2 rounded once to bfloat16 (experts without a gate).
 //
 // Waits are bounded: a wait that runs out sets error code 7 in the flag, every role leaves its loop, nothing is
 // stored and the tensor memory is freed.
@@ -29,7 +30,8 @@ constexpr int kRing = 4;
 constexpr uint32_t kABytes = kRows * kInner * 2, kBBytes = kCols * kInner * 2, kStageBytes = kABytes + kBBytes;
 constexpr int kTcThreads = 192;      // warp 0: copies, warp 1: MMA issue and tensor memory, warps 2-5: epilogue
 
-template <bool GATED>
+enum : int { FORM_PLAIN = 0, FORM_GATED = 1, FORM_SQUARED_RELU = 2 };
+template <int FORM>
 __global__ void __launch_bounds__(kTcThreads) moe_grouped_tc_kernel(const __grid_constant__ CUtensorMap map_a,
                                                                     const __grid_constant__ CUtensorMap map_w,
                                                                     const int* __restrict__ tiles, void* __restrict__ out, int out_cols,
@@ -37,6 +39,7 @@ __global__ void __launch_bounds__(kTcThreads) moe_grouped_tc_kernel(const __grid
                                                                     float up_shift, int* __restrict__ error_flag) {
     pdl_trigger();
     pdl_wait();
+    constexpr bool GATED = FORM == FORM_GATED;
     const int total = tiles[0] * col_tiles;      // (row tile, column tile) pairs; block b takes b, b + gridDim.x, ...
     if ((int)blockIdx.x >= total) return;
     extern __shared__ unsigned char tc_shared_raw[];
@@ -163,6 +166,26 @@ __global__ void __launch_bounds__(kTcThreads) moe_grouped_tc_kernel(const __grid
                         *reinterpret_cast<uint4*>(dst + feature) = make_uint4(packed[0], packed[1], packed[2], packed[3]);
                     }
                 }
+            } else if (FORM == FORM_SQUARED_RELU) {
+                __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(out) + out_row * out_cols;
+#pragma unroll 1
+                for (int j = 0; j < kCols; j += 32) {
+                    uint32_t sums[32];
+                    tc5::tmem_load_32(address + j, sums);
+                    if (!store) continue;
+#pragma unroll
+                    for (int v = 0; v < 32; v += 8) {
+                        const int column = col0 + j + v;
+                        if (column + 8 > out_cols) break;       // out_cols is a multiple of 8
+                        uint32_t packed[4];
+#pragma unroll
+                        for (int e = 0; e < 8; e += 2) {
+                            const float y0 = fmaxf(__uint_as_float(sums[v + e]), 0.0f), y1 = fmaxf(__uint_as_float(sums[v + e + 1]), 0.0f);
+                            packed[e / 2] = tc5::pack2(y0 * y0, y1 * y1);
+                        }
+                        *reinterpret_cast<uint4*>(dst + column) = make_uint4(packed[0], packed[1], packed[2], packed[3]);
+                    }
+                }
             } else {
                 float* dst = reinterpret_cast<float*>(out) + out_row * out_cols;
 #pragma unroll 1
@@ -237,11 +260,12 @@ LLM_EXPORT int llm_moe_gather_rows(const void* x, const int* pair_of_row, int in
 }
 
 // a: bfloat16 [n_rows, inner] in the plan's order; w: bfloat16 [experts, (gated ? 2 : 1) * out_cols, inner]; out: bfloat16
-// [n_rows, out_cols] (gated) or float32 [n_rows, out_cols].
+// [n_rows, out_cols] (gated, squared relu) or float32 [n_rows, out_cols].  `form`: 0 plain, 1 gated, 2 squared relu.
 LLM_EXPORT int llm_moe_grouped_tc(const void* a, int n_rows, const void* w, int experts, const int* tiles, void* out, int out_cols,
-                                  int inner, int max_tiles, int gated, float limit, float alpha, float up_shift, int* error_flag,
+                                  int inner, int max_tiles, int form, float limit, float alpha, float up_shift, int* error_flag,
                                   cudaStream_t stream) {
     if (max_tiles <= 0 || n_rows <= 0) return LLM_OK;
+    const bool gated = form == FORM_GATED;
     if (!llm_moe_grouped_tc_supports(out_cols, inner, gated) || !aligned16(a) || !aligned16(w) || !aligned16(out)) {
         llm_set_error("moe_grouped_tc: %d output columns over an inner size of %d are not supported (both multiples of 8, "
                       "16-byte aligned operands)", out_cols, inner);
@@ -263,14 +287,15 @@ LLM_EXPORT int llm_moe_grouped_tc(const void* a, int n_rows, const void* w, int 
     cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device);
     long long most = (long long)max_tiles * col_tiles;
     const int blocks = (int)(most < sms ? most : sms);
-    if (gated) {
-        if (int status = llm_raise_shared_limit((const void*)moe_grouped_tc_kernel<true>, shared, "moe_grouped_tc")) return status;
-        llm_launch(moe_grouped_tc_kernel<true>, blocks, kTcThreads, shared, stream, map_a, map_w, tiles, out, out_cols, col_tiles, inner,
-                   limit, alpha, up_shift, error_flag);
-    } else {
-        if (int status = llm_raise_shared_limit((const void*)moe_grouped_tc_kernel<false>, shared, "moe_grouped_tc")) return status;
-        llm_launch(moe_grouped_tc_kernel<false>, blocks, kTcThreads, shared, stream, map_a, map_w, tiles, out, out_cols, col_tiles, inner,
-                   limit, alpha, up_shift, error_flag);
-    }
+#define LLM_GROUPED_TC(FORM)                                                                                                            \
+    do {                                                                                                                                \
+        if (int status = llm_raise_shared_limit((const void*)moe_grouped_tc_kernel<FORM>, shared, "moe_grouped_tc")) return status;      \
+        llm_launch(moe_grouped_tc_kernel<FORM>, blocks, kTcThreads, shared, stream, map_a, map_w, tiles, out, out_cols, col_tiles,       \
+                   inner, limit, alpha, up_shift, error_flag);                                                                          \
+    } while (0)
+    if (gated) LLM_GROUPED_TC(FORM_GATED);
+    else if (form == FORM_SQUARED_RELU) LLM_GROUPED_TC(FORM_SQUARED_RELU);
+    else LLM_GROUPED_TC(FORM_PLAIN);
+#undef LLM_GROUPED_TC
     return llm_check_launch("moe_grouped_tc");
 }

@@ -23,7 +23,7 @@ __all__ = ["KernelError", "embedding", "add_rmsnorm", "rmsnorm", "silu_mul", "sa
            "RowScaled", "StreamSink", "STREAM_ROWS", "unscaled_rows_supported", "norm_rope_units", "rotate_units", "attention_diff", "gla_supported",
            "gla_recurrent", "head_linear", "relu_squared", "tanh_narrow", "softcap_", "scaled_sum", "token_shift_mix",
            "short_conv_units", "matrix_recurrence_supported", "wkv_recurrent", "delta_rule_recurrent", "retention_recurrent", "ssd_recurrent", "decay_recurrence_supported",
-           "gelu_mul", "grouped_rmsnorm", "conv_norm_kv"]
+           "gelu_mul", "grouped_rmsnorm", "conv_norm_kv", "streams_norm", "unit_linear_wide", "gated_scan"]
 
 
 def embedding(table: torch.Tensor, ids: torch.Tensor, out: Optional[torch.Tensor] = None, scale: float = 1.0,
@@ -98,19 +98,20 @@ def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: Optional[tor
     return out
 
 
-def silu_mul(gate_up: torch.Tensor, out: Optional[torch.Tensor] = None, group: int = 0) -> torch.Tensor:
+def silu_mul(gate_up: torch.Tensor, out: Optional[torch.Tensor] = None, group: int = 0, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[n, i] = silu(gate_up[n, i]) * gate_up[n, I + i]; gate_up is [N, 2 I], gate half first.  With ``group`` > 0
     gate and up columns are interleaved in groups of that many: output i finds its gate value at column
-    (i // group) * 2 * group + i % group and its up value ``group`` columns further."""
-    return _glu("llm_silu_mul", gate_up, out, group)
+    (i // group) * 2 * group + i % group and its up value ``group`` columns further.  ``bias`` (float32 [2 I], in gate_up's
+    layout) joins both before the activation."""
+    return _glu("llm_silu_mul", gate_up, out, group, bias)
 
 
-def gelu_mul(gate_up: torch.Tensor, out: Optional[torch.Tensor] = None, group: int = 0) -> torch.Tensor:
+def gelu_mul(gate_up: torch.Tensor, out: Optional[torch.Tensor] = None, group: int = 0, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``silu_mul`` with gelu in its tanh form, 0.5 x (1 + tanh(sqrt(2 / pi) (x + 0.044715 x^3))), in silu's place."""
-    return _glu("llm_gelu_mul", gate_up, out, group)
+    return _glu("llm_gelu_mul", gate_up, out, group, bias)
 
 
-def _glu(launcher: str, gate_up: torch.Tensor, out: Optional[torch.Tensor], group: int) -> torch.Tensor:
+def _glu(launcher: str, gate_up: torch.Tensor, out: Optional[torch.Tensor], group: int, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     check(gate_up, "gate_up")
     rows, doubled = gate_up.shape
     if doubled % 2:
@@ -118,7 +119,9 @@ def _glu(launcher: str, gate_up: torch.Tensor, out: Optional[torch.Tensor], grou
     if out is None:
         out = torch.empty((rows, doubled // 2), dtype=gate_up.dtype, device=gate_up.device)
     check(out, "the activation's output", gate_up.dtype, doubled // 2)
-    call(launcher, gate_up.data_ptr(), out.data_ptr(), rows, doubled // 2, int(group), dtype_code(gate_up.dtype), stream_handle())
+    if bias is not None:
+        check(bias, "gate and up bias", torch.float32, doubled)
+    call(launcher, gate_up.data_ptr(), out.data_ptr(), rows, doubled // 2, int(group), pointer(bias), dtype_code(gate_up.dtype), stream_handle())
     return out
 
 
@@ -376,6 +379,54 @@ def scaled_add_rmsnorm(residual: torch.Tensor, a: torch.Tensor, scale_a: torch.T
     call("llm_scaled_add_rmsnorm", residual.data_ptr(), a.data_ptr(), scale_a.data_ptr(), pointer(b), pointer(scale_b),
          pointer(weight) if want_output else 0, pointer(out), pointer(rows), n_rows, width, float(eps), int(rows is None),
          dtype_code(act), dtype_code(weight.dtype if weight is not None else act), stream_handle())
+    return out
+
+
+def streams_norm(streams: torch.Tensor, parts: list, weight: Optional[torch.Tensor], eps: float, centre: bool, mix: Optional[torch.Tensor] = None,
+                 out_weight: Optional[torch.Tensor] = None, read: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
+                 act_dtype: Optional[torch.dtype] = None, want_output: bool = True) -> Optional[torch.Tensor]:
+    """On residual streams ``streams`` (float32 [N, S, H], or [N, H] for one): what the sub-layer behind left (``parts``, up to
+    two tuples (output [N, H], bias or None, RMS norm weight or None, its eps, scale); none: nothing is pending) is written,
+
+        y = sum_p scale_p * norm_p(part_p + bias_p);   x_t <- sum_s mix[s, t] x_s + out_weight[t] * y     (32-bit, in place)
+
+    and, unless ``want_output`` is False, the next sub-layer's input is returned in the activation type: norm(sum_t read[t] x_t) *
+    weight, a layer norm (``centre``: the mean is taken off) or an RMS norm.  ``mix`` [S, S] (from, to), ``out_weight`` and
+    ``read`` [S] are float32; absent they are the identity and ones.  With ``rows`` (int32) output row o comes from token
+    rows[o] and the streams are left as they were."""
+    check(streams, "streams", torch.float32)
+    width = streams.shape[-1]
+    count = streams.shape[1] if streams.dim() == 3 else 1
+    tokens = streams.numel() // (count * width)
+    if len(parts) > 2:
+        raise KernelError(f"streams_norm joins up to two outputs, not {len(parts)}")
+    act = act_dtype or (parts[0][0].dtype if parts else weight.dtype)
+    norm_weights = [weight] if want_output else []
+    described = []
+    for output, bias, norm_weight, norm_eps, scale in parts:
+        check(output, "sub-layer output", act, width)
+        if output.numel() != tokens * width:
+            raise KernelError(f"an output {tuple(output.shape)} does not belong to {tokens} rows of {width}")
+        if bias is not None:
+            check(bias, "output bias", torch.float32, width)
+        if norm_weight is not None:
+            norm_weights.append(norm_weight)
+        described += [output.data_ptr(), pointer(bias), pointer(norm_weight), float(norm_eps), float(scale)]
+    described += [0, 0, 0, 0.0, 1.0] * (2 - len(parts))
+    for tensor in norm_weights:
+        check(tensor, "norm weight", norm_weights[0].dtype, width)
+    for name, tensor, size in (("mix", mix, count * count), ("out weights", out_weight, count), ("read weights", read, count)):
+        if tensor is not None:
+            check(tensor, name, torch.float32)
+            if tensor.numel() != size:
+                raise KernelError(f"the {name} of {count} streams hold {size} numbers, not {tensor.numel()}")
+    if rows is not None:
+        check(rows, "rows", torch.int32)
+    n_rows = tokens if rows is None else rows.numel()
+    out = torch.empty((n_rows, width), dtype=act, device=streams.device) if want_output else None
+    call("llm_streams_norm", streams.data_ptr(), count, width, *described, pointer(mix), pointer(out_weight), pointer(read),
+         pointer(weight) if want_output else 0, float(eps), int(bool(centre)), pointer(out), pointer(rows), n_rows, dtype_code(act),
+         dtype_code(norm_weights[0].dtype if norm_weights else act), stream_handle())
     return out
 
 
@@ -942,6 +993,72 @@ def head_linear(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
 HEAD_LINEAR_ROWS = 32     # up to this many tokens a bfloat16 step multiplies row by row
 
 
+def unit_linear_wide(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
+    """``head_linear`` with 32-bit results, never rounded in between: ``x`` [N, U * K] in units of K channels, ``weight``
+    [U, R, K].  Returns float32 [N, U, R]; its strides depend on who made it (the library's batched product leaves units in
+    front of tokens)."""
+    check(x, "x")
+    units, rows, inner = weight.shape
+    check(weight, "per-unit matrices", x.dtype, inner)
+    tokens = x.shape[0]
+    if x.shape[1] != units * inner:
+        raise KernelError(f"x has {x.shape[1]} columns; {units} units of {inner} are {units * inner}")
+    if x.dtype == torch.bfloat16 and tokens > HEAD_LINEAR_ROWS:
+        return torch.bmm(x.view(tokens, units, inner).transpose(0, 1), weight.transpose(1, 2), out_dtype=torch.float32).transpose(0, 1)
+    return indexed_linear(x.view(tokens * units, inner), weight, None, tokens * units, out_dtype=torch.float32, cyclic=True).view(tokens, units, rows)
+
+
+SCAN_SEGMENT = 32          # fewest tokens per segment of the segmented gated scan
+SCAN_MAX_SEGMENTS = 128    # most segments per sequence
+
+
+def gated_scan(z: torch.Tensor, u: torch.Tensor, gate_bias: torch.Tensor, rate: torch.Tensor, y: torch.Tensor, y_column: int,
+               y_bias: torch.Tensor, state: torch.Tensor, batch, segment: Optional[int] = None) -> torch.Tensor:
+    """The real-gated linear recurrent unit, sequence by sequence, from and into each sequence's slot of ``state`` (float32
+    [slots, width]), per channel:
+
+        r = sigmoid(z_r + b_r), i = sigmoid(z_i + b_i);  a = exp(rate * r);  S <- a S + sqrt(1 - a^2) i u;  out = S * gelu_tanh(y + y_bias)
+
+    ``z`` float32 [N, U, 2 K] as ``unit_linear_wide`` leaves it: per unit of K channels the recurrence gates' pre-activations, then
+    the input gates' (overwritten by the segmented form); ``gate_bias`` float32 [U, 2 K]; ``rate`` and ``y_bias`` float32 [width];
+    ``u`` [N, width] and width columns of ``y`` from ``y_column`` in the activation type, in which the result [N, width] comes.
+
+    ``segment``: tokens per segment of the form that walks a long portion's segments in parallel (results equal to rounding).
+    None: chosen here for bfloat16 steps whose longest portion spans two segments; 0: the one-pass form, which is also what the
+    32-bit path runs."""
+    check(u, "u")
+    tokens, width = u.shape
+    units, doubled = z.shape[1], z.shape[2]
+    if z.dtype != torch.float32 or z.stride(2) != 1 or z.shape[0] != tokens or units * doubled != 2 * width:
+        raise KernelError(f"gate pre-activations {tuple(z.shape)} of {z.dtype} do not belong to {tokens} rows of {width} channels")
+    check(gate_bias, "gate biases", torch.float32, doubled)
+    check(rate, "decay rates", torch.float32, width)
+    check(y, "output gate", u.dtype)
+    if y_column < 0 or y_column + width > y.shape[1] or y.shape[0] != tokens or gate_bias.numel() != 2 * width:
+        raise KernelError(f"{width} columns from {y_column} do not lie in rows of {y.shape[1]}, or the gates have other biases")
+    check(y_bias, "output gate's bias", torch.float32, width)
+    check(state, "recurrent state", torch.float32, width)
+    out = torch.empty((tokens, width), dtype=u.dtype, device=u.device)
+    longest = int(batch.max_q_len)
+    if segment is None:
+        segment = 0 if u.dtype != torch.bfloat16 or longest < 2 * SCAN_SEGMENT else max(SCAN_SEGMENT, -(-longest // SCAN_MAX_SEGMENTS))
+    segments, summary, start = 0, None, None
+    if segment:
+        segments = -(-longest // int(segment))
+        key = ("gated_scan_segments", batch.n_seqs, segments, width)
+        scratch = batch.scratch.get(key)
+        if scratch is None:
+            scratch = (torch.empty((batch.n_seqs, segments, width, 2), dtype=torch.float32, device=u.device),
+                       torch.empty((batch.n_seqs, width), dtype=torch.float32, device=u.device))
+            batch.scratch[key] = scratch
+        summary, start = scratch
+    call("llm_gated_scan", z.data_ptr(), z.stride(0), z.stride(1), u.data_ptr(), gate_bias.data_ptr(), rate.data_ptr(), y.data_ptr(),
+         y.shape[1], int(y_column), y_bias.data_ptr(), state.data_ptr(), batch.state_slots.data_ptr(), batch.q_start.data_ptr(),
+         out.data_ptr(), batch.n_seqs, width, doubled // 2, longest, int(segment), segments, pointer(summary), pointer(start),
+         dtype_code(u.dtype), stream_handle())
+    return out
+
+
 def _route_rule(experts: int, scores: str, groups: Optional[tuple], renormalise: bool):
     """(softmax, groups, keep, renormalise) as the launchers take them."""
     if scores not in ("sigmoid", "softmax"):
@@ -1001,14 +1118,17 @@ def moe_select(logits: torch.Tensor, correction: Optional[torch.Tensor], top: in
 
 def indexed_linear(x: torch.Tensor, weight: torch.Tensor, index: Optional[torch.Tensor], pairs: int, in_div: int = 1,
                    gated: Optional[tuple] = None, out_dtype: Optional[torch.dtype] = None, cyclic: bool = False,
-                   in_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   in_scale: Optional[torch.Tensor] = None, squared_relu: bool = False) -> torch.Tensor:
     """out[p] = weight[index[p]] x[p // in_div] for p < ``pairs``; ``weight`` is [E, R, K] (``index`` None: E = 1, or,
     ``cyclic``, pair p uses matrix p mod E).
     ``gated`` = (limit, alpha): the matrices hold R gate rows and then R up rows, [E, 2 R, K], and the result is
     min(g, limit) * sigmoid(alpha * min(g, limit)) * (clamp(u, -limit, limit) + up_shift); ``gated`` may carry
     up_shift as a third number (default 1; (inf, 1, 0) is silu(g) * u).  ``in_scale`` (float32 [pairs]): pair p's input
-    row is multiplied by in_scale[p] as it is read."""
+    row is multiplied by in_scale[p] as it is read.  ``squared_relu``: the result is max(sum, 0)^2.  Pairs whose index names no
+    matrix are left out (their rows of the result hold nothing)."""
     check(x, "x")
+    if squared_relu and gated:
+        raise KernelError("indexed_linear: a gated product has the gate's activation")
     check(weight, "expert weights", x.dtype, x.shape[-1])
     if in_scale is not None:
         check(in_scale, "input scales", torch.float32)
@@ -1033,7 +1153,7 @@ def indexed_linear(x: torch.Tensor, weight: torch.Tensor, index: Optional[torch.
     call("llm_indexed_linear", x.data_ptr(), weight.data_ptr(), pointer(index), out.data_ptr(), pairs, rows, x.shape[-1],
          int(in_div), int(bool(gated)), limit, alpha, dtype_code(x.dtype),
          int(out_dtype == torch.float32 and x.dtype != torch.float32), weight.shape[0] if cyclic and index is None else 0,
-         pointer(in_scale), up_shift, stream_handle())
+         pointer(in_scale), up_shift, int(bool(squared_relu)), weight.shape[0], stream_handle())
     return out
 
 
@@ -1052,9 +1172,11 @@ def _check_shared_gate(shared_gate: Optional[torch.Tensor], tokens: int) -> None
 
 
 def moe_combine(down: torch.Tensor, weights: torch.Tensor, shared_out: Optional[torch.Tensor], act_dtype: torch.dtype,
-                shared_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                shared_gate: Optional[torch.Tensor] = None, own: Optional[torch.Tensor] = None, chosen: Optional[torch.Tensor] = None,
+                experts: int = 0) -> torch.Tensor:
     """out[t] = sum_j weights[t, j] * down[t * top + j] (+ shared_gate[t] * shared_out[t]); ``down`` float32 [N * top, H],
-    ``shared_gate`` float32 [N] (absent: 1)."""
+    ``shared_gate`` float32 [N] (absent: 1).  With ``own`` ([N, H]) a pair that chose an identity output (``chosen`` int32
+    [N, top], ``experts`` or beyond) contributes own[t] in down's place."""
     check(down, "expert outputs", torch.float32)
     check(weights, "routing weights", torch.float32)
     tokens, top = weights.shape
@@ -1065,8 +1187,11 @@ def moe_combine(down: torch.Tensor, weights: torch.Tensor, shared_out: Optional[
         check(shared_out, "shared expert output", act_dtype, width)
     _check_shared_gate(shared_gate, tokens)
     out = torch.empty((tokens, width), dtype=act_dtype, device=down.device)
+    if own is not None:
+        check(own, "tokens' own rows", act_dtype, width)
+        check(chosen, "chosen experts", torch.int32, top)
     call("llm_moe_combine", down.data_ptr(), weights.data_ptr(), pointer(shared_out), pointer(shared_gate), out.data_ptr(), tokens, width, top,
-         dtype_code(act_dtype), stream_handle())
+         pointer(chosen) if own is not None else 0, int(experts), pointer(own), dtype_code(act_dtype), stream_handle())
     return out
 
 
@@ -1084,7 +1209,8 @@ MOE_TILE_ROWS = 128
 
 
 def moe_plan(chosen: torch.Tensor, experts: int) -> ExpertPlan:
-    """Sorts the pairs of ``chosen`` (int32 [N, top]) by expert on the device; nothing comes back to the host."""
+    """Sorts the pairs of ``chosen`` (int32 [N, top]) by expert on the device; nothing comes back to the host.  Pairs that
+    chose an identity output (``experts`` or beyond) get no row: their ``row_of_pair`` is -1."""
     check(chosen, "chosen experts", torch.int32)
     pairs = chosen.numel()
     max_tiles = -(-pairs // MOE_TILE_ROWS) + experts
@@ -1111,15 +1237,18 @@ def moe_grouped_supported(weight: torch.Tensor, gated: bool) -> bool:
 
 
 def moe_grouped(x: torch.Tensor, weight: torch.Tensor, plan: ExpertPlan, gather_div: Optional[int] = None,
-                gated: Optional[tuple] = None, pair_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
+                gated: Optional[tuple] = None, pair_scale: Optional[torch.Tensor] = None, squared_relu: bool = False) -> torch.Tensor:
     """One tiled product over all experts: row r of the plan's order gets weight[its expert] times its input row,
     which is x[pair_of_row[r] // gather_div] or, with ``gather_div`` None, x[r].  ``gated`` = (limit, alpha): the
     matrices are [E, 2 R, K], gate rows first, and the result is the experts' activation in bfloat16 [pairs, R];
     otherwise the 32-bit sums [pairs, R].  On tcgen05 where that kernel takes the sizes (it reads its rows by TMA, so
     rows that have to be gathered are copied into the plan's order first), else the mma.sync kernel.  ``pair_scale``
     (float32 [pairs], with ``gather_div``): the gathered row of pair p is multiplied by pair_scale[p] on the way.
-    ``gated`` may carry the activation's up_shift as a third number (see ``indexed_linear``)."""
+    ``gated`` may carry the activation's up_shift as a third number (see ``indexed_linear``).  ``squared_relu``: max(sum, 0)^2
+    in bfloat16 [pairs, R]."""
     check(x, "x", torch.bfloat16)
+    if squared_relu and gated:
+        raise KernelError("moe_grouped: a gated product has the gate's activation")
     if pair_scale is not None:
         check(pair_scale, "pair scales", torch.float32)
         if gather_div is None or pair_scale.numel() < plan.pairs:
@@ -1127,7 +1256,8 @@ def moe_grouped(x: torch.Tensor, weight: torch.Tensor, plan: ExpertPlan, gather_
     check(weight, "expert weights", torch.bfloat16, x.shape[-1])
     rows = weight.shape[1] // 2 if gated else weight.shape[1]
     inner = x.shape[-1]
-    out = torch.empty((plan.pairs, rows), dtype=torch.bfloat16 if gated else torch.float32, device=x.device)
+    out = torch.empty((plan.pairs, rows), dtype=torch.bfloat16 if gated or squared_relu else torch.float32, device=x.device)
+    form = 1 if gated else 2 if squared_relu else 0
     limit, alpha, up_shift = _gate_constants(gated)
     tensor_memory = MOE_GROUPED_KERNEL != "mma" and library().llm_moe_grouped_tc_supports(rows, inner, int(bool(gated))) and (gated or rows % 4 == 0)
     if gather_div is not None and (tensor_memory or pair_scale is not None):
@@ -1137,19 +1267,20 @@ def moe_grouped(x: torch.Tensor, weight: torch.Tensor, plan: ExpertPlan, gather_
         x, gather_div = ordered, None
     if tensor_memory:
         call("llm_moe_grouped_tc", x.data_ptr(), plan.pairs, weight.data_ptr(), weight.shape[0], plan.tiles.data_ptr(), out.data_ptr(),
-             rows, inner, plan.max_tiles, int(bool(gated)), limit, alpha, up_shift, wait_error_flag(x.device).data_ptr(),
+             rows, inner, plan.max_tiles, form, limit, alpha, up_shift, wait_error_flag(x.device).data_ptr(),
              stream_handle())
         return out
     call("llm_moe_grouped", x.data_ptr(), weight.data_ptr(), plan.tiles.data_ptr(),
          plan.pair_of_row.data_ptr() if gather_div is not None else 0, int(gather_div or 1), out.data_ptr(), rows,
-         inner, plan.max_tiles, int(bool(gated)), limit, alpha, up_shift, stream_handle())
+         inner, plan.max_tiles, form, limit, alpha, up_shift, stream_handle())
     return out
 
 
 def moe_combine_rows(down: torch.Tensor, plan: ExpertPlan, weights: torch.Tensor, shared_out: Optional[torch.Tensor],
-                     act_dtype: torch.dtype, shared_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     act_dtype: torch.dtype, shared_gate: Optional[torch.Tensor] = None, own: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[t] = sum_j weights[t, j] * down[row_of_pair[t * top + j]] (+ shared_gate[t] * shared_out[t]); ``down`` float32 in
-    the plan's order, ``shared_gate`` float32 [N] (absent: 1)."""
+    the plan's order, ``shared_gate`` float32 [N] (absent: 1).  Pairs without a row (identity outputs) contribute own[t]
+    (``own`` [N, H])."""
     check(down, "expert outputs", torch.float32)
     check(weights, "routing weights", torch.float32)
     tokens, top = weights.shape
@@ -1157,9 +1288,11 @@ def moe_combine_rows(down: torch.Tensor, plan: ExpertPlan, weights: torch.Tensor
     if shared_out is not None:
         check(shared_out, "shared expert output", act_dtype, width)
     _check_shared_gate(shared_gate, tokens)
+    if own is not None:
+        check(own, "tokens' own rows", act_dtype, width)
     out = torch.empty((tokens, width), dtype=act_dtype, device=down.device)
     call("llm_moe_combine_rows", down.data_ptr(), plan.row_of_pair.data_ptr(), weights.data_ptr(), pointer(shared_out),
-         pointer(shared_gate), out.data_ptr(), tokens, width, top, dtype_code(act_dtype), stream_handle())
+         pointer(shared_gate), out.data_ptr(), tokens, width, top, pointer(own), dtype_code(act_dtype), stream_handle())
     return out
 
 

@@ -19,8 +19,8 @@ SIGNATURES = {
     "llm_embedding_gather": [_P, _P, _P, _I, _I, _I, _I, _F, _I, _P, _P, _S],
     "llm_add_rmsnorm": [_P, _P, _P, _P, _P, _I, _I, _F, _I, _I, _I, _P, _S],
     "llm_rmsnorm": [_P, _P, _P, _I, _I, _F, _I, _I, _S],
-    "llm_silu_mul": [_P, _P, _I, _I, _I, _I, _S],
-    "llm_gelu_mul": [_P, _P, _I, _I, _I, _I, _S],
+    "llm_silu_mul": [_P, _P, _I, _I, _I, _P, _I, _S],
+    "llm_gelu_mul": [_P, _P, _I, _I, _I, _P, _I, _S],
     "llm_grouped_rmsnorm": [_P, _P, _P, _I, _I, _I, _F, _I, _I, _S],
     "llm_conv_norm_kv": [_P, _I, _P, _I, _P, _P, _P, _P, _P, _I, _P, _P, _F, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _I, _S],
     "llm_decay_recurrence_threads": [_I, _I],
@@ -42,15 +42,15 @@ SIGNATURES = {
     "llm_pointwise": [_I, _P, _P, _P, ctypes.c_longlong, _F, _F, _I, _I, _S],
     "llm_token_shift_mix": [_P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _S],
     "llm_short_conv_units": [_P, _I, _I, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _F, _P, _I, _P, _I, _I, _I, _S],
-    "llm_gated_scan": [_P, _P, _P, _P, _P, _I, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P, _I, _S],
+    "llm_gated_scan": [_P, ctypes.c_longlong, ctypes.c_longlong, _P, _P, _P, _P, _I, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P, _I, _S],
     "llm_streams_norm": [_P, _I, _I, _P, _P, _P, _F, _F, _P, _P, _P, _F, _F, _P, _P, _P, _P, _F, _I, _P, _P, _I, _I, _I, _S],
     "llm_matrix_recurrence_supports": [_I, _I],
     "llm_wkv_recurrent": [_P, _I, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _F, _P, _P, _I, _I, _I, _I, _I, _P, _P, _S],
     "llm_delta_rule_recurrent": [_P, _I, _I, _P, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _I, _P, _P, _S],
     "llm_moe_route": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _I, _I, _P, _I, _S],
     "llm_moe_select": [_P, _P, _P, _P, _I, _I, _I, _F, _I, _I, _I, _I, _I, _P, _S],
-    "llm_indexed_linear": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _I, _I, _I, _P, _F, _S],
-    "llm_moe_combine": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _S],
+    "llm_indexed_linear": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _I, _I, _I, _P, _F, _I, _I, _S],
+    "llm_moe_combine": [_P, _P, _P, _P, _P, _I, _I, _I, _P, _I, _P, _I, _S],
     "llm_clamped_glu": [_P, _P, _I, _I, _F, _F, _I, _S],
     "llm_moe_plan": [_P, _I, _I, _P, _P, _P, _P, _I, _S],
     "llm_moe_grouped_supports": [_I, _I, _I],
@@ -58,7 +58,7 @@ SIGNATURES = {
     "llm_moe_grouped_tc_supports": [_I, _I, _I],
     "llm_moe_gather_rows": [_P, _P, _I, _P, _I, _I, _P, _S],
     "llm_moe_grouped_tc": [_P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _F, _F, _F, _P, _S],
-    "llm_moe_combine_rows": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _S],
+    "llm_moe_combine_rows": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _P, _I, _S],
     "llm_gemm_f32": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _S],
     "llm_attention_mma_supports": [_I, _I, _I],
     "llm_attention_mma_sinks_supports": [_I, _I, _I, _I],
