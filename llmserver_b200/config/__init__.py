@@ -7,7 +7,8 @@ from .dikusun import DikusunConfig
 from .vibepel import VibepelConfig
 from .zeridra import ZeridraConfig
 from .dozotar import DozotarConfig
+from .rapolix import RapolixConfig
 
 __all__ = ["UnsupportedModelError", "WeightLoadError", "PartSpec", "LayerSpec", "ScheduleEntry", "ModelSpec",
            "ARCHITECTURES", "Architecture", "register_architecture", "architecture_of", "read_config",
-           "Qwen3Config", "GefaraxConfig", "DikusunConfig", "VibepelConfig", "ZeridraConfig", "DozotarConfig", "FULL_ATTENTION", "SLIDING_ATTENTION"]
+           "Qwen3Config", "GefaraxConfig", "DikusunConfig", "VibepelConfig", "ZeridraConfig", "DozotarConfig", "RapolixConfig", "FULL_ATTENTION", "SLIDING_ATTENTION"]

@@ -87,6 +87,7 @@ class ModelSpec:
     embedding_scale: float = 1.0    # the embedded tokens are multiplied by this as they enter the stream
     logit_scale: float = 1.0        # the head's products are multiplied by this (before the cap)
     logit_softcap: float = 0.0      # c > 0: the logits leave as c * tanh(logits / c)
+    streams: int = 1                # residual streams per token, all equal to the embedded tokens at the start; the final norm reads their sum
     max_positions: Optional[int] = None
     eos_token_ids: Tuple[int, ...] = ()
     notes: dict = field(default_factory=dict)

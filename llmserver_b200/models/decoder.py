@@ -33,6 +33,9 @@ class DecoderModel:
         for layer in spec.layers:
             block_cls = BLOCKS.get(layer.block.kind)
             block_params = layer.block.as_dict()
+            if block_cls.streams(block_params) != spec.streams:
+                raise ValueError(f"layer {layer.prefix!r}: its block works on {block_cls.streams(block_params)} residual streams, the "
+                                 f"model has {spec.streams}")
             built = {}
             for role, part, cls, prefix in parts_of_layer(layer):
                 weights = {local: source.get(prefix + local) for local in cls.declare_weights(part.as_dict())}
@@ -81,20 +84,26 @@ class DecoderModel:
         self.entry_caches = views
 
     # ------------------------------------------------------------------ the step
+    def _embed(self, batch, streams: int = 1) -> torch.Tensor:
+        """The embedded tokens, float32 [N, H], or [N, streams, H] with that many equal streams."""
+        terms = {}
+        for position in self.positions.values():
+            terms.update(position.embedding_terms(batch))
+        embedded = ops.embedding(self.embedding, batch.token_ids, scale=self.spec.embedding_scale, copies=streams, **terms)
+        for position in self.positions.values():
+            position.on_embedding(embedded, batch)
+        return embedded
+
     def step(self, batch) -> torch.Tensor:
         if self.entry_caches is None:
             raise RuntimeError("bind_cache() has to be called before the first step")
-        residual = ops.embedding(self.embedding, batch.token_ids, scale=self.spec.embedding_scale)
-        for position in self.positions.values():
-            position.on_embedding(residual, batch)
+        residual = self._embed(batch, self.spec.streams)
         delta = None
         schedule = self.spec.schedule
         embedded = None
         if any(entry.add_embedding for entry in schedule):
             # the stream is updated in place, so entries that take the embedded tokens in again read a second gather
-            embedded = ops.embedding(self.embedding, batch.token_ids, scale=self.spec.embedding_scale)
-            for position in self.positions.values():
-                position.on_embedding(embedded, batch)
+            embedded = self._embed(batch)
         for index, entry in enumerate(schedule):
             block = self.layers[entry.layer]
             if entry.add_embedding:

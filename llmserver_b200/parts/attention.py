@@ -54,10 +54,12 @@ class GQAttention(Mixer):
     right behind their projections (weights: the projection's name with ".conv" added, [channels, taps], the last column
     the current token's); the last taps - 1 projected rows of every request are kept in its state slot.  ``qk_norm``
     "projection": one RMS norm over all of q and one over all of k, weights as long as they, in place of the norms per
-    head.  ``chunk``: a query at position p reads keys floor(p / chunk) * chunk .. p.  ``distance_bias`` = (buckets, largest):
+    head.  ``chunk``: a query at position p reads keys floor(p / chunk) * chunk .. p.  ``keep_first``: with a window, every query also reads
+    the sequence's first ``keep_first`` keys, at their true distances.  ``gate`` (bool): the concatenated heads are multiplied by
+    sigmoid(W_g x) (role g, [heads * value_dim, hidden], part of the fused product) in front of the output projection.  ``distance_bias`` = (buckets, largest):
     a learned number per head and bucket of the distance between query and key (``rel`` [buckets, heads]; see
     ``distance_buckets``; buckets None: as many as the tensor has rows) is added to the scaled score.  ``names``: pairs (role, tensor name behind the prefix) for checkpoints that call the
-    tensors otherwise; roles are q, k, v, o, q_norm, k_norm, sinks, rel.
+    tensors otherwise; roles are q, k, v, o, g, q_norm, k_norm, sinks, rel.
 
     How positions are encoded comes from the position encoding the layer names (``attach``): its inverse
     frequencies, how many elements of a head rotate (``rotary_dim``, at most head_dim) and how they pair
@@ -68,9 +70,9 @@ class GQAttention(Mixer):
 
     KNOWN_PARAMS = ("hidden", "heads", "kv_heads", "head_dim", "scale", "qk_norm", "eps", "window", "bias", "softcap",
                     "value_dim", "sinks", "names", "precise_weights", "values_are_keys", "unit_sink", "query_temperature",
-                    "conv", "chunk", "distance_bias")
+                    "conv", "chunk", "distance_bias", "keep_first", "gate")
     NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
-             "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "sinks": "sinks", "rel": "rel"}
+             "g": "g_proj.weight", "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "sinks": "sinks", "rel": "rel"}
 
     @classmethod
     def names(cls, params) -> dict:
@@ -101,6 +103,10 @@ class GQAttention(Mixer):
                              "without a query temperature")
         if params.get("chunk") and (int(params["chunk"]) <= 0 or params.get("window")):
             raise ValueError("gqa_attention: keys are bounded by a window or by chunks of a positive size, not by both")
+        if int(params.get("keep_first") or 0) < 0 or (params.get("keep_first") and params.get("chunk")):
+            raise ValueError("gqa_attention: first keys are kept beside a window, and not a negative number of them")
+        if params.get("gate") and (cls.by_rows(params) or params.get("values_are_keys")):
+            raise ValueError("gqa_attention: an output gate comes with a value projection and heads normalised one by one")
         if params.get("distance_bias") and params["distance_bias"][0] is not None:
             distance_buckets(int(params["distance_bias"][0]), float(params["distance_bias"][1]), 1)
 
@@ -120,6 +126,8 @@ class GQAttention(Mixer):
                   name["o"]: WeightDecl((hidden, heads * value_dim))}
         if params.get("values_are_keys"):
             del wanted[name["v"]]
+        if params.get("gate"):
+            wanted[name["g"]] = WeightDecl((heads * value_dim, hidden))
         if params.get("qk_norm"):
             whole = params["qk_norm"] == "projection"
             wanted[name["q_norm"]] = WeightDecl((heads * dim if whole else dim,), NORM)
@@ -139,7 +147,8 @@ class GQAttention(Mixer):
             return KVPagesNeed(int(params["kv_heads"]), int(params["head_dim"]), params.get("window"), None, keys_only=True)
         pages = KVPagesNeed(int(params["kv_heads"]), int(params["head_dim"]), params.get("window"),
                             int(params["value_dim"]) if params.get("value_dim") else None,
-                            chunk=int(params["chunk"]) if params.get("chunk") else None)
+                            chunk=int(params["chunk"]) if params.get("chunk") else None,
+                            keep_first=int(params.get("keep_first") or 0))
         if int(params.get("conv") or 1) == 1:
             return pages
         kv_heads, dim = int(params["kv_heads"]), int(params["head_dim"])
@@ -160,8 +169,20 @@ class GQAttention(Mixer):
         name = self.names(params)
         self.values_are_keys = bool(params.get("values_are_keys"))
         self.temperature = tuple(params["query_temperature"]) if params.get("query_temperature") else None
-        self.qkv = torch.cat([weights[name["q"]], weights[name["k"]]] + ([] if self.values_are_keys else [weights[name["v"]]]),
-                             dim=0).contiguous()
+        rows = [weights[name["q"]], weights[name["k"]]] + ([] if self.values_are_keys else [weights[name["v"]]])
+        self.keep_first = int(params.get("keep_first") or 0) if self.window else 0
+        self.gate_column = None
+        if params.get("gate"):
+            # the gate's rows lie behind the values', everything at whole 16-byte pieces of the packed row
+            def fill():
+                ragged = -sum(int(row.shape[0]) for row in rows) % 8
+                if ragged:
+                    rows.append(torch.zeros((ragged, rows[0].shape[1]), dtype=rows[0].dtype, device=rows[0].device))
+            fill()
+            self.gate_column = sum(int(row.shape[0]) for row in rows)
+            rows.append(weights[name["g"]])
+            fill()
+        self.qkv = torch.cat(rows, dim=0).contiguous()
         self.out = weights[name["o"]].contiguous()
         self.q_norm = weights[name["q_norm"]].contiguous() if params.get("qk_norm") else None
         self.k_norm = weights[name["k_norm"]].contiguous() if params.get("qk_norm") else None
@@ -169,7 +190,8 @@ class GQAttention(Mixer):
         if params.get("unit_sink"):
             self.sinks = torch.zeros(self.heads, dtype=torch.float32, device=runtime.device)      # exp(0): a one in every denominator
         # keys that are their own values and queries with a temperature go through the kernel for heads made of units
-        self.by_units = self.values_are_keys or self.temperature is not None
+        # (as do packed rows with a gate behind their values: that kernel takes longer rows)
+        self.by_units = self.values_are_keys or self.temperature is not None or self.gate_column is not None
         self.inv_freq, self.rotary_dim, self.interleaved, self.magnitude = None, self.head_dim, False, 1.0
         self.rows_first = self.by_rows(params)
         self.taps = None
@@ -273,4 +295,5 @@ class GQAttention(Mixer):
         return ops.attention(queries, batch, tables, pages.k_pages, pages.v_pages, self.heads, self.kv_heads, self.head_dim,
                              self.scale, self.window, value_dim=self.value_dim, sinks=self.sinks,
                              precise=bool(self.params.get("precise_weights")), q_stride=q_stride, chunk=self.chunk, bias=self.bias,
-                             bias_log2=self.bias_log2)
+                             bias_log2=self.bias_log2, keep=self.keep_first, gate=queries if self.gate_column is not None else None,
+                             gate_column=self.gate_column or 0)

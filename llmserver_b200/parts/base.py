@@ -109,6 +109,11 @@ class PositionEncoding(Part):
     def on_embedding(self, residual: torch.Tensor, batch) -> None:
         """Hook for encodings that act on the embedded tokens (absolute tables); default: nothing."""
 
+    def embedding_terms(self, batch) -> dict:
+        """Keyword arguments for ``ops.embedding``, for encodings that join the embedded tokens in the kernel that gathers
+        them; default: none."""
+        return {}
+
 
 class Block(Part):
     """An arrangement of parts around the residual stream.  The class says which parts it arranges: ``roles`` maps
@@ -119,6 +124,11 @@ class Block(Part):
     @classmethod
     def roles(cls, params: dict) -> Dict[str, str]:
         return {"mixer": "mixer", "feed_forward": "feed_forward", "mixer_norm": "norm", "feed_forward_norm": "norm"}
+
+    @classmethod
+    def streams(cls, params: dict) -> int:
+        """Residual streams per token that the block works on (more than one: the residual is [N, streams, width])."""
+        return 1
 
     @classmethod
     def prefix_of(cls, params: dict, role: str) -> str:
@@ -134,6 +144,9 @@ class Block(Part):
 
     def __init__(self, params, parts: Dict[str, Part]):
         self.check_params(params)
+        biased = sorted(role for role, part in parts.items() if getattr(part, "output_bias", None) is not None)
+        if biased and not self.adds_output_bias:
+            raise ValueError(f"{type(self).__name__} does not add the bias that {', '.join(biased)} leaves to the kernel on the stream")
         self.params, self.parts = params, dict(parts)
         for role, part in parts.items():
             setattr(self, role, part)
@@ -142,6 +155,9 @@ class Block(Part):
         """(norm, consumer): the norm that this block applies to the stream first and the part that reads its output,
         for a block in front that can prepare that norm's input; None when the block does not start that way."""
         return None
+
+    # True: the block has the bias of a part's last projection (its ``output_bias``) added by the kernel that adds the result.
+    adds_output_bias = False
 
     # True: ``forward`` takes a keyword ``after``, the ``entry()`` of what runs next (the next block, or the final
     # norm with no consumer), and may return a used ``ops.StreamSink`` in place of its not yet added output.

@@ -4,8 +4,8 @@ from __future__ import annotations
 from .base import Block
 import torch
 
-from ..weights.declare import NORM, WeightDecl
-from .norm import NormedDelta, ScaledDelta, add_and_read
+from ..weights.declare import NORM, WIDE, WeightDecl
+from .norm import NormedDelta, ScaledDelta, StreamsDelta, add_and_read
 from .registry import BLOCKS
 
 
@@ -87,6 +87,7 @@ class OutputNormBlock(Block):
     is its mixer alone) and the tensor-name prefixes of its parts."""
 
     KNOWN_PARAMS = ("feed_forward", "mixer_prefix", "feed_forward_prefix", "mixer_out_norm_prefix", "feed_forward_out_norm_prefix")
+    adds_output_bias = True
 
     @classmethod
     def roles(cls, params):
@@ -155,3 +156,74 @@ class ParallelResidualBlock(Block):
         if self.params.get("feed_forward", True):
             pending.append((self.feed_forward.forward(normed), self.feed_forward_scale))
         return residual, ScaledDelta(pending)
+
+
+@BLOCKS.register("hyper_connections")
+class HyperConnectionsBlock(Block):
+    """Several residual streams x_1 .. x_S per token (the scheme of Zhu et al., "Hyper-Connections", with fixed coefficients).
+    Each sub-layer reads one weighted sum of them and writes into all:
+
+        u = sum_s in[s] x_s;  y = sub_layer(norm(u));  x_t <- sum_s mix[s, t] x_s + out[t] * y        all streams at once
+
+    with coefficients of its own (``in`` [S], ``out`` [S], ``mix`` [S, S] from, to; held in 32-bit).  The residual handed through
+    the model is [N, S, width]; writing one sub-layer's output, reading the streams for the next and its norm are one kernel, so
+    an output travels on as a ``StreamsDelta``.  A mixer that leaves several outputs to be normalised and summed
+    (``forward_parts``) has that done by the same kernel, and so has a projection's last bias (``output_bias``).  Parameters:
+    ``streams``; ``feed_forward`` (default True; False: the layer is its mixer alone); the tensor-name prefixes of its parts and of
+    the coefficients (``mixer_connections``, ``feed_forward_connections``; default "hc1." and "hc2.")."""
+
+    KNOWN_PARAMS = ("streams", "feed_forward", "mixer_prefix", "feed_forward_prefix", "mixer_norm_prefix", "feed_forward_norm_prefix",
+                    "mixer_connections", "feed_forward_connections")
+    CONNECTIONS = {"mixer": "hc1.", "feed_forward": "hc2."}
+    adds_output_bias = True
+
+    @classmethod
+    def streams(cls, params) -> int:
+        return int(params["streams"])
+
+    @classmethod
+    def check_params(cls, params):
+        super().check_params(params)
+        if int(params["streams"]) < 1:
+            raise ValueError(f"hyper_connections: {params['streams']} streams")
+
+    @classmethod
+    def roles(cls, params):
+        roles = {"mixer": "mixer", "mixer_norm": "norm"}
+        if params.get("feed_forward", True):
+            roles.update({"feed_forward": "feed_forward", "feed_forward_norm": "norm"})
+        return roles
+
+    @classmethod
+    def _connections(cls, params):
+        return [(role, params.get(f"{role}_connections", prefix)) for role, prefix in cls.CONNECTIONS.items()
+                if role == "mixer" or params.get("feed_forward", True)]
+
+    @classmethod
+    def declare_weights(cls, params):
+        count, wanted = int(params["streams"]), {}
+        for _, prefix in cls._connections(params):
+            wanted.update({prefix + "in": WeightDecl((count,), WIDE), prefix + "out": WeightDecl((count,), WIDE),
+                           prefix + "mix": WeightDecl((count, count), WIDE)})
+        return wanted
+
+    def __init__(self, params, parts, weights=None):
+        super().__init__(params, parts)
+        self.connections = {role: {name: weights[prefix + name].to(torch.float32).contiguous() for name in ("in", "out", "mix")}
+                            for role, prefix in self._connections(params)}
+
+    def _pending(self, role, parts):
+        own = self.connections[role]
+        return StreamsDelta(parts, mix=own["mix"], out=own["out"])
+
+    def forward(self, residual, delta, batch, cache):
+        normed = self.mixer_norm.add_norm(residual, delta, read=self.connections["mixer"]["in"])
+        if hasattr(self.mixer, "forward_parts"):
+            pending = self._pending("mixer", self.mixer.forward_parts(normed, batch, cache))
+        else:
+            pending = self._pending("mixer", [(self.mixer.forward(normed, batch, cache), getattr(self.mixer, "output_bias", None), None, 0.0, 1.0)])
+        if not self.params.get("feed_forward", True):
+            return residual, pending
+        normed = self.feed_forward_norm.add_norm(residual, pending, read=self.connections["feed_forward"]["in"])
+        out = self.feed_forward.forward(normed)
+        return residual, self._pending("feed_forward", [(out, getattr(self.feed_forward, "output_bias", None), None, 0.0, 1.0)])

@@ -1,4 +1,4 @@
-"""Dense feed-forwards: SwiGLU, the gated layer with gelu, one with clamped values, and a layer without a gate."""
+"""Dense feed-forwards: SwiGLU, gated layers with gelu and with biases, one with clamped values, and a layer without a gate."""
 from __future__ import annotations
 
 import functools
@@ -6,7 +6,7 @@ import functools
 import torch
 
 from .. import ops
-from ..weights.declare import WeightDecl
+from ..weights.declare import WIDE, WeightDecl
 from .base import FeedForward
 from .registry import FEED_FORWARDS
 
@@ -82,6 +82,50 @@ class GeluGLU(FeedForward):
 
     def forward(self, x):
         return ops.linear(ops.gelu_mul(ops.linear(x, self.gate_up)), self.down)
+
+
+@FEED_FORWARDS.register("biased_glu")
+class BiasedGLU(FeedForward):
+    """A dense gated feed-forward whose projections have biases: y = W_down (act(W_gate x + b_gate) * (W_up x + b_up)) + b_down.
+    The gate's and up's biases are added in 32-bit by the activation's kernel; the last one is left to the kernel that adds the
+    result to the stream (``output_bias``), so a block has to know it.  Parameters: ``hidden``, ``intermediate``; ``activation``
+    ("silu", the default, or "gelu" in its tanh form); ``names``: pairs (role, tensor name behind the prefix) for the roles gate,
+    up and down (a bias is the tensor's name with ".b" added)."""
+
+    KNOWN_PARAMS = ("hidden", "intermediate", "activation", "names")
+    NAMES = {"gate": "gate", "up": "up", "down": "down"}
+    ACTIVATIONS = {"silu": "silu_mul", "gelu": "gelu_mul"}
+
+    @classmethod
+    def names(cls, params) -> dict:
+        return {**cls.NAMES, **dict(params.get("names") or ())}
+
+    @classmethod
+    def check_params(cls, params):
+        super().check_params(params)
+        if params.get("activation", "silu") not in cls.ACTIVATIONS:
+            raise ValueError(f"biased_glu gates with {' or '.join(cls.ACTIVATIONS)}, not {params['activation']!r}")
+
+    @classmethod
+    def declare_weights(cls, params):
+        hidden, intermediate = int(params["hidden"]), int(params["intermediate"])
+        name, wanted = cls.names(params), {}
+        for role, shape in (("gate", (intermediate, hidden)), ("up", (intermediate, hidden)), ("down", (hidden, intermediate))):
+            wanted[name[role]] = WeightDecl(shape)
+            wanted[name[role] + ".b"] = WeightDecl(shape[:1], WIDE)
+        return wanted
+
+    def __init__(self, params, weights, runtime):
+        super().__init__(params, weights, runtime)
+        name = self.names(params)
+        self.gate_up = torch.cat([weights[name["gate"]], weights[name["up"]]], dim=0).contiguous()
+        self.gate_up_bias = torch.cat([weights[name[role] + ".b"].to(torch.float32) for role in ("gate", "up")]).contiguous()
+        self.down = weights[name["down"]].contiguous()
+        self.output_bias = weights[name["down"] + ".b"].to(torch.float32).contiguous()
+        self.gate = getattr(ops, self.ACTIVATIONS[params.get("activation", "silu")])
+
+    def forward(self, x):
+        return ops.linear(self.gate(ops.linear(x, self.gate_up), bias=self.gate_up_bias), self.down)
 
 
 @FEED_FORWARDS.register("clamped_glu")

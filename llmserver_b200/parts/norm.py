@@ -1,4 +1,4 @@
-"""RMSNorm over the residual stream."""
+"""Norms over the residual stream, or over several of them."""
 from __future__ import annotations
 
 from dataclasses import dataclass
@@ -30,6 +30,17 @@ class ScaledDelta:
     per channel (float32 [width]): ``parts`` is a list of (output, scale).  The next norm's kernel multiplies, adds all of
     them to the 32-bit stream and normalises it in one pass."""
     parts: list
+
+
+@dataclass
+class StreamsDelta:
+    """A sub-layer's output that has not been written into the token's several residual streams yet: ``parts`` as
+    ``ops.streams_norm`` takes them (up to two outputs, each with the bias of its projection and a norm of its own where it
+    has them), ``mix`` and ``out`` the streams' coefficients (float32 [S, S] from, to; [S]).  The next norm's kernel writes all
+    streams at once from the old ones, reads them through the weights of what runs next and normalises."""
+    parts: list
+    mix: Optional[torch.Tensor] = None
+    out: Optional[torch.Tensor] = None
 
 
 def add_and_read(residual: torch.Tensor, delta, act_dtype: torch.dtype) -> torch.Tensor:
@@ -70,7 +81,9 @@ class RMSNorm(Norm):
             self.weight = self.weight.to(torch.float32).expand(int(params["width"])).contiguous()
         self.eps = float(params["eps"])
 
-    def add_norm(self, residual, delta, rows=None, unscaled=False):
+    def add_norm(self, residual, delta, rows=None, unscaled=False, read=None):
+        if residual.dim() == 3 or isinstance(delta, StreamsDelta):
+            return _streams_norm(self, False, residual, delta, rows, read)
         if isinstance(delta, NormedDelta):
             post = delta.norm
             return ops.normed_add_rmsnorm(residual, delta.delta, post.weight if post is not None else None,
@@ -106,3 +119,39 @@ class RMSNorm(Norm):
 
     def norm(self, x):
         return ops.rmsnorm(x, self.weight, self.eps)
+
+
+def _streams_norm(norm, centre: bool, residual, delta, rows, read):
+    """``add_norm`` over several streams (or one): what is pending is written, the streams are read through ``read`` (None:
+    their sum) and normalised."""
+    if delta is None:
+        delta = StreamsDelta([])
+    elif isinstance(delta, torch.Tensor):
+        delta = StreamsDelta([(delta, None, None, 0.0, 1.0)])
+    elif isinstance(delta, NormedDelta) and delta.norm is not None and delta.extra is None:
+        delta = StreamsDelta([(delta.delta, delta.bias, delta.norm.weight, delta.norm.eps, 1.0)])
+    elif not isinstance(delta, StreamsDelta):
+        raise TypeError(f"several streams take a StreamsDelta, an output or nothing, not {type(delta).__name__}")
+    return ops.streams_norm(residual, delta.parts, norm.weight, norm.eps, centre, mix=delta.mix, out_weight=delta.out, read=read,
+                            rows=rows, act_dtype=norm.runtime.dtype)
+
+
+@NORMS.register("layernorm")
+class LayerNorm(Norm):
+    """y = weight * (x - mean) / sqrt(mean((x - mean)^2) + eps), no bias.  Parameters: ``width``, ``eps``; ``tensor``: the weight's
+    name behind the part's prefix (default "weight"; "" when the prefix is the whole name).  The kernel that adds what is
+    pending also normalises, on one stream as on several (``ops.streams_norm``)."""
+
+    KNOWN_PARAMS = ("width", "eps", "tensor")
+
+    @classmethod
+    def declare_weights(cls, params):
+        return {params.get("tensor", "weight"): WeightDecl((params["width"],), NORM)}
+
+    def __init__(self, params, weights, runtime):
+        super().__init__(params, weights, runtime)
+        self.weight = weights[params.get("tensor", "weight")].contiguous()
+        self.eps = float(params["eps"])
+
+    def add_norm(self, residual, delta, rows=None, read=None):
+        return _streams_norm(self, True, residual, delta, rows, read)

@@ -1,4 +1,4 @@
-"""Rotary position encoding (NeoX half-split form)."""
+"""Position encodings: rotary ones (NeoX half-split and neighbouring pairs), and sinusoids that join the embedding."""
 from __future__ import annotations
 
 import torch
@@ -121,3 +121,24 @@ class BandedRotaryPosition(PositionEncoding):
         self.pairing = params.get("pairing") or "halves"
         self.attention_factor = 1.0
         self.inv_freq = torch.tensor(table, dtype=torch.float64).to(torch.float32).to(runtime.device).contiguous()
+
+
+@POSITION_ENCODINGS.register("sinusoidal")
+class SinusoidalPosition(PositionEncoding):
+    """A vector of sines and cosines added to the embedded tokens: element 2i is sin(p f_i), element 2i + 1 cos(p f_i) with f_i =
+    base^(-2i / width).  No layer names it; the kernel that gathers the embedding adds it (``embedding_terms``).  Frequencies
+    are kept as sums of two floats, so that the angles of far positions are 32-bit exact.  Parameters: ``width``, ``base``
+    (default 10000)."""
+
+    KNOWN_PARAMS = ("width", "base")
+
+    def __init__(self, params, weights, runtime):
+        super().__init__(params, weights, runtime)
+        width = int(params["width"])
+        exact = float(params.get("base") or 10000.0) ** (-2.0 * torch.arange((width + 1) // 2, dtype=torch.float64) / width)
+        high = exact.to(torch.float32)
+        low = (exact - high.to(torch.float64)).to(torch.float32)
+        self.frequencies = torch.stack([high, low], dim=1).contiguous().to(runtime.device)
+
+    def embedding_terms(self, batch):
+        return {"positions": batch.positions, "frequencies": self.frequencies}
