@@ -1012,6 +1012,13 @@ SCAN_SEGMENT = 32          # fewest tokens per segment of the segmented gated sc
 SCAN_MAX_SEGMENTS = 128    # most segments per sequence
 
 
+def scan_segment(dtype: torch.dtype, longest: int) -> int:
+    """Tokens per segment of the gated scan for a step whose longest portion has ``longest`` tokens; 0: one pass."""
+    if dtype != torch.bfloat16 or longest < 2 * SCAN_SEGMENT:
+        return 0
+    return max(SCAN_SEGMENT, -(-longest // SCAN_MAX_SEGMENTS))
+
+
 def gated_scan(z: torch.Tensor, u: torch.Tensor, gate_bias: torch.Tensor, rate: torch.Tensor, y: torch.Tensor, y_column: int,
                y_bias: torch.Tensor, state: torch.Tensor, batch, segment: Optional[int] = None) -> torch.Tensor:
     """The real-gated linear recurrent unit, sequence by sequence, from and into each sequence's slot of ``state`` (float32
@@ -1041,7 +1048,7 @@ def gated_scan(z: torch.Tensor, u: torch.Tensor, gate_bias: torch.Tensor, rate: 
     out = torch.empty((tokens, width), dtype=u.dtype, device=u.device)
     longest = int(batch.max_q_len)
     if segment is None:
-        segment = 0 if u.dtype != torch.bfloat16 or longest < 2 * SCAN_SEGMENT else max(SCAN_SEGMENT, -(-longest // SCAN_MAX_SEGMENTS))
+        segment = scan_segment(u.dtype, longest)
     segments, summary, start = 0, None, None
     if segment:
         segments = -(-longest // int(segment))
