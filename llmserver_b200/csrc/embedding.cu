@@ -5,7 +5,7 @@
 // With `frequencies` ([(hidden + 1) / 2] pairs of floats whose sum is the frequency) a sinusoidal position vector joins the
 // row: element 2i gets sin(p f_i), element 2i + 1 cos(p f_i) at position p.  Far positions turn many times, so the angle is
 // kept as two floats: a = fl(p * high), what that product's rounding left over (one fused multiply-add) and p * low are
-// the small rest e, and sin(a + e) = sin a + e cos a to 32-bit.
+// the small rest e, and sin(a + e) = sin a cos e + cos a sin e.
 //
 // `copies` > 1: the row is written that many times, one behind the other (models that carry several streams per token).
 #include "common.cuh"
@@ -15,8 +15,10 @@ __device__ __forceinline__ void position_wave(float position, float2 frequency, 
     const float rest = fmaf(position, frequency.x, -angle) + position * frequency.y;
     float s, c;
     sincosf(angle, &s, &c);
-    sine = fmaf(rest, c, s);
-    cosine = fmaf(-rest, s, c);
+    const float square = rest * rest;      // the first terms of the rest's own sine and cosine
+    const float turn = fmaf(-rest * square, 1.0f / 6.0f, rest), shrink = square * fmaf(square, 1.0f / 24.0f, -0.5f);
+    sine = s + fmaf(turn, c, shrink * s);
+    cosine = c + fmaf(-turn, s, shrink * c);
 }
 
 template <typename T>

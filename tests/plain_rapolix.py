@@ -159,22 +159,28 @@ def route(z, correction, router):
     return chosen, picked / (picked.sum() + 1e-20)
 
 
-def routing_margin(z, correction, router):
+def routing_margin(z, correction, router, matters=0.0):
     """How far one token's choice is from another one, in choice scores: the gap between the last output chosen and the
-    first one left out, and between the last group kept and the first one dropped."""
+    first one left out, and between the last group kept and the first one dropped.  Calls between outputs (or groups whose
+    outputs) have less than the share ``matters`` of the chosen scores are left out: either way changes little."""
     total, top = z.shape[0], int(router["top"])
-    choice = torch.softmax(z, dim=-1) + correction
+    s = torch.softmax(z, dim=-1)
+    choice = s + correction
+    chosen, _ = route(z, correction, router)
+    weight = float(s[chosen].sum())
     gaps, allowed = [], list(range(total))
     if router.get("groups"):
         count, keep = int(router["groups"]["count"]), int(router["groups"]["keep"])
         size = total // count
         best = sorted(((float(choice[g * size:(g + 1) * size].max()), g) for g in range(count)), reverse=True)
         if keep < count:
-            gaps.append(best[keep - 1][0] - best[keep][0])
+            at_stake = max(float(s[g * size:(g + 1) * size].max()) for _, g in best[keep - 1:keep + 1])
+            if at_stake >= matters * weight:
+                gaps.append(best[keep - 1][0] - best[keep][0])
         allowed = [e for e in allowed if e // size in [g for _, g in best[:keep]]]
-    ranked = sorted((float(choice[e]) for e in allowed), reverse=True)
-    if top < len(ranked):
-        gaps.append(ranked[top - 1] - ranked[top])
+    ranked = sorted(((float(choice[e]), float(s[e])) for e in allowed), reverse=True)
+    if top < len(ranked) and max(ranked[top - 1][1], ranked[top][1]) >= matters * weight:
+        gaps.append(ranked[top - 1][0] - ranked[top][0])
     return min(gaps) if gaps else math.inf
 
 
@@ -198,7 +204,7 @@ def feed_forward(h, weights, prefix, mlp):
 # ------------------------------------------------------------------------------------------------ the model
 def forward(config, weights, tokens, lose_state_at=None, streams=None, margins=None):
     """float64 logits [T, vocab] of the whole sequence.  ``streams``: receives the sum of the streams behind every layer;
-    ``margins``: receives each token's smallest routing margin."""
+    ``margins``: receives each token's smallest routing margin that matters."""
     eps = float(config["norm"]["eps"])
     embedded = weights["embed"][torch.tensor(list(tokens))] + sinusoids(torch.arange(len(tokens)), int(config["width"]))
     x = embedded.expand(int(config["streams"]), -1, -1).clone()
@@ -210,7 +216,7 @@ def forward(config, weights, tokens, lose_state_at=None, streams=None, margins=N
             h = layer_norm(read_streams(x, weights, prefix + "hc2."), weights[prefix + "norm2"], eps)
             if margins is not None and layer["mlp"]["kind"] == "moe":
                 z = h @ weights[prefix + "mlp.router"].T
-                found = torch.tensor([routing_margin(row, weights[prefix + "mlp.correction"], layer["mlp"]["router"]) for row in z])
+                found = torch.tensor([routing_margin(row, weights[prefix + "mlp.correction"], layer["mlp"]["router"], matters=0.04) for row in z])
                 margins.append(found if not margins else torch.minimum(margins.pop(), found))
             x = write_streams(x, feed_forward(h, weights, prefix + "mlp.", layer["mlp"]), weights, prefix + "hc2.")
         if streams is not None:
