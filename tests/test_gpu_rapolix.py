@@ -547,7 +547,7 @@ def test_squared_relu_experts_with_identities(dtype, tokens, width, experts, top
         want = plain.routed_feed_forward(x.double(), {name: tensor.double() for name, tensor in weights.items()}, "", config)
         z = x.double() @ weights["router"].double().T      # (rows whose choice hangs on the last bit of a score are left out)
         clear = torch.tensor([plain.routing_margin(row, weights["correction"].double(), config["router"]) > 1e-5 for row in z])
-        assert clear.float().mean() > 0.9
+        assert clear.float().mean() > 0.75
         _close((got.cpu().double() / want.abs().max())[clear], (want / want.abs().max())[clear], 2e-5 if dtype == torch.float32 else 1e-2)
 
 
