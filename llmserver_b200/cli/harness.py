@@ -723,3 +723,90 @@ def dozotar_step_cost(size: dict, layers: int, tokens: int, sequences: int, cont
         total_bytes += 2.0 * weights
         flops += 2.0 * tokens * weights
     return total_bytes, flops
+
+
+# ---------------------------------------------------------------------------------------------------------------------
+# Rapolix beside the closest design of each of its layers at equal size: Vibepel for the dense layers (two mixers side by
+# side, windowed attention and a recurrence with a convolution in front), Dozotar for the routed ones (softmax scores, groups, a
+# shared expert, attention bounded by chunks)
+# ---------------------------------------------------------------------------------------------------------------------
+# Layer sizes that resemble served models: attention with heads of 128 over a window of 1024 tokens that keeps the first 16, a
+# recurrent branch as wide as the stream in blocks of 128 channels, two residual streams; four layers with a dense feed-forward
+# three times as wide as the stream, four with routed experts, or both in turn.
+RAPOLIX_SIZES = {}
+for _width, _heads, _kv, _experts, _top, _ff in ((2048, 16, 4, 32, 4, 768), (4096, 32, 8, 64, 6, 1792)):
+    for _label, _kinds in (("dense", ("dense",) * 4), ("moe", ("moe",) * 4), ("mixed", ("dense", "moe", "dense", "moe"))):
+        RAPOLIX_SIZES[f"w{_width}-{_label}"] = dict(width=_width, heads=_heads, kv_heads=_kv, window=1024, keep=16, streams=2,
+                                                    dense_ff=3 * _width, experts=_experts, top=_top, identity=_experts // 4, groups=8,
+                                                    keep_groups=4, ff=_ff * 3 // 2, shared_ff=_ff * 3, kinds=_kinds)
+
+
+def _rapolix_kinds(size: dict, layers: int):
+    return [size["kinds"][index % len(size["kinds"])] for index in range(layers)]
+
+
+def rapolix_config(size: dict, layers: int = None):
+    from llmserver_b200.config import RapolixConfig
+    width = size["width"]
+    mixer = {"left": dict(heads=size["heads"], kv_heads=size["kv_heads"], dim=128, vdim=128, scale=128 ** -0.5,
+                          mask={"size": size["window"], "keep_first": size["keep"]}),
+             "right": dict(width=width, blocks=width // 128, conv=4)}
+    mlp = {"dense": {"kind": "dense", "ff": size["dense_ff"]},
+           "moe": {"kind": "moe", "router": {"experts": size["experts"], "top": size["top"], "identity": size["identity"],
+                                             "groups": {"count": size["groups"], "keep": size["keep_groups"]}},
+                   "expert": {"ff": size["ff"]}, "shared": {"ff": size["shared_ff"]}}}
+    return RapolixConfig.from_dict({"architecture": "Rapolix", "vocab": COMPARE_VOCAB, "width": width, "streams": size["streams"],
+                                    "norm": {"eps": 1e-6}, "logit_softcap": 30.0,
+                                    "layers": [{"type": "parallel", "mixer": mixer, "mlp": mlp[kind]}
+                                               for kind in _rapolix_kinds(size, layers or len(size["kinds"]))]})
+
+
+def rapolix_twin(size: dict, layers: int):
+    """(label, size, configuration, cost function) of the closest design with as many weights; None for a mix of kinds."""
+    kinds = set(size["kinds"])
+    if len(kinds) > 1:
+        return None
+    width, heads, kv_heads = size["width"], size["heads"], size["kv_heads"]
+    if kinds == {"dense"}:
+        # as many value channels in the recurrence as the recurrent branch has; two matrices in place of a gated layer's three
+        left = dict(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, scale=128 ** -0.5, mask={"size": size["window"]})
+        right = dict(heads=width // 128, kv_heads=kv_heads, dim=128, vdim=128, conv=4)
+        twin = dict(width=width, ff=size["dense_ff"] * 3 // 2, parallel=dict(left=left, right=right, left_scale=0.5, right_scale=0.5),
+                    wkv=None, kinds=("parallel",) * len(size["kinds"]))
+        return "vibepel", twin, vibepel_config(twin, layers), vibepel_step_cost
+    # gated experts of two thirds the width have as many weights
+    attention = dict(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, conv=4, scale=128 ** -0.5, bias_max=128, buckets=32,
+                     mask={"size": size["window"]})
+    twin = dict(width=width, attention=attention, retention=None, mamba2=None, experts=size["experts"], top=size["top"],
+                ff=size["ff"] * 2 // 3, shared_ff=size["shared_ff"] * 2 // 3, groups=8, keep=4, dense_ff=0, moe=True,
+                kinds=("attention",) * len(size["kinds"]))
+    return "dozotar", twin, dozotar_config(twin, layers), dozotar_step_cost
+
+
+def rapolix_step_cost(size: dict, layers: int, tokens: int, sequences: int, context: float):
+    """(bytes, FLOPs) of one step in which each of ``sequences`` requests brings tokens / sequences new tokens behind
+    ``context`` cached ones: bytes = every weight the step touches once (of the routed experts the expected number of distinct
+    ones its tokens choose) + the cached rows inside the window and in front of it that attention reads + the states read and
+    written; FLOPs = the products of the tokens (identity outputs have none) + attention per (query, key) pair + a multiply-add
+    and the gates per channel of the recurrence."""
+    width, heads, kv, window, keep = size["width"], size["heads"], size["kv_heads"], size["window"], size["keep"]
+    outputs = size["experts"] + size["identity"]
+    per_sequence = tokens / sequences
+    total_bytes = COMPARE_VOCAB * width * 2.0
+    flops = 0.0
+    distinct = size["experts"] * (1.0 - (1.0 - size["top"] / outputs) ** tokens)
+    for kind in _rapolix_kinds(size, layers):
+        weights = (2 * heads * 128 + 2 * kv * 128) * width + width * heads * 128           # q, g, k, v and the output
+        weights += 2 * width * width + 2 * 128 * width + width * width                      # y, x, both gates, the output
+        total_bytes += sequences * min(context + per_sequence, window + keep) * kv * 256 * 2.0 + sequences * width * 4.0 * 2
+        pairs = sequences * sum(min(context + i + 1, window + keep) for i in range(int(per_sequence)))
+        flops += 2.0 * heads * 256 * pairs + tokens * width * 16.0
+        if kind == "dense":
+            weights += 3 * width * size["dense_ff"]
+        else:
+            weights += 2 * width * size["shared_ff"] + outputs * width
+            total_bytes += 2.0 * 2 * width * distinct * size["ff"]
+            flops += 2.0 * tokens * 2 * width * size["top"] * size["experts"] / outputs * size["ff"]
+        total_bytes += 2.0 * weights
+        flops += 2.0 * tokens * weights
+    return total_bytes, flops
