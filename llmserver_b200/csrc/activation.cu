@@ -37,6 +37,18 @@ __device__ __forceinline__ int gate_column(int column, int group) {
     return group > 0 ? (column / group) * 2 * group + column % group : column;
 }
 
+template <int COUNT>
+__device__ __forceinline__ void add_bias(const float* __restrict__ bias, float (&values)[COUNT]) {
+#pragma unroll
+    for (int i = 0; i < COUNT; i += 4) {
+        const float4 four = *reinterpret_cast<const float4*>(bias + i);
+        values[i] += four.x;
+        values[i + 1] += four.y;
+        values[i + 2] += four.z;
+        values[i + 3] += four.w;
+    }
+}
+
 template <typename T, int ACT>
 __global__ void silu_mul_vec_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int intermediate,
                                     size_t total_vectors, int group, const float* __restrict__ bias) {
@@ -61,15 +73,10 @@ __global__ void silu_mul_vec_kernel(const T* __restrict__ gate_up, T* __restrict
         Vec16<T>::load(src_w, gate_w);
         Vec16<T>::load(src_w + to_up, up_w);
         if (bias) {
-            const float* bias_v = bias + gate_column(column_v, group);
-            const float* bias_w = bias + gate_column(column_w, group);
-#pragma unroll
-            for (int i = 0; i < kCount; ++i) {
-                gate_v[i] += bias_v[i];
-                up_v[i] += bias_v[to_up + i];
-                gate_w[i] += bias_w[i];
-                up_w[i] += bias_w[to_up + i];
-            }
+            add_bias<kCount>(bias + gate_column(column_v, group), gate_v);
+            add_bias<kCount>(bias + gate_column(column_v, group) + to_up, up_v);
+            add_bias<kCount>(bias + gate_column(column_w, group), gate_w);
+            add_bias<kCount>(bias + gate_column(column_w, group) + to_up, up_w);
         }
 #pragma unroll
         for (int i = 0; i < kCount; ++i) result[i] = gate_times<T, ACT>(gate_v[i], up_v[i]);
@@ -107,7 +114,7 @@ static int glu_launch(const void* gate_up, void* out, int n_rows, int intermedia
     }
     const int per_vector = dtype == LLM_F32 ? 4 : 8;
     const int threads = 256;
-    const bool vector_form = intermediate % per_vector == 0 && group % per_vector == 0 && aligned16(gate_up) && aligned16(out);
+    const bool vector_form = intermediate % per_vector == 0 && group % per_vector == 0 && aligned16(gate_up) && aligned16(out) && aligned16(bias);
     const size_t work = vector_form ? (size_t)n_rows * (intermediate / per_vector) : (size_t)n_rows * intermediate;
     size_t blocks = (work + threads - 1) / threads;
     if (vector_form) blocks = (blocks + 1) / 2;      // two vectors per thread and turn

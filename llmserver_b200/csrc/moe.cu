@@ -58,7 +58,18 @@ __device__ __forceinline__ void choose_experts(float* score, float* choice, cons
         // a lane looks after whole groups: it ranks each of them among all (ties: the lower index) and, when `keep` groups
         // are better, takes its experts out of the choice; every rank is formed before anything is taken out
         const int size = experts / rule.groups;
-        for (int first = 0; first < rule.groups; first += 32) {
+        if (rule.groups <= 32) {      // a lane per group: the ranks from one another's best by shuffles
+            float own = -INFINITY;
+            if (lane < rule.groups)
+                for (int e = 0; e < size; ++e) own = fmaxf(own, choice[lane * size + e]);
+            int better = 0;
+            for (int other = 0; other < rule.groups; ++other) {
+                const float theirs = __shfl_sync(0xffffffffu, own, other);
+                better += theirs > own || (theirs == own && other < lane);
+            }
+            if (lane < rule.groups && better >= rule.keep)
+                for (int e = 0; e < size; ++e) choice[lane * size + e] = -INFINITY;
+        } else for (int first = 0; first < rule.groups; first += 32) {
             const int g = first + lane;
             bool out = false;
             if (g < rule.groups) {

@@ -29,7 +29,7 @@ __global__ void norm_rope_units_kernel(T* __restrict__ qkv, int row_width, const
                                        int n_q_heads, int n_kv_heads, int maps, int q_dim, int k_dim, int value_dim,
                                        int page_size, int num_pages, int write_cache, int* __restrict__ error_flag,
                                        int rotary_dim, int max_dim, int k_norm_dim, int q_rot_start, int k_rot_start,
-                                       int interleaved, float temp_coef, int temp_every) {
+                                       int interleaved, float temp_coef, int temp_every, int first_unit) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float unit_values[];     // [warps][max_dim]
@@ -50,7 +50,7 @@ __global__ void norm_rope_units_kernel(T* __restrict__ qkv, int row_width, const
     const int q_units = n_q_heads * maps, k_units = n_kv_heads * maps;
     const int total_units = q_units + k_units + (value_dim > 0 ? n_kv_heads : 0);
     T* row = qkv + (size_t)token * row_width;
-    for (int unit = blockIdx.y * warps + warp; unit < total_units; unit += gridDim.y * warps) {
+    for (int unit = first_unit + blockIdx.y * warps + warp; unit < total_units; unit += gridDim.y * warps) {
         const bool is_q = unit < q_units;
         const bool is_k = !is_q && unit < q_units + k_units;
         int dim, column;
@@ -163,7 +163,11 @@ LLM_EXPORT int llm_norm_rope_units(void* qkv, int row_width, const float* bias, 
         llm_set_error("norm_rope_units: units of %d elements need %zu bytes of shared memory", max_dim, shared);
         return LLM_REFUSED;
     }
-    const int total_units = (n_q_heads + n_kv_heads) * maps + (value_dim > 0 ? n_kv_heads : 0);
+    // queries that stay where they lie and as they are: the blocks begin with the keys
+    const bool queries_stay = !q_out && !q_weight && !bias && temp_every <= 0 && (rotary_dim == 0 || q_rot_start < 0);
+    const int first_unit = queries_stay ? n_q_heads * maps : 0;
+    const int total_units = (n_q_heads + n_kv_heads) * maps + (value_dim > 0 ? n_kv_heads : 0) - first_unit;
+    if (total_units <= 0) return LLM_OK;
     int slices = (total_units + warps - 1) / warps;
     if (n_tokens >= 1024 && slices > 2) slices = 2;      // long prompts: fewer, longer-lived blocks
     dim3 grid(n_tokens, slices);
@@ -175,7 +179,7 @@ LLM_EXPORT int llm_norm_rope_units(void* qkv, int row_width, const float* bias, 
         llm_launch(norm_rope_units_kernel<T, W>, grid, warps * 32, shared, stream, (T*)qkv, row_width, bias, (const W*)q_weight,
                    (const W*)k_weight, eps, inv_freq, positions, seq_of_token, block_tables, max_blocks, (T*)q_out, (T*)k_pages,
                    (T*)v_pages, n_q_heads, n_kv_heads, maps, q_dim, k_dim, value_dim, page_size, num_pages, write_cache, error_flag,
-                   rotary_dim, max_dim, k_norm_dim, q_rot_start, k_rot_start, interleaved, temp_coef, temp_every);
+                   rotary_dim, max_dim, k_norm_dim, q_rot_start, k_rot_start, interleaved, temp_coef, temp_every, first_unit);
     });
     return llm_check_launch("norm_rope_units");
 }

@@ -4,7 +4,7 @@ from __future__ import annotations
 from .base import Block
 import torch
 
-from ..weights.declare import NORM, WIDE, WeightDecl
+from ..weights.declare import MIXING, NORM, WeightDecl
 from .norm import NormedDelta, ScaledDelta, StreamsDelta, add_and_read
 from .registry import BLOCKS
 
@@ -203,8 +203,8 @@ class HyperConnectionsBlock(Block):
     def declare_weights(cls, params):
         count, wanted = int(params["streams"]), {}
         for _, prefix in cls._connections(params):
-            wanted.update({prefix + "in": WeightDecl((count,), WIDE), prefix + "out": WeightDecl((count,), WIDE),
-                           prefix + "mix": WeightDecl((count, count), WIDE)})
+            wanted.update({prefix + "in": WeightDecl((count,), MIXING), prefix + "out": WeightDecl((count,), MIXING),
+                           prefix + "mix": WeightDecl((count, count), MIXING)})
         return wanted
 
     def __init__(self, params, parts, weights=None):

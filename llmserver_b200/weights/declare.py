@@ -9,6 +9,8 @@ NORM = "norm"       # random mode: 1 + N(0, 0.1)
 OFFSET = "offset"   # a norm weight stored as its distance from one; random mode: N(0, 0.1)
 TABLE = "table"     # integer table (kept as int32)
 WIDE = "wide"       # always held in float32, whatever the compute dtype (routers, per-head scalars); random mode: N(0, 0.02)
+MIXING = "mixing"   # coefficients between residual streams, held in float32 as WIDE; random mode: N(0, 0.1) around the identity (a
+                    # matrix) or around one (a vector), so that the streams stay of their size
 
 
 @dataclass(frozen=True)

@@ -14,7 +14,7 @@ from typing import Dict
 
 import torch
 
-from .declare import MATRIX, NORM, OFFSET, TABLE, WIDE, WeightDecl, declared_weights
+from .declare import MATRIX, MIXING, NORM, OFFSET, TABLE, WIDE, WeightDecl, declared_weights
 
 
 def _tensor_seed(seed: int, name: str) -> int:
@@ -39,6 +39,8 @@ def random_tensor(name: str, declaration: WeightDecl, seed: int, device="cpu") -
         return values.mul_(0.1).add_(1.0)
     if declaration.kind == OFFSET:
         return values.mul_(0.1)
+    if declaration.kind == MIXING:
+        return values.mul_(0.1).add_(torch.eye(declaration.shape[0], device=device) if len(declaration.shape) == 2 else 1.0)
     return values.mul_(0.02)
 
 
@@ -52,7 +54,7 @@ class RandomSource:
     def get(self, name: str) -> torch.Tensor:
         declaration = self.wanted[name]
         tensor = random_tensor(name, declaration, self.seed, self.device)
-        if declaration.kind == WIDE:
+        if declaration.kind in (WIDE, MIXING):
             # what a bfloat16 checkpoint would hold, widened: the values do not depend on the compute dtype
             return tensor.to(torch.bfloat16).to(torch.float32)
         return tensor if declaration.kind == TABLE else tensor.to(self.dtype)
