@@ -17,7 +17,8 @@
 //      the token's slot of the K pages [page, Hkv, slot, M * Dk]; value heads (bias added) into the V pages
 //      [page, Hkv, slot, Dv].
 // Each of bias, norms, rotation and values may be absent (Dv = 0: a cache of keys alone, as for a latent that serves as
-// key and value).  Sums, angles and products are 32-bit; every element is rounded once, when it is stored.
+// key and value).  Sums, angles and products are 32-bit; every element is rounded once, when it is stored.  When nothing is
+// left to do but to cache keys and values as they were projected, a copy kernel moves them in 16-byte pieces.
 #include "common.cuh"
 
 template <typename T, typename W>
@@ -120,6 +121,30 @@ __global__ void norm_rope_units_kernel(T* __restrict__ qkv, int row_width, const
     }
 }
 
+// Keys and values as they lie behind the queries in a token's row into the token's slots of the pages.
+__global__ void kv_copy_kernel(const uint4* __restrict__ rows, int row_pieces, int first_piece, const int* __restrict__ positions,
+                               const int* __restrict__ seq_of_token, const int* __restrict__ block_tables, int max_blocks,
+                               uint4* __restrict__ k_pages, uint4* __restrict__ v_pages, long long total, int n_kv_heads, int k_pieces, int v_pieces,
+                               int page_size, int num_pages, int* __restrict__ error_flag) {
+    pdl_trigger();
+    pdl_wait();
+    const int per_token = n_kv_heads * (k_pieces + v_pieces);
+    for (long long e = (long long)blockIdx.x * blockDim.x + threadIdx.x; e < total; e += (long long)gridDim.x * blockDim.x) {
+        const int token = (int)(e / per_token), piece = (int)(e % per_token);
+        const uint4 value = rows[(size_t)token * row_pieces + first_piece + piece];
+        const int position = positions[token];
+        const int page = block_tables[(size_t)seq_of_token[token] * max_blocks + position / page_size];
+        if (page < 0 || page >= num_pages) {
+            atomicExch(error_flag, 1 + token);
+            continue;
+        }
+        const bool is_k = piece < n_kv_heads * k_pieces;
+        const int inside = is_k ? piece : piece - n_kv_heads * k_pieces, pieces = is_k ? k_pieces : v_pieces;
+        const size_t slot = ((size_t)page * n_kv_heads + inside / pieces) * page_size + position % page_size;
+        (is_k ? k_pages : v_pages)[slot * pieces + inside % pieces] = value;
+    }
+}
+
 LLM_EXPORT int llm_norm_rope_units(void* qkv, int row_width, const float* bias, const void* q_weight, const void* k_weight,
                                    float eps, const float* inv_freq, const int* positions, const int* seq_of_token,
                                    const int* block_tables, int max_blocks, void* q_out, void* k_pages, void* v_pages,
@@ -168,6 +193,18 @@ LLM_EXPORT int llm_norm_rope_units(void* qkv, int row_width, const float* bias, 
     const int first_unit = queries_stay ? n_q_heads * maps : 0;
     const int total_units = (n_q_heads + n_kv_heads) * maps + (value_dim > 0 ? n_kv_heads : 0) - first_unit;
     if (total_units <= 0) return LLM_OK;
+    const int per_piece = dtype == LLM_F32 ? 4 : 8, key = maps * k_dim;
+    if (queries_stay && !k_weight && (rotary_dim == 0 || k_rot_start < 0) && row_width % per_piece == 0 && (n_q_heads * maps * q_dim) % per_piece == 0 &&
+        key % per_piece == 0 && value_dim % per_piece == 0 && aligned16(qkv) && aligned16(k_pages) && aligned16(v_pages)) {
+        if (!write_cache) return LLM_OK;
+        const long long total = (long long)n_tokens * n_kv_heads * ((key + value_dim) / per_piece);
+        long long blocks = (total + 255) / 256;
+        if (blocks > 148 * 8) blocks = 148 * 8;
+        llm_launch(kv_copy_kernel, (unsigned)blocks, 256, 0, stream, (const uint4*)qkv, row_width / per_piece, n_q_heads * maps * q_dim / per_piece,
+                   positions, seq_of_token, block_tables, max_blocks, (uint4*)k_pages, (uint4*)v_pages, total, n_kv_heads, key / per_piece,
+                   value_dim / per_piece, page_size, num_pages, error_flag);
+        return llm_check_launch("norm_rope_units");
+    }
     int slices = (total_units + warps - 1) / warps;
     if (n_tokens >= 1024 && slices > 2) slices = 2;      // long prompts: fewer, longer-lived blocks
     dim3 grid(n_tokens, slices);

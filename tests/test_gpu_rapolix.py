@@ -483,6 +483,36 @@ def test_window_edges_and_kept_tokens_in_prompts_and_decoding(dtype, heads, kv_h
             assert spike_weight > 0.9       # a kernel that missed the key would be far off
 
 
+@pytest.mark.parametrize("dtype", TORCH_DTYPES)
+@pytest.mark.parametrize("heads,kv_heads,dim,vdim,gate", [(4, 2, 16, 24, 8), (3, 3, 128, 128, 40), (2, 1, 9, 7, 0), (6, 2, 8, 12, 4)])
+def test_keys_and_values_cached_as_projected(dtype, heads, kv_heads, dim, vdim, gate):
+    """Nothing is normalised or turned: keys and values go to their (shuffled) pages in 16-byte pieces where the sizes allow it; queries,
+    what lies behind the values and everybody else's pages stay as they are, and so does the cache when it may not be written."""
+    from llmserver_b200 import ops
+    generator = torch.Generator().manual_seed(heads * dim)
+    pieces, page_size = [(0, 21), (13, 5), (40, 1)], 8
+    used = (heads + kv_heads) * dim + kv_heads * vdim
+    packed = torch.randn((27, used + gate), generator=generator).to(dtype)
+    order = torch.randperm(20, generator=generator).tolist()
+    tables = [[order.pop() for _ in range(-(-(before + now) // page_size))] for before, now in pieces]
+    batch = _batch(pieces, [0] * 3, tables)
+    for write in (True, False):
+        k_pages, v_pages = (torch.full((20, kv_heads, page_size, size), 5.0, dtype=dtype, device=DEVICE) for size in (dim, vdim))
+        rows = packed.clone().to(DEVICE)
+        ops.norm_rope_units(rows, batch.positions, batch.seq_of_token, batch.block_tables[0], k_pages, v_pages, heads, kv_heads, 1, dim, dim, vdim,
+                            batch.error_flag, write_cache=write)
+        assert torch.equal(rows.cpu(), packed) and int(batch.error_flag.item()) == 0
+        want_k, want_v, at = torch.full_like(k_pages.cpu(), 5.0), torch.full_like(v_pages.cpu(), 5.0), 0
+        for (before, now), table in zip(pieces, tables):
+            for position in range(before, before + now):
+                if write:
+                    k = packed[at, heads * dim:(heads + kv_heads) * dim].view(kv_heads, dim)
+                    want_k[table[position // page_size], :, position % page_size] = k
+                    want_v[table[position // page_size], :, position % page_size] = packed[at, (heads + kv_heads) * dim:used].view(kv_heads, vdim)
+                at += 1
+        assert torch.equal(k_pages.cpu(), want_k) and torch.equal(v_pages.cpu(), want_v)
+
+
 ROUTERS = [(6, 2, None, 0), (7, 3, (3, 2), 2), (8, 4, (2, 1), 0), (13, 5, (4, 4), 3), (12, 1, (14, 1), 2), (60, 6, (8, 3), 4), (33, 8, (9, 2), 3), (5, 6, None, 2)]
 
 
